@@ -269,10 +269,10 @@ enum { SSDK_DT_F32 = 0, SSDK_DT_BF16 = 1 };
 enum { SSDK_MIX_WKV = 0, SSDK_MIX_MLSTM = 1, SSDK_MIX_LATENT_ATTN = 2,
        SSDK_MIX_RGLRU = 3,        /* gated diagonal linear recurrence behind a short convolution, times a gelu branch */
        SSDK_MIX_SELECTIVE = 4,    /* selective scan (input-dependent step, B, C) behind a short convolution, silu gate */
-       SSDK_MIX_ATTN_DELTA = 5,   /* grouped-query sink attention and a gated delta rule side by side on the same input */
+       SSDK_MIX_ATTN_DELTA = 5,   /* grouped-query attention and a gated delta rule side by side on the same input (variants: pair_* and d_* fields) */
        SSDK_MIX_ATTENTION = 6 };  /* grouped-query attention alone: biased q | k | v projections behind a short convolution,
                                    * rotate-half rotation of the first rot_dims entries, optional sliding window, learned sink */
-enum { SSDK_MLP_NONE = 0, SSDK_MLP_MOE = 1, SSDK_MLP_GLU = 2, /* dense: down(gelu_tanh(gate h) * (up h)) */
+enum { SSDK_MLP_NONE = 0, SSDK_MLP_MOE = 1, SSDK_MLP_GLU = 2, /* dense: down(act(gate h) * (up h)), act = ff_act (silu or gelu_tanh) */
        SSDK_MLP_FFN = 3 };        /* dense, not gated: down(act(up h + b_up)) + b_down, act = ff_act */
 /* activations of the feed-forward kernels; CLAMPED is the limited GLU g sigmoid(1.702 g) (u + 1) */
 enum { SSDK_ACT_CLAMPED = 0, SSDK_ACT_SILU = 1, SSDK_ACT_GELU_TANH = 2, SSDK_ACT_RELU2 = 3, /* relu(z)^2 */
@@ -281,6 +281,8 @@ enum { SSDK_ACT_CLAMPED = 0, SSDK_ACT_SILU = 1, SSDK_ACT_GELU_TANH = 2, SSDK_ACT
 enum { SSDK_BLOCK_PARALLEL_PRENORM = 0,  /* x += ls1 * mixer(h) + ls2 * ff(h), h = norm(x) */
        SSDK_BLOCK_SERIAL_POSTNORM = 1,   /* x += m * norm1(mixer(x)); x += m * norm2(ff(x)): the sublayers read x itself */
        SSDK_BLOCK_PARALLEL_TWO_NORMS = 2, /* x += mixer(norm1(x)) + ff(norm2(x)): one statistic, two weights, no layer scales */
+       SSDK_BLOCK_SERIAL_PRENORM = 4,    /* x += mixer(norm1(x)); x += ff(norm2(x)).  streams > 0: the residual is `streams` copies x_s, a
+                                          * sublayer reads norm(sum_s in[s] x_s) and its result y enters as x_t = sum_s mix[s, t] x_s + out[t] y */
        SSDK_BLOCK_PARALLEL_ONE_NORM = 3 }; /* h = norm(x); x += g1 * mixer(h + conv1(h)) + g2 * ff(h + conv2(h)): plain norm weight; the
                                             * input convolutions (canon_taps > 0) and the gates g = sigmoid(W_g h + b) (gated_residual) are optional */
 
@@ -340,11 +342,12 @@ enum {
   SSDK_HT_SEL_ALOG,      /* [inner, state] */
   SSDK_HT_SEL_D,         /* [inner] */
   /* attention + delta rule pair: ONE stacked input projection,
-   * rows: attn q [H D] | k [G D] | v [G V] | gate [H V] | delta q [Gd Dd] | k [Gd Dd] | v [Hd Vd] | gate [Hd Vd] | beta [Hd] | a [Hd] */
+   * rows: attn q [H D] | k [G D] | v [G V] | gate [H V] (pair_gate) | delta q [Gd Dd] | k [Gd Dd] | v [Hd Vd] | gate [Hd Vd] (d_gate_rank = 0) |
+   * beta [Hd] | a [Hd] (d_decay_rank = 0) | decay bottleneck [d_decay_rank] | gate bottleneck [d_gate_rank] */
   SSDK_HT_PAIR_IN,
   SSDK_HT_ATTN_OUT,      /* [width, H V] */
   SSDK_HT_DELTA_ALOG,    /* [Hd] */
-  SSDK_HT_DELTA_DT_B,    /* [Hd] */
+  SSDK_HT_DELTA_DT_B,    /* [Hd], or [Hd Dd] with a decay per key channel (d_decay_rank > 0) */
   /* latent attention with full-rank queries (q_rank = 0): ONE stacked input projection,
    * rows: q [H (D + R)] | dkv [kv_rank + rot_dim] (absent when kv_from >= 0) | output gate [H V] (when out_gate) */
   SSDK_HT_LAT_IN,
@@ -364,6 +367,18 @@ enum {
   SSDK_HT_CANON_W,       /* [2, width, canon_taps]: taps of the mixer's input convolution, then of the feed-forward's */
   SSDK_HT_RES_GATE,      /* [2 width, width]: rows of the mixer's residual gate, then of the feed-forward's */
   SSDK_HT_RES_GATE_B,    /* [2 width] */
+  /* attention of the pair: taps of its convolution over q | k | v (pair_conv > 0; the bias is SSDK_HT_ATTN_IN_B) and the weights of the
+   * RMS norms over the whole query and key projections (qk_norm = 2) */
+  SSDK_HT_ATTN_CONV_W,   /* [H D + G D + G V, pair_conv] */
+  SSDK_HT_ATTN_QK_NORM,  /* [H D + G D]: query weight, then key weight */
+  /* delta rule: second halves of the low-rank projections */
+  SSDK_HT_DELTA_A2,      /* [Hd Dd, d_decay_rank] */
+  SSDK_HT_DELTA_G2,      /* [Hd Vd, d_gate_rank] */
+  SSDK_HT_PAIR_NORM,     /* [2, width] weights of the norms on the attention's and the delta rule's result (pair_norm) */
+  /* residual streams of SSDK_BLOCK_SERIAL_PRENORM: one set for the mixer, one for the feed-forward (absent without one) */
+  SSDK_HT_HC_IN,         /* [1 or 2, streams] */
+  SSDK_HT_HC_OUT,        /* [1 or 2, streams] */
+  SSDK_HT_HC_MIX,        /* [1 or 2, streams (from), streams (to)] */
   SSDK_HT_COUNT
 };
 
@@ -380,7 +395,8 @@ typedef struct ssdk_hyb_layer_cfg {
   float   route_scale, limit, shared_limit;
   /* grouped-query attention (SSDK_MIX_ATTN_DELTA uses heads / dim / vdim / rot_dims / rot_base / attn_scale above) */
   int32_t kv_heads;                  /* key/value heads; query head h reads head h / (heads / kv_heads) */
-  int32_t qk_norm;                   /* 1: q and k divided by their RMS over dim after the rotation */
+  int32_t qk_norm;                   /* 1: q and k divided by their RMS over dim after the rotation; 2: RMS norm with a weight over the whole
+                                      * query (key) projection before the rotation */
   float   sink;                      /* constant added to the softmax denominator (0: plain softmax; 1: a sink of score 0) */
   float   yarn_factor;               /* 0: no frequency scaling; else YaRN with the three values below */
   float   yarn_original, yarn_fast, yarn_slow;
@@ -410,6 +426,14 @@ typedef struct ssdk_hyb_layer_cfg {
   int32_t expert_glu;                /* 1: experts are down(act(gate h) * (up h)), SSDK_HT_EXPERT_IN / SHARED_IN hold gate | up rows;
                                       * 0: down(act(up h)), they hold the up rows only */
   int32_t route_top_softmax;         /* 1: the choice is made on the raw logits and the weights are the softmax over the chosen logits */
+  int32_t chunk;                     /* attention: a query at position p reads the keys of its own chunk, floor(p / chunk) * chunk .. p; 0: no chunks */
+  /* variants of SSDK_MIX_ATTN_DELTA */
+  int32_t pair_gate;                 /* 1: the attention's heads are multiplied by sigmoid(W_g h) before their output projection */
+  int32_t pair_conv;                 /* taps of a convolution (no activation) over the attention's q | k | v; 0: none */
+  int32_t pair_norm;                 /* 1: both results are RMS-normed with weights (SSDK_HT_PAIR_NORM) before left_scale / right_scale */
+  int32_t d_decay_rank;              /* 0: one decay per head; r: one per head and key channel from a rank-r projection */
+  int32_t d_gate_rank;               /* 0: output gate straight from h; r: from a rank-r projection */
+  int32_t d_gate_act;                /* output gate of the delta rule: 0 silu, 1 sigmoid */
 } ssdk_hyb_layer_cfg;
 
 typedef struct ssdk_hyb_cfg {
@@ -425,6 +449,8 @@ typedef struct ssdk_hyb_cfg {
   float   residual_mult;     /* m of SSDK_BLOCK_SERIAL_POSTNORM */
   int32_t canon_taps;        /* SSDK_BLOCK_PARALLEL_ONE_NORM: taps of the sublayers' input convolutions (0: none) */
   int32_t gated_residual;    /* SSDK_BLOCK_PARALLEL_ONE_NORM: 1 = each sublayer's result is multiplied by sigmoid(W_g h + b) */
+  int32_t streams;           /* SSDK_BLOCK_SERIAL_PRENORM: residual streams (0: one plain residual) */
+  float   logit_scale;       /* logits = (head h) * logit_scale */
 } ssdk_hyb_cfg;
 
 typedef struct ssdk_hyb_engine* ssdk_hyb_handle;

@@ -28,7 +28,7 @@ struct ConvArgs {
   const float* in;      // [M, ld_in] rows before the convolution; channel c is column c
   int ld_in;
   const void* in_bias;  // [C] T added to every input row (not to the zeros before the sequence), or nullptr
-  const void* w;        // [C, taps] T
+  const void* w;        // [C, taps] T, or nullptr: weight 1 (one tap)
   const void* bias;     // [C] T added to the result, or nullptr
   float* out;           // [M, ld_out] fp32, or nullptr
   int ld_out;
@@ -51,7 +51,7 @@ SSDK_DEVINL float conv_at(const ConvArgs& p, const Ragged& rg, int m, int s, int
     float v;
     if (back <= t) v = p.in[(size_t)(m - back) * p.ld_in + c] + ib;
     else v = carried ? hist[(size_t)(p.taps - 1 - (back - t)) * p.C + c] : 0.f;
-    acc = fmaf(ld_f<T>((const T*)p.w + (size_t)c * p.taps + j), v, acc);
+    acc = fmaf(p.w ? ld_f<T>((const T*)p.w + (size_t)c * p.taps + j) : 1.f, v, acc);
   }
   return acc;
 }
@@ -368,20 +368,22 @@ __global__ void selective_scan_kernel(const SelScanArgs p, const Ragged rg) {
 // ---------------------------------------------------------------------------------------------- gated delta rule
 struct DeltaPrepArgs {
   ConvArgs conv;          // over the q | k | v columns (C = 2 G D + H V); out / out_t unused
-  const float* ba; int ld_ba;  // [M, ...]: beta pre-activations in columns [0, H), decay pre-activations in [H, 2H)
+  const float* b; int ld_b;    // [M, ...]: beta pre-activations in columns [0, H)
+  const float* a; int ld_a;    // decay pre-activations: [M, ...] columns [0, H), or (per_channel) [M, H D]
   const void* A_log;      // [H] T
-  const void* dt_bias;    // [H] T
+  const void* dt_bias;    // [H] T, or (per_channel) [H D]
   float* q;               // [M, G D] unit vectors * q_scale
   float* k;               // [M, G D] unit vectors
   float* v;               // [M, H V]
   float* beta;            // [M, H]
-  float* decay;           // [M, H]
-  int H, G, D, V;
+  float* decay;           // g - 1 (exact also where the decay g is within an ulp of 1): [M, H], or (per_channel) [M, H D]; may be `a` itself
+  int H, G, D, V, per_channel;
   float q_scale, unit_eps;
 };
 
-// grid (M, 2 G + H): unit u < G is a query head, u < 2 G a key head, the rest value heads; one CTA convolves the unit's
-// channels (SiLU), and makes a query or key head a unit vector.  dynamic shared memory: max(D, V) floats.
+// grid (M, 2 G + H (+ H when per_channel)): unit u < G is a query head, u < 2 G a key head, then value heads, then the decays of
+// the heads' key channels; one CTA convolves the unit's channels (SiLU), and makes a query or key head a unit vector.
+// dynamic shared memory: max(D, V) floats.
 template <typename T>
 __global__ void delta_prep_kernel(const DeltaPrepArgs p, const Ragged rg) {
   extern __shared__ float dp_sm[];
@@ -390,10 +392,21 @@ __global__ void delta_prep_kernel(const DeltaPrepArgs p, const Ragged rg) {
   const int GD = p.G * p.D, HV = p.H * p.V;
   if (unit == 0) {
     for (int h = threadIdx.x; h < p.H; h += blockDim.x) {
-      p.beta[(size_t)m * p.H + h] = sigmoid_f(p.ba[(size_t)m * p.ld_ba + h]);
-      const float sp = softplus_f(p.ba[(size_t)m * p.ld_ba + p.H + h] + ld_f<T>((const T*)p.dt_bias + h));
-      p.decay[(size_t)m * p.H + h] = expf(-expf(ld_f<T>((const T*)p.A_log + h)) * sp);
+      p.beta[(size_t)m * p.H + h] = sigmoid_f(p.b[(size_t)m * p.ld_b + h]);
+      if (!p.per_channel) {
+        const float sp = softplus_f(p.a[(size_t)m * p.ld_a + h] + ld_f<T>((const T*)p.dt_bias + h));
+        p.decay[(size_t)m * p.H + h] = expm1f(-expf(ld_f<T>((const T*)p.A_log + h)) * sp);
+      }
     }
+  }
+  if (unit >= 2 * p.G + p.H) {  // the decays of one head's key channels
+    const int h = unit - 2 * p.G - p.H;
+    const float rate = -expf(ld_f<T>((const T*)p.A_log + h));
+    for (int d = threadIdx.x; d < p.D; d += blockDim.x) {
+      const int c = h * p.D + d;
+      p.decay[(size_t)m * p.H * p.D + c] = expm1f(rate * softplus_f(p.a[(size_t)m * p.ld_a + c] + ld_f<T>((const T*)p.dt_bias + c)));
+    }
+    return;
   }
   if (unit >= 2 * p.G) {  // a value head: convolution and SiLU only
     const int c0 = 2 * GD + (unit - 2 * p.G) * p.V;
@@ -418,156 +431,200 @@ __global__ void delta_prep_kernel(const DeltaPrepArgs p, const Ragged rg) {
 struct DeltaArgs {
   const float* q; const float* k;    // [M, G D]
   const float* v;                    // [M, H V]
-  const float* beta; const float* decay;  // [M, H]
+  const float* beta;                 // [M, H]
+  const float* decay;                // g - 1: [M, H], or one per key channel [M, H D]
   float* o;                          // [M, H V]
-  float* S; size_t slot_stride;      // [H, D, V] per slot
+  float* S; size_t slot_stride;      // [H, V, D] per slot: a column of the state (one value channel) is contiguous
   int H, G, D, V;
+  int vec;                           // D, V, row offsets and the slot are whole 16-byte pieces
 };
 
-constexpr int kDeltaRows = 16;  // rows staged together (two such buffers: the next chunk arrives under the current one's walk)
+constexpr int kDeltaRows = 16;   // rows staged together (two such buffers: the next chunk arrives under the current one's walk)
+constexpr int kDeltaWarps = 4;
 
-// shared memory of delta_scan_kernel<DR> with G row groups (DR == 0: G = 1 and the state itself lives there)
-inline size_t delta_scan_smem(int D, int Vr, int DR, int G) {
-  const int DP = DR > 0 ? DR * G : D;
-  return ((size_t)(DR > 0 ? 0 : D * Vr) + (size_t)2 * kDeltaRows * (2 * DP + Vr + 2) + (size_t)2 * G * Vr) * 4;
+// floats of one staged row: k | q (| decay per channel), DP entries each, then value columns, beta, decay per head (padded to 4)
+inline __host__ __device__ int delta_row_floats(int DP, int cols, bool per_channel) {
+  return (per_channel ? 3 : 2) * DP + (cols + 2 + 3) / 4 * 4;
+}
+inline size_t delta_scan_smem(int DP, int cols, bool per_channel) {
+  return (size_t)2 * kDeltaRows * delta_row_floats(DP, cols, per_channel) * 4;
 }
 
-// grid (n_seqs, H, column splits), block (Vr, G) with Vr a multiple of 32 columns per CTA (the columns of the state are
-// independent of one another, so a head may be spread over several CTAs): thread (j, gi) owns rows [gi DR, (gi + 1) DR)
-// of one column of the head's D x V state, in registers.  The rows' k, q, v, beta and decay arrive by cp.async, sixteen
-// rows at a time, under the walk of the previous sixteen; k and q are read from shared memory four rows at a time.
-// Both contractions over D (S^T k and S^T q) are thread-local sums over the thread's rows; with G > 1 the row groups'
-// partial sums meet in shared memory and are added in group order (two CTA barriers per row, none with G == 1).
-// Padded rows meet k = q = 0.  DR == 0: any D, one group, the column lives in shared memory.  Everything is fp32
-// whatever the model's storage type.
-template <int DR>
-__global__ void delta_scan_kernel(const DeltaArgs p, const Ragged rg) {
+// The walk over a sequence's rows.  grid (n_seqs, H, ceil(V / cols)), kDeltaWarps warps, cols = kDeltaWarps * 32 / LC.
+// The columns of the state (value channels) are independent of one another: LC neighbouring lanes share one column, lane r
+// of them holds the key channels 4 (r + LC i) .. + 3, i < NQ, in registers (D <= 4 LC NQ; padded channels meet k = q = 0).
+// Both contractions over D (S^T k and S^T q) are thread-local sums followed by a shuffle tree over the LC lanes: no CTA
+// barrier inside a row.  Rows arrive by cp.async, sixteen at a time, under the walk of the previous sixteen.  CH: one decay
+// per key channel instead of one per head.  Everything is fp32 whatever the model's storage type.
+template <int LC, int NQ, bool CH>
+__global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(const DeltaArgs p, const Ragged rg) {
   extern __shared__ __align__(16) float ds_sm[];
-  const int s = blockIdx.x, hd = blockIdx.y, g = hd / (p.H / p.G);
-  const int jl = threadIdx.x, gi = threadIdx.y, Vr = blockDim.x, NG = blockDim.y, tid = gi * Vr + jl, nthr = Vr * NG;
-  const int j = blockIdx.z * Vr + jl;  // column of the head's state
-  const int D = p.D, V = p.V, DP = DR > 0 ? DR * NG : D;
-  float* Ssm = ds_sm;                                     // [D][Vr] (DR == 0)
-  constexpr int kR = kDeltaRows;
-  const int stage = kR * (2 * DP + Vr + 2);               // floats of one staging buffer
-  float* st0 = ds_sm + (DR > 0 ? 0 : (size_t)D * Vr);     // two buffers: [rows][2 DP] k then q | [rows][Vr] v | [rows][2] beta, decay
-  float* part = st0 + 2 * stage;                          // [2][NG][Vr] partial contractions
-  float Sr[DR > 0 ? DR : 1];
+  constexpr int DP = 4 * LC * NQ, kCols = kDeltaWarps * 32 / LC, kR = kDeltaRows, kThreads = kDeltaWarps * 32;
+  const int RF = delta_row_floats(DP, kCols, CH), off_v = (CH ? 3 : 2) * DP, off_b = off_v + kCols;
+  const int s = blockIdx.x, hd = blockIdx.y, g = hd / (p.H / p.G), tid = threadIdx.x;
+  const int lr = tid % LC, jl = tid / LC, j = blockIdx.z * kCols + jl;
+  const int D = p.D, V = p.V, GD = p.G * D, HV = p.H * V, HDk = p.H * D;
   const bool col = j < V, carried = rg.pos0[s] > 0;
-  const int d0 = gi * DR;
-  float* Sg = p.S + (size_t)rg.slot[s] * p.slot_stride + (size_t)hd * D * V + (col ? j : 0);
-  if (DR > 0) {
+  float* Sg = p.S + (size_t)rg.slot[s] * p.slot_stride + ((size_t)hd * V + (col ? j : 0)) * D;
+  float4 S[NQ];
 #pragma unroll
-    for (int d = 0; d < DR; ++d) Sr[d] = (col && carried && d0 + d < D) ? Sg[(size_t)(d0 + d) * V] : 0.f;
-  } else {
-    for (int d = 0; d < D; ++d) Ssm[(size_t)d * Vr + jl] = (col && carried) ? Sg[(size_t)d * V] : 0.f;
-  }
-  // padding (rows of k and q from D up to DP, value columns beyond V) is zero in both buffers and never written again
-  for (int i = tid; i < 2 * stage; i += nthr) st0[i] = 0.f;
-  __syncthreads();
-  const int r0 = rg.cu[s], r1 = rg.cu[s + 1], GD = p.G * D, HV = p.H * V;
-  const int vcols = max(0, min(Vr, V - (int)blockIdx.z * Vr));
-  auto issue = [&](int m0, float* buf) {  // 4-byte asynchronous copies: no alignment rule beyond the element's own
-    const int nr = min(kR, r1 - m0);
-    float* kq = buf;
-    float* vs = kq + kR * 2 * DP;
-    float* bg = vs + kR * Vr;
-    for (int i = tid; i < nr * D; i += nthr) {
-      const int r = i / D, d = i - r * D;
-      cp_async4(kq + r * 2 * DP + d, p.k + (size_t)(m0 + r) * GD + g * D + d);
-      cp_async4(kq + r * 2 * DP + DP + d, p.q + (size_t)(m0 + r) * GD + g * D + d);
+  for (int i = 0; i < NQ; ++i) {
+    const int d = 4 * (lr + LC * i);
+    S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (col && carried) {
+      if (p.vec) {
+        if (d < D) S[i] = *reinterpret_cast<const float4*>(Sg + d);
+      } else {
+        if (d < D) S[i].x = Sg[d];
+        if (d + 1 < D) S[i].y = Sg[d + 1];
+        if (d + 2 < D) S[i].z = Sg[d + 2];
+        if (d + 3 < D) S[i].w = Sg[d + 3];
+      }
     }
-    for (int i = tid; i < nr * vcols; i += nthr) {
-      const int r = i / vcols, c = i - r * vcols;
-      cp_async4(vs + r * Vr + c, p.v + (size_t)(m0 + r) * HV + hd * V + blockIdx.z * Vr + c);
+  }
+  // padding (channels from D up to DP, value columns beyond V) is zero in both buffers and never written again
+  for (int i = tid; i < 2 * kR * RF; i += kThreads) ds_sm[i] = 0.f;
+  __syncthreads();
+  const int r0 = rg.cu[s], r1 = rg.cu[s + 1];
+  const int c0 = blockIdx.z * kCols, vcols = min(kCols, V - c0);
+  auto issue = [&](int m0, float* buf) {
+    const int nr = min(kR, r1 - m0);
+    if (p.vec) {
+      const int dq = D >> 2, per = (CH ? 3 : 2) * dq, vq = vcols >> 2;
+      for (int i = tid; i < nr * per; i += kThreads) {
+        const int r = i / per, x = i - r * per, part = x / dq, d = (x - part * dq) * 4;
+        const size_t m = m0 + r;
+        const float* src = part == 0 ? p.k + m * GD + g * D + d : part == 1 ? p.q + m * GD + g * D + d : p.decay + m * HDk + hd * D + d;
+        cp_async16(buf + r * RF + part * DP + d, src, true);
+      }
+      for (int i = tid; i < nr * vq; i += kThreads) {
+        const int r = i / vq, c = (i - r * vq) * 4;
+        cp_async16(buf + r * RF + off_v + c, p.v + (size_t)(m0 + r) * HV + hd * V + c0 + c, true);
+      }
+    } else {   // 4-byte copies: no alignment rule beyond the element's own
+      for (int i = tid; i < nr * D; i += kThreads) {
+        const int r = i / D, d = i - r * D;
+        const size_t m = m0 + r;
+        cp_async4(buf + r * RF + d, p.k + m * GD + g * D + d);
+        cp_async4(buf + r * RF + DP + d, p.q + m * GD + g * D + d);
+        if (CH) cp_async4(buf + r * RF + 2 * DP + d, p.decay + m * HDk + hd * D + d);
+      }
+      for (int i = tid; i < nr * vcols; i += kThreads) {
+        const int r = i / vcols, c = i - r * vcols;
+        cp_async4(buf + r * RF + off_v + c, p.v + (size_t)(m0 + r) * HV + hd * V + c0 + c);
+      }
     }
     if (tid < nr) {
-      cp_async4(bg + 2 * tid, p.beta + (size_t)(m0 + tid) * p.H + hd);
-      cp_async4(bg + 2 * tid + 1, p.decay + (size_t)(m0 + tid) * p.H + hd);
+      cp_async4(buf + tid * RF + off_b, p.beta + (size_t)(m0 + tid) * p.H + hd);
+      if (!CH) cp_async4(buf + tid * RF + off_b + 1, p.decay + (size_t)(m0 + tid) * p.H + hd);
     }
     cp_async_commit();
   };
-  issue(r0, st0);
+  issue(r0, ds_sm);
   int cur = 0;
   for (int m0 = r0; m0 < r1; m0 += kR, cur ^= 1) {
     const int nr = min(kR, r1 - m0);
     if (m0 + kR < r1) {
-      issue(m0 + kR, st0 + (cur ^ 1) * stage);
+      issue(m0 + kR, ds_sm + (cur ^ 1) * kR * RF);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
     }
     __syncthreads();
-    const float* kq = st0 + cur * stage;
-    const float* vs = kq + kR * 2 * DP;
-    const float* bg = vs + kR * Vr;
+    const float* buf = ds_sm + cur * kR * RF;
+#pragma unroll 2
     for (int r = 0; r < nr; ++r) {
-      const float* kr = kq + r * 2 * DP + d0;
-      const float* qr = kr + DP;
-      const float beta = bg[2 * r], dec = bg[2 * r + 1];
-      float o = 0.f;
-      if (DR > 0) {
-        float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+      const float* row = buf + r * RF;
+      const float4* k4 = reinterpret_cast<const float4*>(row) + lr;
+      const float beta = row[off_b], v = row[off_v + jl];
+      float dec = 0.f;
+      if (!CH) dec = row[off_b + 1];
+      float4 kk[NQ];
+      float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
 #pragma unroll
-        for (int d = 0; d < DR; d += 4) {
-          const float4 k4 = *reinterpret_cast<const float4*>(kr + d);
-          Sr[d] *= dec; Sr[d + 1] *= dec; Sr[d + 2] *= dec; Sr[d + 3] *= dec;
-          a0 = fmaf(Sr[d], k4.x, a0); a1 = fmaf(Sr[d + 1], k4.y, a1);
-          a2 = fmaf(Sr[d + 2], k4.z, a2); a3 = fmaf(Sr[d + 3], k4.w, a3);
-        }
-        float dot = (a0 + a1) + (a2 + a3);
-        if (NG > 1) {
-          part[gi * Vr + jl] = dot;
-          __syncthreads();
-          dot = part[jl];
-          for (int w = 1; w < NG; ++w) dot += part[w * Vr + jl];
-        }
-        const float u = beta * (vs[r * Vr + jl] - dot);
-        a0 = a1 = a2 = a3 = 0.f;
-#pragma unroll
-        for (int d = 0; d < DR; d += 4) {
-          const float4 k4 = *reinterpret_cast<const float4*>(kr + d);
-          const float4 q4 = *reinterpret_cast<const float4*>(qr + d);
-          Sr[d] = fmaf(k4.x, u, Sr[d]); Sr[d + 1] = fmaf(k4.y, u, Sr[d + 1]);
-          Sr[d + 2] = fmaf(k4.z, u, Sr[d + 2]); Sr[d + 3] = fmaf(k4.w, u, Sr[d + 3]);
-          a0 = fmaf(Sr[d], q4.x, a0); a1 = fmaf(Sr[d + 1], q4.y, a1);
-          a2 = fmaf(Sr[d + 2], q4.z, a2); a3 = fmaf(Sr[d + 3], q4.w, a3);
-        }
-        o = (a0 + a1) + (a2 + a3);
-        if (NG > 1) {
-          part[(NG + gi) * Vr + jl] = o;
-          __syncthreads();
-          if (gi == 0) {
-            o = part[NG * Vr + jl];
-            for (int w = 1; w < NG; ++w) o += part[(NG + w) * Vr + jl];
-          }
-        }
-      } else {
-        float dot = 0.f;
-        for (int d = 0; d < D; ++d) {
-          const float sv = Ssm[(size_t)d * Vr + jl] * dec;
-          Ssm[(size_t)d * Vr + jl] = sv;
-          dot = fmaf(sv, kr[d], dot);
-        }
-        const float u = beta * (vs[r * Vr + jl] - dot);
-        for (int d = 0; d < D; ++d) {
-          const float sv = fmaf(kr[d], u, Ssm[(size_t)d * Vr + jl]);
-          Ssm[(size_t)d * Vr + jl] = sv;
-          o = fmaf(sv, qr[d], o);
-        }
+      for (int i = 0; i < NQ; ++i) {
+        kk[i] = k4[LC * i];
+        const float4 gg = CH ? k4[DP / 2 + LC * i] : make_float4(dec, dec, dec, dec);
+        S[i].x = fmaf(S[i].x, gg.x, S[i].x); S[i].y = fmaf(S[i].y, gg.y, S[i].y);   // S g = S + S (g - 1), rounded once
+        S[i].z = fmaf(S[i].z, gg.z, S[i].z); S[i].w = fmaf(S[i].w, gg.w, S[i].w);
+        a0 = fmaf(S[i].x, kk[i].x, a0); a1 = fmaf(S[i].y, kk[i].y, a1);
+        a2 = fmaf(S[i].z, kk[i].z, a2); a3 = fmaf(S[i].w, kk[i].w, a3);
       }
-      if (col && gi == 0) p.o[(size_t)(m0 + r) * HV + hd * V + j] = o;
+      float dot = (a0 + a1) + (a2 + a3);
+#pragma unroll
+      for (int o = LC >> 1; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+      const float u = beta * (v - dot);
+      a0 = a1 = a2 = a3 = 0.f;
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) {
+        const float4 qq = k4[DP / 4 + LC * i];
+        S[i].x = fmaf(kk[i].x, u, S[i].x); S[i].y = fmaf(kk[i].y, u, S[i].y);
+        S[i].z = fmaf(kk[i].z, u, S[i].z); S[i].w = fmaf(kk[i].w, u, S[i].w);
+        a0 = fmaf(S[i].x, qq.x, a0); a1 = fmaf(S[i].y, qq.y, a1);
+        a2 = fmaf(S[i].z, qq.z, a2); a3 = fmaf(S[i].w, qq.w, a3);
+      }
+      float o = (a0 + a1) + (a2 + a3);
+#pragma unroll
+      for (int x = LC >> 1; x > 0; x >>= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
+      if (col && lr == 0) p.o[(size_t)(m0 + r) * HV + hd * V + j] = o;
     }
     __syncthreads();  // every thread is done with this buffer before the chunk after next is copied into it
   }
   if (col) {
-    if (DR > 0) {
 #pragma unroll
-      for (int d = 0; d < DR; ++d)
-        if (d0 + d < D) Sg[(size_t)(d0 + d) * V] = Sr[d];
-    } else {
-      for (int d = 0; d < D; ++d) Sg[(size_t)d * V] = Ssm[(size_t)d * Vr + jl];
+    for (int i = 0; i < NQ; ++i) {
+      const int d = 4 * (lr + LC * i);
+      if (p.vec) {
+        if (d < D) *reinterpret_cast<float4*>(Sg + d) = S[i];
+      } else {
+        if (d < D) Sg[d] = S[i].x;
+        if (d + 1 < D) Sg[d + 1] = S[i].y;
+        if (d + 2 < D) Sg[d + 2] = S[i].z;
+        if (d + 3 < D) Sg[d + 3] = S[i].w;
+      }
     }
+  }
+}
+
+// Any D: one thread per column, the column in shared memory ([D][blockDim], dynamic), operands read from global memory.
+// grid (n_seqs, H, ceil(V / blockDim))
+template <bool CH>
+__global__ void delta_scan_any_kernel(const DeltaArgs p, const Ragged rg) {
+  extern __shared__ __align__(16) float ds_sm[];
+  const int s = blockIdx.x, hd = blockIdx.y, g = hd / (p.H / p.G), jl = threadIdx.x, Vr = blockDim.x, j = blockIdx.z * Vr + jl;
+  const int D = p.D, V = p.V;
+  if (j >= V) return;
+  float* Sg = p.S + (size_t)rg.slot[s] * p.slot_stride + ((size_t)hd * V + j) * D;
+  const bool carried = rg.pos0[s] > 0;
+  for (int d = 0; d < D; ++d) ds_sm[(size_t)d * Vr + jl] = carried ? Sg[d] : 0.f;
+  for (int m = rg.cu[s]; m < rg.cu[s + 1]; ++m) {
+    const float* k = p.k + (size_t)m * p.G * D + g * D;
+    const float* q = p.q + (size_t)m * p.G * D + g * D;
+    const float* gc = p.decay + (CH ? ((size_t)m * p.H + hd) * D : (size_t)m * p.H + hd);
+    float dot = 0.f, o = 0.f;
+    for (int d = 0; d < D; ++d) {
+      const float so = ds_sm[(size_t)d * Vr + jl], sv = fmaf(so, gc[CH ? d : 0], so);
+      ds_sm[(size_t)d * Vr + jl] = sv;
+      dot = fmaf(sv, k[d], dot);
+    }
+    const float u = p.beta[(size_t)m * p.H + hd] * (p.v[((size_t)m * p.H + hd) * V + j] - dot);
+    for (int d = 0; d < D; ++d) {
+      const float sv = fmaf(k[d], u, ds_sm[(size_t)d * Vr + jl]);
+      ds_sm[(size_t)d * Vr + jl] = sv;
+      o = fmaf(sv, q[d], o);
+    }
+    p.o[((size_t)m * p.H + hd) * V + j] = o;
+  }
+  for (int d = 0; d < D; ++d) Sg[d] = ds_sm[(size_t)d * Vr + jl];
+}
+
+// fp32 columns [c0, c0 + n1) and [c0 + n1, c0 + n1 + n2) of each row -> two dense T matrices (operands of two linear layers)
+template <typename T>
+__global__ void cast_split_kernel(const float* __restrict__ src, int ld_src, T* __restrict__ d1, int n1, T* __restrict__ d2, int n2) {
+  const float* r = src + (size_t)blockIdx.x * ld_src;
+  for (int c = threadIdx.x; c < n1 + n2; c += blockDim.x) {
+    if (c < n1) st_f<T>(d1 + (size_t)blockIdx.x * n1 + c, r[c]);
+    else st_f<T>(d2 + (size_t)blockIdx.x * n2 + (c - n1), r[c]);
   }
 }
 

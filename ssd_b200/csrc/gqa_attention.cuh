@@ -2,17 +2,21 @@
 // models.  H query heads share G key/value heads (query head h reads head h / (H / G)); key size D and value size V are
 // independent.  A page row holds, for one token, the keys of all G heads (rotated, optionally unit-RMS) and then their
 // values: [G D | G V] of storage type T.  The softmax denominator may carry a constant (`sink`: 1 = a sink of score 0
-// that has no value) or a learned logit per query head; a sliding window limits a query to its last `window` positions.
+// that has no value) or a learned logit per query head; a key mask limits a query to its last `window` positions or to its own
+// chunk of positions.
 //
 //   gqa_prep_kernel      per (token, head): rotation of the first rot_dims dimensions in adjacent or half-apart pairs (angle = position *
 //                        frequency in fp32, cos and sin times a constant), optional unit RMS over D; queries go to a
 //                        group-major buffer [G, M, H/G, D] (T), keys and raw values into the token's page row
+//   gqa_conv_prep_kernel the same behind a short convolution over time of q | k | v (bias, taps, history in the state slot) and an
+//                        optional weighted RMS norm over the whole query and key projection, one CTA per row
 //   kv_gather_kernel     one sequence's pages -> contiguous keys [G, ctx_pad, D] and transposed values [G, V, ctx_pad]
 //   portions (>= 2 rows) two batched GEMMs per query block around sink_softmax_kernel (HybRun::gqa_attention)
 //   single-token rows    gqa_decode_partial_kernel (all decoding sequences in one launch, context split flash-decoding
 //                        style, fp32 weights) + gqa_decode_merge_kernel
 //   attn_gate_kernel     group-major fp32 output x sigmoid(gate pre-activation) -> [M, H V] (T) for the output projection
 #pragma once
+#include "conv_scan.cuh"  // ConvArgs, conv_at
 #include "latent_attention.cuh"
 
 namespace ssdk {
@@ -76,6 +80,67 @@ __global__ void gqa_prep_kernel(const GqaPrepArgs p, const Ragged rg) {
   }
 }
 
+struct GqaConvPrepArgs {
+  GqaPrepArgs g;               // z / ldz unused: the rows come through the convolution; qk_norm 0 or 2
+  ConvArgs conv;               // over the q | k | v columns (C = H D + G D + G V); out / out_t unused, w may be nullptr (one tap of 1)
+  const void* norm_w;          // [H D + G D] T weights of the two projection norms (qk_norm == 2)
+};
+
+inline size_t gqa_conv_prep_smem(int C, int rot_dims) { return ((size_t)C + rot_dims + 4) * 4; }
+
+// grid (M): a CTA convolves the row's q | k | v channels into shared memory, norms the whole query and the whole key
+// projection there, turns the first rot_dims entries of every head and stores queries (group-major) and the token's page row.
+template <typename T>
+__global__ void gqa_conv_prep_kernel(const GqaConvPrepArgs p, const Ragged rg) {
+  extern __shared__ float gc_sm[];
+  __shared__ float red[33];
+  const int m = blockIdx.x, s = rg.tok_seq[m], t = m - rg.cu[s], pos = rg.pos0[s] + t;
+  const int H = p.g.H, G = p.g.G, D = p.g.D, V = p.g.V, HD = H * D, QK = (H + G) * D, C = QK + G * V;
+  const int rd = p.g.inv_freq ? p.g.rot_dims : 0, half = rd >> 1;
+  float* y = gc_sm;            // [C]
+  float* cs = y + C;           // [half] cos, [half] sin
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, c;
+    sincosf((float)pos * p.g.inv_freq[i], &sn, &c);
+    cs[i] = c * p.g.rot_mult; cs[half + i] = sn * p.g.rot_mult;
+  }
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x; c < C; c += blockDim.x) {
+    const float v = conv_at<T>(p.conv, rg, m, s, t, c);
+    y[c] = v;
+    if (c < HD) sq = fmaf(v, v, sq);
+    else if (c < QK) sk = fmaf(v, v, sk);
+  }
+  if (p.g.qk_norm == 2) {
+    sq = block_sum(sq, red);
+    sk = block_sum(sk, red);
+    const float iq = 1.0f / sqrtf(sq / (float)HD + p.g.eps), ik = 1.0f / sqrtf(sk / (float)(G * D) + p.g.eps);
+    for (int c = threadIdx.x; c < QK; c += blockDim.x) y[c] *= (c < HD ? iq : ik) * ld_f<T>((const T*)p.norm_w + c);
+  }
+  __syncthreads();
+  T* row = (T*)p.g.cache + page_row(rg, s, pos) * (size_t)(G * (D + V));
+  const int hpg = H / G;
+  for (int c = threadIdx.x; c < C; c += blockDim.x) {
+    float v = y[c];
+    if (c < QK) {
+      const int hd = c / D, d = c - hd * D;
+      if (d < rd) {
+        const int i = p.g.rot_half ? (d < half ? d : d - half) : d >> 1;
+        const bool first = p.g.rot_half ? d < half : (d & 1) == 0;
+        const int step = p.g.rot_half ? half : 1;
+        const float o = y[first ? c + step : c - step];   // the other entry of the pair
+        v = first ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
+      }
+      if (c < HD) {
+        const int g = hd / hpg;
+        st_f<T>((T*)p.g.q + (((size_t)g * rg.M + m) * hpg + (hd - g * hpg)) * D + d, v);
+        continue;
+      }
+    }
+    st_f<T>(row + (c - HD), v);   // keys of all heads, then values: the page row's own order
+  }
+}
+
 // grid (ctx_pad): position lo + j of sequence s -> keys[g][j][:] and vt[g][:][j]; zero from ctx up to ctx_pad
 template <typename T>
 __global__ void kv_gather_kernel(const T* __restrict__ cache, T* __restrict__ keys, T* __restrict__ vt, const Ragged rg, int s,
@@ -97,7 +162,7 @@ struct GqaDecodeArgs {
   int H, G, D, V, splits;
   float scale, sink;
   const void* sinks;  // [H] T learned sink logits (they replace the constant), or nullptr
-  int window;         // as LatentDecodeArgs::window
+  KeyMask mask;       // first key the token sees
 };
 
 constexpr int kGqaDecWarps = 4;
@@ -123,7 +188,7 @@ __global__ void __launch_bounds__(kGqaDecWarps * 32) gqa_decode_partial_kernel(c
   for (int d = tid; d < Dp; d += blockDim.x) qs[d] = d < D ? ld_f<T>(q + d) * p.scale : 0.f;
   __syncthreads();
   int k_lo, k_hi;
-  decode_split(rg.pos0[s] + 1, p.window, sp, p.splits, &k_lo, &k_hi);
+  decode_split(rg.pos0[s] + 1, p.mask, sp, p.splits, &k_lo, &k_hi);
   const size_t roww = (size_t)G * (D + V);
   constexpr int kPer = 16 / (int)sizeof(T);
   const bool pool16 = ((uintptr_t)p.cache & 15) == 0;

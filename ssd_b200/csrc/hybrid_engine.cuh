@@ -20,6 +20,7 @@ struct HybLayer {
   HybTensor t[SSDK_HT_COUNT];
   size_t state_off = 0;      // floats from the start of a slot
   size_t canon_off = 0;      // one-norm blocks: the input convolutions' history [canon_taps - 1, width], floats from the start of a slot
+  size_t attn_hist_off = 0;  // attention pair: history of the attention's convolution, floats from the start of a slot
   size_t cache_row = 0;      // row width (elements) of this layer's latent pool
   size_t cache_rows_before = 0;  // sum of the row widths of the latent layers before this one
   float* inv_freq = nullptr; // device, [rot_dims / 2]
@@ -79,15 +80,19 @@ struct ssdk_hyb_engine {
   bool smem_attr_done = false;
 };
 
-// delta rule: rows of a state column per thread (DR) and row groups (NG); DR = 0: the shared-memory walk
-static void delta_shape(int D, int Vr, int* DR, int* NG) {
-  *DR = 0; *NG = 1;
-  if (D <= 16) { *DR = 16; return; }
-  for (int dr : {32, 64}) {  // (16 rows per thread in eight row groups measured 5 % slower: the barriers outweigh the extra warps)
-    const int g = (D + dr - 1) / dr;
-    if (Vr * g <= 512 && g <= 8) { *DR = dr; *NG = g; return; }  // 512 threads: the register file holds DR + ~40 each
-  }
+// delta rule: lanes per state column (LC) and 16-byte pieces per lane (NQ) of delta_scan_kernel, 4 LC NQ >= D; few columns in
+// flight spread each over more lanes.  LC = 0: no register form, the column lives in shared memory (delta_scan_any_kernel)
+static void delta_shape(int D, bool few, int* LC, int* NQ) {
+  auto set = [&](int lc, int nq) { *LC = lc; *NQ = nq; };
+  if (D <= 16) set(4, 1);
+  else if (D <= 32) set(4, 2);
+  else if (D <= 64) few ? set(8, 2) : set(4, 4);
+  else if (D <= 128) few ? set(8, 4) : set(4, 8);
+  else if (D <= 256) set(8, 8);
+  else if (D <= 512) set(16, 8);
+  else set(0, 0);
 }
+constexpr int kDeltaAnyCols = 32;  // columns per CTA of the shared-memory form
 
 static int hyb_derive(ssdk_hyb_engine* e) {
   const ssdk_hyb_cfg& g = e->cfg;
@@ -98,7 +103,9 @@ static int hyb_derive(ssdk_hyb_engine* e) {
     const ssdk_hyb_layer_cfg& c = L.c;
     const int H = c.heads, D = c.dim, V = c.vdim;
     if (H < 1 || D < 1) return fail("hybrid layer: heads / dim must be positive");
-    if (c.window < 0) return fail("hybrid layer: window %d", c.window);
+    if (c.window < 0 || c.chunk < 0) return fail("hybrid layer: window %d, chunk %d", c.window, c.chunk);
+    if (g.block == SSDK_BLOCK_SERIAL_PRENORM && (c.mixer == SSDK_MIX_WKV || c.mixer == SSDK_MIX_MLSTM))
+      return fail("wkv and mlstm are built for parallel blocks");
     if (g.block == SSDK_BLOCK_PARALLEL_ONE_NORM) {
       if (c.mixer != SSDK_MIX_ATTENTION && c.mixer != SSDK_MIX_LATENT_ATTN && c.mixer != SSDK_MIX_RGLRU && c.mixer != SSDK_MIX_SELECTIVE)
         return fail("one-norm blocks are built for the attention, latent-attention, rglru and selective-scan mixers");
@@ -161,20 +168,26 @@ static int hyb_derive(ssdk_hyb_engine* e) {
       if (V > 256 * 4) return fail("attention: value size %d too large", V);
       if (Hd < 1 || Gd < 1 || Hd % Gd || Dd < 1 || Vd < 1 || Vd > 1024 || c.conv < 1)
         return fail("delta rule: %d heads on %d query/key heads, %d x %d, %d taps", Hd, Gd, Dd, Vd, c.conv);
-      {
-        const int Vr = (Vd + 31) / 32 * 32;
-        int dr = 0, ng = 1;
-        delta_shape(Dd, Vr, &dr, &ng);
-        if (dr == 0 && ssdk::delta_scan_smem(Dd, Vr, 0, 1) > 200 * 1024) return fail("delta rule: head %d x %d too large", Dd, Vd);
-      }
-      const long long Cd = 2LL * Gd * Dd + (long long)Hd * Vd;
+      if ((size_t)Dd * kDeltaAnyCols * 4 > 200 * 1024) return fail("delta rule: key size %d too large", Dd);
+      if (c.qk_norm < 0 || c.qk_norm > 2 || c.pair_conv < 0 || c.d_decay_rank < 0 || c.d_gate_rank < 0 || (c.d_gate_act & ~1))
+        return fail("attention pair: bad variant");
+      if (c.qk_norm == 1 && c.pair_conv > 0) return fail("attention pair: the per-head unit norm is built for projections without a convolution");
+      if (c.pair_norm && g.block != SSDK_BLOCK_SERIAL_PRENORM) return fail("attention pair: norms on the two results are built for serial pre-norm blocks");
+      const long long Cd = 2LL * Gd * Dd + (long long)Hd * Vd, Ca = (long long)H * D + (long long)G * (D + V);
+      if (ssdk::gqa_conv_prep_smem((int)Ca, c.rot_dims) > 200 * 1024) return fail("attention pair: %lld projected channels too many", Ca);
+      soff = align_up(soff, 4);                      // the state's columns start on 16-byte boundaries (if their length allows)
+      L.state_off = soff;
       soff += (size_t)Hd * Dd * Vd + (size_t)(c.conv - 1) * Cd;
+      L.attn_hist_off = soff;
+      if (c.pair_conv > 1) soff += (size_t)(c.pair_conv - 1) * Ca;
       L.cache_row = (size_t)G * (D + V);
       L.cache_rows_before = crow;
       crow += L.cache_row;
-      up(e->w_p0, (long long)H * D + (long long)G * D + (long long)G * V + (long long)H * V + Cd + (long long)Hd * Vd + 2 * Hd);
-      up(e->w_p1, std::max((long long)H * V, (long long)Hd * Vd)); up(e->w_p2, Cd + 2 * Hd);
-      up(e->w_t0, (long long)H * V); up(e->w_t1, (long long)Hd * Vd);
+      up(e->w_p0, Ca + (c.pair_gate ? (long long)H * V : 0) + Cd + (c.d_gate_rank ? c.d_gate_rank : (long long)Hd * Vd) + Hd +
+                      (c.d_decay_rank ? c.d_decay_rank : Hd));
+      up(e->w_p1, std::max((long long)H * V, (long long)Hd * Vd));
+      up(e->w_p2, Cd + Hd + (c.d_decay_rank ? (long long)Hd * Dd : Hd) + (c.d_gate_rank ? (long long)Hd * Vd : 0));
+      up(e->w_t0, (long long)H * V); up(e->w_t1, std::max((long long)Hd * Vd, (long long)c.d_decay_rank + c.d_gate_rank));
       up(e->w_qcat, (long long)H * D); up(e->w_key, (long long)G * D); up(e->w_kr, (long long)G * V); up(e->w_lh, H);
       e->any_pair = true;
     } else if (c.mixer == SSDK_MIX_ATTENTION) {
@@ -183,30 +196,33 @@ static int hyb_derive(ssdk_hyb_engine* e) {
       if (c.rot_dims < 0 || c.rot_dims > D || (c.rot_dims & 1)) return fail("attention: rot dims %d of %d", c.rot_dims, D);
       if (V > 256 * 4) return fail("attention: value size %d too large", V);
       if (c.conv < 1) return fail("attention: %d taps", c.conv);
+      if (c.qk_norm) return fail("attention: query and key norms are built for the pair");
+      if (ssdk::gqa_conv_prep_smem(H * D + G * (D + V), c.rot_dims) > 200 * 1024) return fail("attention: too many projected channels");
       const long long Nqkv = (long long)H * D + (long long)G * D + (long long)G * V;
       soff += (size_t)(c.conv - 1) * Nqkv;
       L.cache_row = (size_t)G * (D + V);
       L.cache_rows_before = crow;
       crow += L.cache_row;
-      up(e->w_p0, Nqkv); up(e->w_p1, Nqkv); up(e->w_p2, (long long)H * V); up(e->w_t0, (long long)H * V);
+      up(e->w_p0, Nqkv); up(e->w_p2, (long long)H * V); up(e->w_t0, (long long)H * V);
       up(e->w_qcat, (long long)H * D); up(e->w_key, (long long)G * D); up(e->w_kr, (long long)G * V); up(e->w_lh, H);
     } else {
       return fail("hybrid layer: unknown mixer %d", c.mixer);
     }
     if (c.mlp == SSDK_MLP_GLU) {
       if (c.ff < 1) return fail("dense feed-forward: ff %d", c.ff);
-      if (e->cfg.block != SSDK_BLOCK_SERIAL_POSTNORM) return fail("the dense feed-forward is built for serial blocks");
+      if (e->cfg.block != SSDK_BLOCK_SERIAL_POSTNORM && e->cfg.block != SSDK_BLOCK_SERIAL_PRENORM) return fail("the gated dense feed-forward is built for serial blocks");
+      if (c.ff_act != SSDK_ACT_SILU && c.ff_act != SSDK_ACT_GELU_TANH) return fail("dense feed-forward: unknown gate activation %d", c.ff_act);
       up(e->w_p0, 2LL * c.ff); up(e->w_t0, c.ff);
     } else if (c.mlp == SSDK_MLP_FFN) {
       if (c.ff < 1) return fail("dense feed-forward: ff %d", c.ff);
-      if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM) return fail("the ungated feed-forward is built for parallel blocks");
+      if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM || e->cfg.block == SSDK_BLOCK_SERIAL_PRENORM) return fail("the ungated feed-forward is built for parallel blocks");
       if (c.ff_act != SSDK_ACT_RELU2 && c.ff_act != SSDK_ACT_GELU_TANH && c.ff_act != SSDK_ACT_SILU && c.ff_act != SSDK_ACT_POLYNORM)
         return fail("dense feed-forward: unknown activation %d", c.ff_act);
       up(e->w_sff2, c.ff); up(e->w_sff, c.ff);   // it shares the shared expert's buffers: no layer has both
       e->any_ffn = true;
     } else if (c.mlp == SSDK_MLP_MOE) {
       const int Et = c.experts + c.identity;   // router outputs: real experts, then identity experts
-      if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM) return fail("the mixture of experts is built for parallel blocks");
+      if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM || e->cfg.block == SSDK_BLOCK_SERIAL_PRENORM) return fail("the mixture of experts is built for parallel blocks");
       if (c.experts < 1 || c.identity < 0 || Et > kRouterMaxE) return fail("moe: 1 <= experts (+ identity) <= %d", kRouterMaxE);
       if (c.groups < 1 || Et % c.groups) return fail("moe: %d router outputs do not form %d equal groups", Et, c.groups);
       if (c.keep < 1 || c.keep > c.groups) return fail("moe: keep %d of %d groups", c.keep, c.groups);
@@ -224,7 +240,7 @@ static int hyb_derive(ssdk_hyb_engine* e) {
       return fail("hybrid layer: unknown feed-forward kind %d", c.mlp);
     }
   }
-  e->slot_floats = soff;
+  e->slot_floats = e->any_pair ? align_up(soff, 4) : soff;
   e->cache_row_total = crow;
   return 0;
 }
@@ -235,7 +251,7 @@ static int64_t hyb_carve(ssdk_hyb_engine* e, uint8_t* base) {
   const size_t cap = g.max_tokens, A = cap * (size_t)std::max(1, e->w_top), es = e->esz;
   size_t off = 0;
   auto take = [&](size_t bytes) { uint8_t* p = base ? base + off : nullptr; off = align_up(off + bytes, 256); return p; };
-  e->x = (float*)take(cap * g.width * 4);
+  e->x = (float*)take(cap * g.width * 4 * std::max(1, g.streams));
   e->h = take(cap * g.width * es);
   const bool one_norm = g.block == SSDK_BLOCK_PARALLEL_ONE_NORM;
   e->h2 = take(g.block == SSDK_BLOCK_PARALLEL_TWO_NORMS || (one_norm && g.canon_taps > 0) ? cap * g.width * es : 0);
@@ -482,12 +498,29 @@ struct HybRun {
 
   // query rows per block of a windowed attention's portion path
   static int window_block(int win) { return std::max(128, (win + 63) / 64 * 64); }
+  // rows of the query block that starts at position pos, `left` rows remain: short blocks keep the scores to the rows + the keys
+  // the mask leaves visible; a block ends with its chunk (unless chunks are shorter than a tile of rows)
+  static int mask_block(const ssdk::KeyMask& mask, int pos, int left, int qb) {
+    if (mask.window > 0) qb = std::min(qb, window_block(mask.window));
+    if (mask.chunk >= 128) qb = std::min(qb, mask.chunk - pos % mask.chunk);
+    else if (mask.chunk > 0) qb = std::min(qb, 256);
+    return std::min(qb, left);
+  }
+  // context the single-token sequences of this step see at most, and how many there are
+  int decode_rows(const ssdk::KeyMask& mask, int* ctx_max) const {
+    int n = 0;
+    *ctx_max = 0;
+    for (int s = 0; s < rg.n_seqs; ++s)
+      if (h_cu[s + 1] - h_cu[s] == 1) { ++n; *ctx_max = std::max(*ctx_max, h_pos0[s] + 1 - mask.first(h_pos0[s])); }
+    return n;
+  }
 
   int latent(HybLayer& Lr) {
     const ssdk_hyb_layer_cfg& c = Lr.c;
     const int H = c.heads, D = c.dim, V = c.vdim, R = c.rot_dim, KR = c.kv_rank, QR = c.q_rank, W = e->cfg.width;
     const bool own = c.kv_from < 0;   // the layer fills a pool of its own (else it reads an earlier layer's rows of this step and before)
-    const int Nq = H * (D + R), Nkv = own ? KR + R : 0, win = c.window;
+    const int Nq = H * (D + R), Nkv = own ? KR + R : 0;
+    const ssdk::KeyMask mask = {c.window, c.chunk};
     CKI(check_tensor(Lr, SSDK_HT_LAT_UKT, (int64_t)H * KR, D, "uk^T")); CKI(check_tensor(Lr, SSDK_HT_LAT_UV, (int64_t)H * V, KR, "uv"));
     CKI(check_tensor(Lr, SSDK_HT_MIX_OUT, W, (int64_t)H * V, "mix.o"));
     if (own) CKI(check_tensor(Lr, SSDK_HT_LAT_KVNORM, KR, 1, "dkv.norm"));
@@ -532,10 +565,8 @@ struct HybRun {
     // single-token sequences (decode) share ONE fused launch + a merge; the others take the GEMM path below
     bool fused_decode = false;
     {
-      int n_dec = 0, ctx_max = 0;
-      for (int s = 0; s < rg.n_seqs; ++s)
-        if (h_cu[s + 1] - h_cu[s] == 1) { ++n_dec; ctx_max = std::max(ctx_max, h_pos0[s] + 1); }
-      if (win > 0) ctx_max = std::min(ctx_max, win);
+      int ctx_max = 0;
+      const int n_dec = decode_rows(mask, &ctx_max);
       const size_t smem = ssdk::latent_decode_smem(H, KR, Wd, sizeof(T));
       const bool pool_aligned = ((uintptr_t)pool & 15) == 0;
       // bf16 rows that start on 16-byte boundaries go through the tensor cores: k-steps of 16 columns and n-tiles of 8
@@ -550,7 +581,7 @@ struct HybRun {
         if (splits >= 1) {
           ssdk::LatentDecodeArgs da;
           da.qcat = e->qcat; da.cache = pool; da.sink = sink; da.part = e->att_s; da.out = e->t0;
-          da.H = H; da.KR = KR; da.W = Wd; da.splits = splits; da.scale = c.attn_scale; da.pool_aligned = pool_aligned; da.window = win;
+          da.H = H; da.KR = KR; da.W = Wd; da.splits = splits; da.scale = c.attn_scale; da.pool_aligned = pool_aligned; da.mask = mask;
           if (mma) {
             const dim3 grid(rg.n_seqs, splits, (H + 15) / 16), block(ssdk::kDmThreads);
             const size_t sm = ssdk::latent_decode_mma_smem(Wd);
@@ -572,15 +603,15 @@ struct HybRun {
     for (int s = 0; s < rg.n_seqs; ++s) {
       const int r0 = h_cu[s], n = h_cu[s + 1] - r0, p0 = h_pos0[s];
       if (fused_decode && n == 1) continue;
-      // the portion's keys: positions lo .. p0 + n - 1 (a window hides the positions before lo from every row of the portion)
-      const int lo = win > 0 ? std::max(0, p0 - win + 1) : 0, ctx = p0 + n - lo, ctx_pad = (ctx + kpad - 1) / kpad * kpad;
+      // the portion's keys: positions lo .. p0 + n - 1 (the mask hides the positions before lo from every row of the portion)
+      const int lo = mask.first(p0), ctx = p0 + n - lo, ctx_pad = (ctx + kpad - 1) / kpad * kpad;
       CKI(L.go(ssdk::latent_gather_kernel<T>, dim3(ctx_pad), dim3(128), 0, (const T*)pool, (T*)e->keys, (T*)e->lat_t, rg, s, lo, ctx, ctx_pad,
                KR, Wd));
-      int qb = (int)std::max<size_t>(1, e->att_elems / ((size_t)H * ctx_pad));
-      if (win > 0) qb = std::min(qb, window_block(win));   // short query blocks: a block's scores span its rows + the window
-      for (int q0 = 0; q0 < n; q0 += qb) {
+      const int qb = (int)std::max<size_t>(1, e->att_elems / ((size_t)H * ctx_pad));
+      for (int q0 = 0, nq; q0 < n; q0 += nq) {
+        nq = mask_block(mask, p0 + q0, n - q0, qb);
         // gathered keys kb .. kb + cb - 1 are what this block can see (whole pads, so that the operands stay aligned)
-        const int nq = std::min(qb, n - q0), rows = nq * H, kb = win > 0 ? std::max(0, p0 + q0 - win + 1 - lo) / kpad * kpad : 0;
+        const int rows = nq * H, kb = (mask.first(p0 + q0) - lo) / kpad * kpad;
         const int cb = (p0 + q0 + nq - lo - kb + kpad - 1) / kpad * kpad;
         const T* qrows = (const T*)e->qcat + (size_t)(r0 + q0) * H * Wd;
         const T* krows = (const T*)e->keys + (size_t)kb * Wd;
@@ -588,7 +619,7 @@ struct HybRun {
         // scores: keys are the 128-row operand, (query, head) rows the tokens
         CKI(lin(qrows, Wd, krows, Wd, e->att_s, cb, rows, cb, Wd, false, 1, 0, 0, 0, tc_attn));
         CKI(L.go(ssdk::sink_softmax_kernel<T>, dim3(rows), dim3(256), 0, (const float*)e->att_s, (T*)e->att_p,
-                 (const T*)sink, H, cb, p0 + q0, c.attn_scale, rows, 0.f, lo + kb, win));
+                 (const T*)sink, H, cb, p0 + q0, c.attn_scale, rows, 0.f, lo + kb, mask));
         T* o_rows = (T*)e->t0 + (size_t)(r0 + q0) * H * KR;
         if (tc_attn && tc_ok(e->att_p, cb, lat_t, ctx_pad, KR, KR, cb)) {
           // P C: the transposed latents [kv_rank, ctx_pad] are the 128-row operand, read with the row stride of the gather
@@ -705,7 +736,10 @@ struct HybRun {
     const int W = e->cfg.width, ff = Lr.c.ff;
     CKI(check_tensor(Lr, SSDK_HT_GLU_IN, 2 * ff, W, "mlp.gate|up")); CKI(check_tensor(Lr, SSDK_HT_GLU_OUT, W, ff, "mlp.down"));
     CKI(lin(hin, W, Lr.t[SSDK_HT_GLU_IN].p, W, e->p0, 2 * ff, M, 2 * ff, W));
-    CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_GELU_TANH>, dim3(M), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
+    if (Lr.c.ff_act == SSDK_ACT_SILU)
+      CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_SILU>, dim3(M), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
+    else
+      CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_GELU_TANH>, dim3(M), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
     return lin(e->t0, ff, Lr.t[SSDK_HT_GLU_OUT].p, ff, e->mix_out, W, M, W, ff);
   }
 
@@ -787,10 +821,14 @@ struct HybRun {
     return lin(e->t1, I, Lr.t[SSDK_HT_MIX_OUT].p, I, e->mix_out, W, M, W, I);
   }
 
-  // grouped-query sink attention over the layer's page pool: z holds q | k | v (fp32); og [G, M, H/G, V] fp32
-  int gqa_attention(HybLayer& Lr, const float* z, int ldz, float* og, const void* sinks = nullptr) {
+  // grouped-query attention over the layer's page pool: z holds q | k | v (fp32); og [G, M, H/G, V] fp32.  conv (optional): z's
+  // columns pass through a bias and a short convolution over time first, norm_w: then through a norm over the whole query
+  // and key projection
+  int gqa_attention(HybLayer& Lr, const float* z, int ldz, float* og, const void* sinks = nullptr, const ssdk::ConvArgs* conv = nullptr,
+                    const void* norm_w = nullptr) {
     const ssdk_hyb_layer_cfg& c = Lr.c;
-    const int H = c.heads, G = c.kv_heads, D = c.dim, V = c.vdim, hpg = H / G, win = c.window;
+    const int H = c.heads, G = c.kv_heads, D = c.dim, V = c.vdim, hpg = H / G;
+    const ssdk::KeyMask mask = {c.window, c.chunk};
     const float sink_const = sinks ? 0.f : c.sink;
     if (!e->cache) return fail("hybrid: attention cache not bound");
     uint8_t* pool = e->cache + (size_t)e->num_blocks * e->cfg.block_size * Lr.cache_rows_before * e->esz;
@@ -798,13 +836,19 @@ struct HybRun {
     pa.z = z; pa.ldz = ldz; pa.q = e->qcat; pa.cache = pool; pa.inv_freq = c.rot_dims >= 2 ? Lr.inv_freq : nullptr;
     pa.H = H; pa.G = G; pa.D = D; pa.V = V; pa.rot_dims = c.rot_dims; pa.qk_norm = c.qk_norm; pa.rot_mult = Lr.rot_mult; pa.eps = e->cfg.eps;
     pa.rot_half = c.rot_half;
-    CKI(L.go(ssdk::gqa_prep_kernel<T>, dim3(M, H + G), dim3(32), 0, pa, rg));
+    if (conv) {
+      ssdk::GqaConvPrepArgs cp;
+      cp.g = pa; cp.conv = *conv; cp.norm_w = norm_w;
+      // a CTA per row: few rows take more threads each
+      CKI(L.go(ssdk::gqa_conv_prep_kernel<T>, dim3(M), dim3(M < num_sms() ? 1024 : 256), ssdk::gqa_conv_prep_smem(conv->C, c.rot_dims), cp, rg));
+      if (conv->taps > 1) CKI(L.go(ssdk::conv_state_kernel<T>, dim3(rg.n_seqs, (conv->C + 255) / 256), dim3(256), 0, *conv, rg));
+    } else {
+      CKI(L.go(ssdk::gqa_prep_kernel<T>, dim3(M, H + G), dim3(32), 0, pa, rg));
+    }
     bool fused_decode = false;
     {
-      int n_dec = 0, ctx_max = 0;
-      for (int s = 0; s < rg.n_seqs; ++s)
-        if (h_cu[s + 1] - h_cu[s] == 1) { ++n_dec; ctx_max = std::max(ctx_max, h_pos0[s] + 1); }
-      if (win > 0) ctx_max = std::min(ctx_max, win);
+      int ctx_max = 0;
+      const int n_dec = decode_rows(mask, &ctx_max);
       const int vpl = (V + 31) / 32;
       if (n_dec > 0 && vpl <= 8 && e->use_decode_attn) {
         int splits = std::max(1, std::min({32, 8 * num_sms() / std::max(1, n_dec * H), (ctx_max + 127) / 128}));  // ~8 four-warp CTAs per SM
@@ -813,7 +857,7 @@ struct HybRun {
         if (splits >= 1) {
           ssdk::GqaDecodeArgs da;
           da.q = e->qcat; da.cache = pool; da.part = e->att_s; da.out = og; da.H = H; da.G = G; da.D = D; da.V = V; da.splits = splits;
-          da.scale = c.attn_scale; da.sink = sink_const; da.sinks = sinks; da.window = win;
+          da.scale = c.attn_scale; da.sink = sink_const; da.sinks = sinks; da.mask = mask;
           const dim3 grid(rg.n_seqs, H, splits), block(ssdk::kGqaDecWarps * 32);
           const size_t smem = ssdk::gqa_decode_smem(D, V);
           if (vpl <= 1) CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 1>, grid, block, smem, da, rg));
@@ -828,18 +872,18 @@ struct HybRun {
     for (int s = 0; s < rg.n_seqs; ++s) {
       const int r0 = h_cu[s], n = h_cu[s + 1] - r0, p0 = h_pos0[s];
       if (fused_decode && n == 1) continue;
-      const int lo = win > 0 ? std::max(0, p0 - win + 1) : 0, ctx = p0 + n - lo, ctx_pad = (ctx + 7) / 8 * 8;   // keys lo .. p0 + n - 1
+      const int lo = mask.first(p0), ctx = p0 + n - lo, ctx_pad = (ctx + 7) / 8 * 8;   // keys lo .. p0 + n - 1
       CKI(L.go(ssdk::kv_gather_kernel<T>, dim3(ctx_pad), dim3(128), 0, (const T*)pool, (T*)e->keys, (T*)e->lat_t, rg, s, lo, ctx, ctx_pad, G, D, V));
-      int qb = (int)std::max<size_t>(1, e->att_elems / ((size_t)H * ctx_pad));
-      if (win > 0) qb = std::min(qb, window_block(win));
-      for (int q0 = 0; q0 < n; q0 += qb) {
-        const int nq = std::min(qb, n - q0), rows = nq * hpg, kb = win > 0 ? std::max(0, p0 + q0 - win + 1 - lo) / 8 * 8 : 0;
+      const int qb = (int)std::max<size_t>(1, e->att_elems / ((size_t)H * ctx_pad));
+      for (int q0 = 0, nq; q0 < n; q0 += nq) {
+        nq = mask_block(mask, p0 + q0, n - q0, qb);
+        const int rows = nq * hpg, kb = (mask.first(p0 + q0) - lo) / 8 * 8;
         const int cb = (p0 + q0 + nq - lo - kb + 7) / 8 * 8;   // gathered keys kb .. kb + cb - 1 are what this block can see
         const T* qrows = (const T*)e->qcat + (size_t)(r0 + q0) * hpg * D;
         CKI(lin(qrows, D, (const T*)e->keys + (size_t)kb * D, D, e->att_s, cb, rows, cb, D, false, G, (long long)M * hpg * D, (long long)ctx_pad * D,
                 (long long)rows * cb, false));
         CKI(L.go(ssdk::sink_softmax_kernel<T>, dim3(G * rows), dim3(256), 0, (const float*)e->att_s, (T*)e->att_p, (const T*)sinks, hpg, cb,
-                 p0 + q0, c.attn_scale, rows, sink_const, lo + kb, win));
+                 p0 + q0, c.attn_scale, rows, sink_const, lo + kb, mask));
         CKI(lin(e->att_p, cb, (const T*)e->lat_t + kb, ctx_pad, og + (size_t)(r0 + q0) * hpg * V, V, rows, V, cb, false, G, (long long)rows * cb,
                 (long long)V * ctx_pad, (long long)M * hpg * V, false));
       }
@@ -858,61 +902,110 @@ struct HybRun {
     if (c.learned_sink) CKI(check_tensor(Lr, SSDK_HT_ATTN_SINK, H, 1, "sink"));
     CKI(lin(hin, W, Lr.t[SSDK_HT_ATTN_IN].p, W, e->p0, Nqkv, M, Nqkv, W));
     ssdk::ConvArgs ca = {};
-    ca.in = e->p0; ca.ld_in = Nqkv; ca.in_bias = Lr.t[SSDK_HT_ATTN_IN_B].p; ca.w = Lr.t[SSDK_HT_CONV_W].p; ca.out = e->p1; ca.ld_out = Nqkv;
+    ca.in = e->p0; ca.ld_in = Nqkv; ca.in_bias = Lr.t[SSDK_HT_ATTN_IN_B].p; ca.w = Lr.t[SSDK_HT_CONV_W].p;
     ca.hist = e->state + Lr.state_off; ca.slot_stride = e->slot_floats; ca.C = Nqkv; ca.taps = taps;
-    CKI(L.go(ssdk::short_conv_kernel<T, 0>, dim3(M, (Nqkv + 255) / 256), dim3(256), 0, ca, rg));
-    if (taps > 1) CKI(L.go(ssdk::conv_state_kernel<T>, dim3(rg.n_seqs, (Nqkv + 255) / 256), dim3(256), 0, ca, rg));
-    CKI(gqa_attention(Lr, e->p1, Nqkv, e->p2, c.learned_sink ? Lr.t[SSDK_HT_ATTN_SINK].p : nullptr));
+    CKI(gqa_attention(Lr, e->p0, Nqkv, e->p2, c.learned_sink ? Lr.t[SSDK_HT_ATTN_SINK].p : nullptr, &ca));
     CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(M), dim3(256), 0, (const float*)e->p2, (const float*)nullptr, 0, (T*)e->t0, M, H, G, V));
     return lin(e->t0, H * V, Lr.t[SSDK_HT_MIX_OUT].p, H * V, e->mix_out, W, M, W, H * V);
   }
 
+  // attention beside a gated delta rule on the same input: ONE stacked input projection; results in mix_out and mix2
   int attn_delta(HybLayer& Lr) {
     const ssdk_hyb_layer_cfg& c = Lr.c;
     const int W = e->cfg.width, H = c.heads, G = c.kv_heads, D = c.dim, V = c.vdim, taps = c.conv;
-    const int Hd = c.d_heads, Gd = c.d_kv_heads, Dd = c.d_dim, Vd = c.d_vdim;
-    const int HV = H * V, dGD = Gd * Dd, dHV = Hd * Vd, Cd = 2 * dGD + dHV;
-    const int o_g = H * D + G * D + G * V, o_dq = o_g + HV, o_dg = o_dq + Cd, o_b = o_dg + dHV, Ntot = o_b + 2 * Hd;
+    const int Hd = c.d_heads, Gd = c.d_kv_heads, Dd = c.d_dim, Vd = c.d_vdim, Ra = c.d_decay_rank, Rg = c.d_gate_rank;
+    const int HV = H * V, dGD = Gd * Dd, dHV = Hd * Vd, Cd = 2 * dGD + dHV, Ca = H * D + G * D + G * V;
+    // columns of the projection: q | k | v (| gate) | delta q | k | v (| gate) | beta | decay or its bottleneck (| gate's bottleneck)
+    const int o_g = Ca, o_dq = o_g + (c.pair_gate ? HV : 0), o_dg = o_dq + Cd, o_b = o_dg + (Rg ? 0 : dHV), o_a = o_b + Hd,
+              o_g1 = o_a + (Ra ? Ra : Hd), Ntot = o_g1 + Rg;
     CKI(check_tensor(Lr, SSDK_HT_PAIR_IN, Ntot, W, "pair.in")); CKI(check_tensor(Lr, SSDK_HT_ATTN_OUT, W, HV, "left.o"));
     CKI(check_tensor(Lr, SSDK_HT_MIX_OUT, W, dHV, "right.o")); CKI(check_tensor(Lr, SSDK_HT_CONV_W, Cd, taps, "right.conv"));
-    CKI(check_tensor(Lr, SSDK_HT_DELTA_ALOG, Hd, 1, "right.A_log")); CKI(check_tensor(Lr, SSDK_HT_DELTA_DT_B, Hd, 1, "right.dt_bias"));
+    CKI(check_tensor(Lr, SSDK_HT_DELTA_ALOG, Hd, 1, "right.A_log")); CKI(check_tensor(Lr, SSDK_HT_DELTA_DT_B, Ra ? Hd * Dd : Hd, 1, "right.dt_bias"));
     CKI(check_tensor(Lr, SSDK_HT_MIX_NORM, dHV, 1, "right.norm"));
+    if (Lr.t[SSDK_HT_ATTN_IN_B].p) CKI(check_tensor(Lr, SSDK_HT_ATTN_IN_B, Ca, 1, "left.b"));
+    if (c.pair_conv) CKI(check_tensor(Lr, SSDK_HT_ATTN_CONV_W, Ca, c.pair_conv, "left.conv"));
+    if (c.qk_norm == 2) CKI(check_tensor(Lr, SSDK_HT_ATTN_QK_NORM, (int64_t)(H + G) * D, 1, "left.q.norm|k.norm"));
+    if (Ra) CKI(check_tensor(Lr, SSDK_HT_DELTA_A2, (int64_t)Hd * Dd, Ra, "right.a2"));
+    if (Rg) CKI(check_tensor(Lr, SSDK_HT_DELTA_G2, dHV, Rg, "right.g2"));
     CKI(lin(hin, W, Lr.t[SSDK_HT_PAIR_IN].p, W, e->p0, Ntot, M, Ntot, W));
     // left: attention
-    CKI(gqa_attention(Lr, e->p0, Ntot, e->p1));
-    CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(M), dim3(256), 0, (const float*)e->p1, (const float*)(e->p0 + o_g), Ntot, (T*)e->t0, M, H, G, V));
+    if (c.pair_conv || c.qk_norm == 2 || Lr.t[SSDK_HT_ATTN_IN_B].p) {
+      if (c.qk_norm == 1) return fail("attention pair: the per-head unit norm is built for projections without a bias");
+      ssdk::ConvArgs ca = {};
+      ca.in = e->p0; ca.ld_in = Ntot; ca.in_bias = Lr.t[SSDK_HT_ATTN_IN_B].p; ca.w = c.pair_conv ? Lr.t[SSDK_HT_ATTN_CONV_W].p : nullptr;
+      ca.hist = e->state + Lr.attn_hist_off; ca.slot_stride = e->slot_floats; ca.C = Ca; ca.taps = std::max(1, c.pair_conv);
+      CKI(gqa_attention(Lr, e->p0, Ntot, e->p1, nullptr, &ca, Lr.t[SSDK_HT_ATTN_QK_NORM].p));
+    } else {
+      CKI(gqa_attention(Lr, e->p0, Ntot, e->p1));
+    }
+    CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(M), dim3(256), 0, (const float*)e->p1, (const float*)(c.pair_gate ? e->p0 + o_g : nullptr), Ntot,
+             (T*)e->t0, M, H, G, V));
     CKI(lin(e->t0, HV, Lr.t[SSDK_HT_ATTN_OUT].p, HV, e->mix_out, W, M, W, HV));
     // right: gated delta rule
     float* st = e->state + Lr.state_off;
     ssdk::DeltaPrepArgs dp = {};
     dp.conv.in = e->p0 + o_dq; dp.conv.ld_in = Ntot; dp.conv.w = Lr.t[SSDK_HT_CONV_W].p; dp.conv.hist = st + (size_t)Hd * Dd * Vd;
     dp.conv.slot_stride = e->slot_floats; dp.conv.C = Cd; dp.conv.taps = taps;
-    dp.ba = e->p0 + o_b; dp.ld_ba = Ntot; dp.A_log = Lr.t[SSDK_HT_DELTA_ALOG].p; dp.dt_bias = Lr.t[SSDK_HT_DELTA_DT_B].p;
-    dp.q = e->p2; dp.k = dp.q + (size_t)M * dGD; dp.v = dp.k + (size_t)M * dGD; dp.beta = dp.v + (size_t)M * dHV; dp.decay = dp.beta + (size_t)M * Hd;
+    dp.q = e->p2; dp.k = dp.q + (size_t)M * dGD; dp.v = dp.k + (size_t)M * dGD;
+    float* rest = dp.v + (size_t)M * dHV;          // (per-channel decays first: they stay on 16-byte boundaries)
+    float* dz = rest;
+    if (Ra) rest += (size_t)M * Hd * Dd;
+    float* gz = rest;
+    if (Rg) rest += (size_t)M * dHV;
+    dp.beta = rest; dp.decay = Ra ? dz : rest + (size_t)M * Hd;
+    dp.b = e->p0 + o_b; dp.ld_b = Ntot;
+    if (Ra || Rg) {   // second halves of the low-rank projections
+      const void *za = e->p0 + o_a, *zg = e->p0 + o_g1;
+      int lda = Ntot, ldg = Ntot;
+      if (!kF32) {
+        T* ta = (T*)e->t1;
+        T* tg = ta + (size_t)M * Ra;
+        CKI(L.go(ssdk::cast_split_kernel<T>, dim3(M), dim3(Ra + Rg <= 128 ? 128 : 256), 0, (const float*)e->p0 + (Ra ? o_a : o_g1), Ntot, ta, Ra, tg, Rg));
+        za = ta; zg = tg; lda = Ra; ldg = Rg;
+      }
+      if (Ra) CKI(lin(za, lda, Lr.t[SSDK_HT_DELTA_A2].p, Ra, dz, Hd * Dd, M, Hd * Dd, Ra));
+      if (Rg) CKI(lin(zg, ldg, Lr.t[SSDK_HT_DELTA_G2].p, Rg, gz, dHV, M, dHV, Rg));
+    }
+    dp.a = Ra ? dz : e->p0 + o_a; dp.ld_a = Ra ? Hd * Dd : Ntot; dp.per_channel = Ra > 0;
+    dp.A_log = Lr.t[SSDK_HT_DELTA_ALOG].p; dp.dt_bias = Lr.t[SSDK_HT_DELTA_DT_B].p;
     dp.H = Hd; dp.G = Gd; dp.D = Dd; dp.V = Vd; dp.q_scale = 1.0f / sqrtf((float)Dd); dp.unit_eps = 1e-6f;
-    CKI(L.go(ssdk::delta_prep_kernel<T>, dim3(M, 2 * Gd + Hd), dim3(std::min(256, (std::max(Dd, Vd) + 31) / 32 * 32)),
+    CKI(L.go(ssdk::delta_prep_kernel<T>, dim3(M, 2 * Gd + Hd + (Ra ? Hd : 0)), dim3(std::min(256, (std::max(Dd, Vd) + 31) / 32 * 32)),
              (size_t)std::max(Dd, Vd) * 4, dp, rg));
-    CKI(L.go(ssdk::conv_state_kernel<T>, dim3(rg.n_seqs, (Cd + 255) / 256), dim3(256), 0, dp.conv, rg));
+    if (taps > 1) CKI(L.go(ssdk::conv_state_kernel<T>, dim3(rg.n_seqs, (Cd + 255) / 256), dim3(256), 0, dp.conv, rg));
     ssdk::DeltaArgs da;
     da.q = dp.q; da.k = dp.k; da.v = dp.v; da.beta = dp.beta; da.decay = dp.decay; da.o = e->p1; da.S = st; da.slot_stride = e->slot_floats;
-    da.H = Hd; da.G = Gd; da.D = Dd; da.V = Vd;
-    const int Vall = (Vd + 31) / 32 * 32;
-    int Vr = Vall, DR = 0, NG = 1;
-    delta_shape(Dd, Vr, &DR, &NG);
-    // the state's columns are independent: few (sequence, head) pairs spread a head's columns over several CTAs
-    while (DR > 0 && Vr % 64 == 0 && rg.n_seqs * Hd * (Vall / Vr) < num_sms()) {
-      Vr /= 2;
-      delta_shape(Dd, Vr, &DR, &NG);
-    }
-    const dim3 grid(rg.n_seqs, Hd, (Vall + Vr - 1) / Vr), block(Vr, NG);
-    const size_t smem = ssdk::delta_scan_smem(Dd, Vr, DR, NG);
-    if (DR == 16) CKI(L.go(ssdk::delta_scan_kernel<16>, grid, block, smem, da, rg));
-    else if (DR == 32) CKI(L.go(ssdk::delta_scan_kernel<32>, grid, block, smem, da, rg));
-    else if (DR == 64) CKI(L.go(ssdk::delta_scan_kernel<64>, grid, block, smem, da, rg));
-    else CKI(L.go(ssdk::delta_scan_kernel<0>, grid, block, smem, da, rg));
-    CKI(L.go(ssdk::head_rmsnorm_gate_kernel<T, 0>, dim3(M, Hd), dim3(std::min(256, Vall)), 0, (const float*)e->p1, (const float*)(e->p0 + o_dg), Ntot,
-             (const T*)Lr.t[SSDK_HT_MIX_NORM].p, (T*)e->t1, Hd, Vd, e->cfg.eps));
+    da.H = Hd; da.G = Gd; da.D = Dd; da.V = Vd; da.vec = Dd % 4 == 0 && Vd % 4 == 0;
+    CKI(Ra ? delta_scan<true>(da) : delta_scan<false>(da));
+    const dim3 ngrid(M, Hd), nblock(std::min(256, (Vd + 31) / 32 * 32));
+    const float* gate = Rg ? gz : e->p0 + o_dg;
+    const int ld_gate = Rg ? dHV : Ntot;
+    const T* nw = (const T*)Lr.t[SSDK_HT_MIX_NORM].p;
+    if (c.d_gate_act) CKI(L.go(ssdk::head_rmsnorm_gate_kernel<T, 1>, ngrid, nblock, 0, (const float*)e->p1, gate, ld_gate, nw, (T*)e->t1, Hd, Vd, e->cfg.eps));
+    else CKI(L.go(ssdk::head_rmsnorm_gate_kernel<T, 0>, ngrid, nblock, 0, (const float*)e->p1, gate, ld_gate, nw, (T*)e->t1, Hd, Vd, e->cfg.eps));
     return lin(e->t1, dHV, Lr.t[SSDK_HT_MIX_OUT].p, dHV, e->mix2, W, M, W, dHV);
+  }
+
+  // the walk of the delta rule over this step's rows; CH: one decay per key channel
+  template <bool CH>
+  int delta_scan(const ssdk::DeltaArgs& da) {
+    // fewer columns than the machine's schedulers hold warps for at four lanes each: twice the lanes per column
+    const bool few = (long long)rg.n_seqs * da.H * da.V * 4 / 32 < 4LL * num_sms();
+    int LC = 0, NQ = 0;
+    delta_shape(da.D, few, &LC, &NQ);
+    if (LC == 0)
+      return L.go(ssdk::delta_scan_any_kernel<CH>, dim3(rg.n_seqs, da.H, (da.V + kDeltaAnyCols - 1) / kDeltaAnyCols), dim3(kDeltaAnyCols),
+                  (size_t)da.D * kDeltaAnyCols * 4, da, rg);
+    const int cols = ssdk::kDeltaWarps * 32 / LC;
+    const dim3 grid(rg.n_seqs, da.H, (da.V + cols - 1) / cols), block(ssdk::kDeltaWarps * 32);
+    const size_t smem = ssdk::delta_scan_smem(4 * LC * NQ, cols, CH);
+    if (LC == 4 && NQ == 1) return L.go(ssdk::delta_scan_kernel<4, 1, CH>, grid, block, smem, da, rg);
+    if (LC == 4 && NQ == 2) return L.go(ssdk::delta_scan_kernel<4, 2, CH>, grid, block, smem, da, rg);
+    if (LC == 8 && NQ == 2) return L.go(ssdk::delta_scan_kernel<8, 2, CH>, grid, block, smem, da, rg);
+    if (LC == 4 && NQ == 4) return L.go(ssdk::delta_scan_kernel<4, 4, CH>, grid, block, smem, da, rg);
+    if (LC == 8 && NQ == 4) return L.go(ssdk::delta_scan_kernel<8, 4, CH>, grid, block, smem, da, rg);
+    if (LC == 4 && NQ == 8) return L.go(ssdk::delta_scan_kernel<4, 8, CH>, grid, block, smem, da, rg);
+    if (LC == 8 && NQ == 8) return L.go(ssdk::delta_scan_kernel<8, 8, CH>, grid, block, smem, da, rg);
+    return L.go(ssdk::delta_scan_kernel<16, 8, CH>, grid, block, smem, da, rg);
   }
 
   int run_mixer(HybLayer& Lr) {
@@ -950,8 +1043,68 @@ struct HybRun {
     return 0;
   }
 
+  // ---- serial pre-norm blocks: x += mixer(norm1(x)); x += ff(norm2(x)), on one residual or on several streams ----
+  int streams() const { return std::max(1, e->cfg.streams); }
+  // coefficients of sublayer q (0: mixer, 1: feed-forward); nullptr without streams
+  const void* hc(const HybLayer& Lr, int id, int q, size_t n) const { return e->cfg.streams ? w_at(Lr.t[id], q * n) : nullptr; }
+
+  // input of a first sublayer, or of the head: h = norm(sum_s in_s x_s)
+  int stream_norm(const void* in, const void* w, void* y, const int* rows, int n_rows, float mult) {
+    return L.go(ssdk::stream_norm_kernel<T>, dim3(n_rows), dim3(256), (size_t)e->cfg.width * 4, (const float*)e->x, streams(), (const T*)in,
+                (const T*)w, (T*)y, rows, e->cfg.width, e->cfg.eps, e->cfg.norm_offset, mult);
+  }
+
+  // the result of sublayer q of layer Lr (mix_out, for the pair also mix2) enters the streams; the next sublayer's input follows
+  int stream_step(HybLayer& Lr, int q, const HybLayer* next, int next_q) {
+    const int S = streams(), W = e->cfg.width;
+    ssdk::StreamStepArgs a = {};
+    a.x = e->x; a.y1 = e->mix_out; a.s1 = 1.f; a.S = S; a.width = W; a.eps = e->cfg.eps; a.offset = e->cfg.norm_offset;
+    if (q == 0 && Lr.c.mixer == SSDK_MIX_ATTN_DELTA) {
+      a.y2 = e->mix2; a.s1 = Lr.c.left_scale; a.s2 = Lr.c.right_scale;
+      if (Lr.c.pair_norm) { a.w1 = Lr.t[SSDK_HT_PAIR_NORM].p; a.w2 = w_at(Lr.t[SSDK_HT_PAIR_NORM], W); }
+    }
+    a.mix = hc(Lr, SSDK_HT_HC_MIX, q, (size_t)S * S); a.out = hc(Lr, SSDK_HT_HC_OUT, q, S);
+    if (next) {
+      a.in = hc(*next, SSDK_HT_HC_IN, next_q, S); a.nw = next->t[next_q ? SSDK_HT_NORM2 : SSDK_HT_NORM].p; a.h = e->h;
+    }
+    const dim3 grid(M), block(256);
+    const size_t smem = (size_t)W * 4;
+    if (W % 4 == 0 && S <= 8) {
+      if (S == 1) return L.go(ssdk::stream_step_kernel<T, 1, 4>, grid, block, smem, a);
+      if (S == 2) return L.go(ssdk::stream_step_kernel<T, 2, 4>, grid, block, smem, a);
+      if (S <= 4) return L.go(ssdk::stream_step_kernel<T, 4, 4>, grid, block, smem, a);
+      return L.go(ssdk::stream_step_kernel<T, 8, 4>, grid, block, smem, a);
+    }
+    if (S <= 4) return L.go(ssdk::stream_step_kernel<T, 4, 1>, grid, block, smem, a);
+    return L.go(ssdk::stream_step_kernel<T, ssdk::kMaxStreams, 1>, grid, block, smem, a);
+  }
+
+  int check_prenorm_layer(const HybLayer& Lr) {
+    const int W = e->cfg.width, S = e->cfg.streams, sub = Lr.c.mlp == SSDK_MLP_NONE ? 1 : 2;
+    CKI(check_tensor(Lr, SSDK_HT_NORM, W, 1, "norm1"));
+    if (sub == 2) CKI(check_tensor(Lr, SSDK_HT_NORM2, W, 1, "norm2"));
+    if (Lr.c.pair_norm) CKI(check_tensor(Lr, SSDK_HT_PAIR_NORM, 2, W, "left.out|right.out"));
+    if (S == 0) return 0;
+    CKI(check_tensor(Lr, SSDK_HT_HC_IN, sub, S, "hc.in")); CKI(check_tensor(Lr, SSDK_HT_HC_OUT, sub, S, "hc.out"));
+    return check_tensor(Lr, SSDK_HT_HC_MIX, sub, (int64_t)S * S, "hc.mix");
+  }
+
+  int prenorm_layer(HybLayer& Lr, int li) {
+    const HybLayer* next = li + 1 < e->cfg.n_layers ? &e->layers[li + 1] : nullptr;
+    CKI(check_prenorm_layer(Lr));
+    if (next) CKI(check_prenorm_layer(*next));
+    if (li == 0) CKI(stream_norm(hc(Lr, SSDK_HT_HC_IN, 0, streams()), Lr.t[SSDK_HT_NORM].p, e->h, nullptr, M, 1.0f));
+    hin = e->h;
+    CKI(run_mixer(Lr));
+    if (Lr.c.mlp == SSDK_MLP_NONE) return stream_step(Lr, 0, next, 0);
+    CKI(stream_step(Lr, 0, &Lr, 1));
+    CKI(glu(Lr));
+    return stream_step(Lr, 1, next, 0);
+  }
+
   int layer(HybLayer& Lr, int li) {
     if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM) return serial_layer(Lr);
+    if (e->cfg.block == SSDK_BLOCK_SERIAL_PRENORM) return prenorm_layer(Lr, li);
     const int W = e->cfg.width;
     const bool two = e->cfg.block == SSDK_BLOCK_PARALLEL_TWO_NORMS;   // norm1 feeds the mixer, norm2 the feed-forward; no layer scales
     const bool one = e->cfg.block == SSDK_BLOCK_PARALLEL_ONE_NORM;    // one norm; input convolutions and residual gates; no layer scales
@@ -996,7 +1149,7 @@ struct HybRun {
       }
     }
     if (Lr.c.mixer == SSDK_MIX_ATTN_DELTA) return fail("the attention pair is built for serial blocks");
-    if (Lr.c.mixer == SSDK_MIX_ATTENTION && !one) return fail("the attention mixer is built for one-norm blocks");
+    if (Lr.c.mixer == SSDK_MIX_ATTENTION && !one) return fail("the attention mixer is built for one-norm and serial pre-norm blocks");
     CKI(run_mixer(Lr));
     ca.x = e->x; ca.mix = e->mix_out; ca.ls1 = scales ? Lr.t[SSDK_HT_LS_MIX].p : nullptr; ca.width = W;
     if (Lr.c.mlp == SSDK_MLP_MOE) {
@@ -1038,10 +1191,23 @@ static int hyb_smem_attrs(ssdk_hyb_engine* e) {
   CK(cudaFuncSetAttribute(ssdk::latent_decode_mma_kernel<3, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::latent_decode_mma_kernel<5, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::latent_decode_mma_kernel<9, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::delta_scan_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::delta_scan_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::delta_scan_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::delta_scan_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+#define SSDK_DELTA_ATTR(LC, NQ) \
+  CK(cudaFuncSetAttribute(ssdk::delta_scan_kernel<LC, NQ, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::delta_scan_kernel<LC, NQ, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  SSDK_DELTA_ATTR(4, 1) SSDK_DELTA_ATTR(4, 2) SSDK_DELTA_ATTR(8, 2) SSDK_DELTA_ATTR(4, 4) SSDK_DELTA_ATTR(8, 4) SSDK_DELTA_ATTR(4, 8)
+  SSDK_DELTA_ATTR(8, 8) SSDK_DELTA_ATTR(16, 8)
+#undef SSDK_DELTA_ATTR
+  CK(cudaFuncSetAttribute(ssdk::delta_scan_any_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::delta_scan_any_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+#define SSDK_STREAM_ATTR(SM, VEC) \
+  CK(cudaFuncSetAttribute(ssdk::stream_step_kernel<bf16, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::stream_step_kernel<float, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  SSDK_STREAM_ATTR(1, 4) SSDK_STREAM_ATTR(2, 4) SSDK_STREAM_ATTR(4, 4) SSDK_STREAM_ATTR(8, 4) SSDK_STREAM_ATTR(4, 1) SSDK_STREAM_ATTR(ssdk::kMaxStreams, 1)
+#undef SSDK_STREAM_ATTR
+  CK(cudaFuncSetAttribute(ssdk::stream_norm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::stream_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::delta_prep_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::delta_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   e->smem_attr_done = true;
@@ -1075,14 +1241,23 @@ static int hyb_forward_t(ssdk_hyb_engine* e, int n_seqs, int M, const int32_t* i
   run.rg.cu = d + o_cu; run.rg.pos0 = d + o_pos; run.rg.slot = d + o_slot; run.rg.tok_seq = d + o_seq; run.rg.tables = d + o_tab;
   run.rg.n_seqs = n_seqs; run.rg.M = M; run.rg.max_blocks = g.max_blocks_per_seq; run.rg.block_size = g.block_size;
   CKI(run.L.go(ssdk::embed_rows_kernel<T>, dim3(M), dim3(128), 0, (const int*)(d + o_ids), (const T*)e->embed.p, e->x, g.width, g.vocab,
-               g.embed_scale, (g.block == SSDK_BLOCK_SERIAL_POSTNORM && !std::is_same<T, float>::value) ? (T*)e->h : (T*)nullptr));
+               g.embed_scale, (g.block == SSDK_BLOCK_SERIAL_POSTNORM && !std::is_same<T, float>::value) ? (T*)e->h : (T*)nullptr, run.streams()));
   for (int li = 0; li < g.n_layers; ++li) {
     CKI(run.layer(e->layers[li], li));
-    if (residual_host)
-      CK(cudaMemcpyAsync(residual_host + (size_t)li * M * g.width, e->x, (size_t)M * g.width * 4, cudaMemcpyDeviceToHost, st));
+    if (residual_host) {
+      const float* res = e->x;
+      if (g.streams > 1) {
+        CKI(run.L.go(ssdk::stream_sum_kernel, dim3(M), dim3(256), 0, (const float*)e->x, e->mix_out, g.streams, g.width));
+        res = e->mix_out;
+      }
+      CK(cudaMemcpyAsync(residual_host + (size_t)li * M * g.width, res, (size_t)M * g.width * 4, cudaMemcpyDeviceToHost, st));
+    }
   }
   if (n_want > 0) {
-    CKI(run.L.go(ssdk::offset_rmsnorm_kernel<T>, dim3(n_want), dim3(256), 0, (const float*)e->x, (const T*)e->final_norm.p, (T*)e->hn,
+    // (a factor on the logits is taken on the normed rows: the head is linear)
+    if (g.block == SSDK_BLOCK_SERIAL_PRENORM || g.logit_scale != 1.0f)
+      CKI(run.stream_norm(nullptr, e->final_norm.p, e->hn, d + o_want, n_want, g.logit_scale));
+    else CKI(run.L.go(ssdk::offset_rmsnorm_kernel<T>, dim3(n_want), dim3(256), 0, (const float*)e->x, (const T*)e->final_norm.p, (T*)e->hn,
                  (const int*)(d + o_want), g.width, g.eps, g.norm_offset, (const T*)nullptr, (T*)nullptr));
     CKI(run.lin(e->hn, g.width, e->head.p, g.width, e->logits, g.vocab, n_want, g.vocab, g.width));
     if (logits_host) CK(cudaMemcpyAsync(logits_host, e->logits, (size_t)n_want * g.vocab * 4, cudaMemcpyDeviceToHost, st));
@@ -1116,7 +1291,10 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
   if (cfg->width < 1 || cfg->vocab < 1 || cfg->n_layers < 1) return fail("ssdk_hyb_create: bad sizes");
   if (cfg->dtype != SSDK_DT_F32 && cfg->dtype != SSDK_DT_BF16) return fail("ssdk_hyb_create: unknown dtype %d", cfg->dtype);
   if (cfg->block != SSDK_BLOCK_PARALLEL_PRENORM && cfg->block != SSDK_BLOCK_SERIAL_POSTNORM && cfg->block != SSDK_BLOCK_PARALLEL_TWO_NORMS &&
-      cfg->block != SSDK_BLOCK_PARALLEL_ONE_NORM) return fail("ssdk_hyb_create: unknown block kind %d", cfg->block);
+      cfg->block != SSDK_BLOCK_PARALLEL_ONE_NORM && cfg->block != SSDK_BLOCK_SERIAL_PRENORM) return fail("ssdk_hyb_create: unknown block kind %d", cfg->block);
+  if (cfg->streams < 0 || cfg->streams > ssdk::kMaxStreams || (cfg->streams && cfg->block != SSDK_BLOCK_SERIAL_PRENORM))
+    return fail("ssdk_hyb_create: %d residual streams (serial pre-norm blocks take up to %d)", cfg->streams, ssdk::kMaxStreams);
+  if ((size_t)cfg->width * 4 > kScanSmemMax) return fail("ssdk_hyb_create: width %d too large", cfg->width);
   if (cfg->canon_taps < 0 || (cfg->block != SSDK_BLOCK_PARALLEL_ONE_NORM && (cfg->canon_taps || cfg->gated_residual)))
     return fail("ssdk_hyb_create: input convolutions and residual gates belong to one-norm blocks");
   if (cfg->max_tokens < 1 || cfg->max_seqs < 1 || cfg->max_logit_rows < 1 || cfg->block_size < 1 || cfg->max_blocks_per_seq < 1)
@@ -1140,7 +1318,7 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
     std::vector<float> f(half);
     const double dims = (double)L.c.rot_dims, base = (double)L.c.rot_base;
     for (int i = 0; i < half; ++i) f[i] = (float)pow(base, -2.0 * i / dims);
-    if (L.c.mixer == SSDK_MIX_ATTN_DELTA && L.c.yarn_factor > 0.f) {
+    if (L.c.yarn_factor > 0.f) {
       // YaRN: dimensions that turn fewer than `slow` times over the original length are slowed by `factor`, those that
       // turn more than `fast` times are kept, a linear ramp in between; cos and sin grow by 0.1 ln(factor) + 1
       const double kPi = 3.14159265358979323846, factor = (double)L.c.yarn_factor, orig = (double)L.c.yarn_original;

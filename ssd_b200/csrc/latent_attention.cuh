@@ -111,21 +111,33 @@ __global__ void latent_gather_kernel(const T* __restrict__ cache, T* __restrict_
   }
 }
 
+// Which keys a causal query sees: those at first(pos) .. pos.  A sliding window keeps the last `window` positions, chunks are
+// counted from the sequence's start and end at the query's own chunk; 0 = no window, no chunks.
+struct KeyMask {
+  int window, chunk;
+  __host__ __device__ __forceinline__ int first(int pos) const {
+    int f = window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0;
+    if (chunk > 0) { const int c = pos / chunk * chunk; f = c > f ? c : f; }
+    return f;
+  }
+  __host__ __device__ __forceinline__ bool any() const { return window > 0 || chunk > 0; }
+};
+
 // Softmax with a sink over the score rows of one query block.  The rows come in `batches` of rows_per_batch (one batch
 // per key/value head of grouped-query attention; a single batch for latent attention); inside a batch row r is
 // (query q0 + r / H, head r % H) with H the heads that share the batch's keys.  Column j of a row is the key at position
-// key_first + j; the query at position pos sees the keys at max(0, pos - window + 1) .. pos (window = 0: at 0 .. pos).
+// key_first + j; the query at position pos sees the keys at mask.first(pos) .. pos.
 // sc [rows, ld] fp32 raw dot products -> pr [rows, ld] (T) weights, zero outside the visible range and in the padding.
 // The sink is a learned per-head logit (`sink`, indexed batch * H + head) or, without one, the constant sink_const added
 // to the denominator (0: plain softmax); it joins the maximum, is not scaled and contributes nothing to the output.
 template <typename T>
 __global__ void sink_softmax_kernel(const float* __restrict__ sc, T* __restrict__ pr, const T* __restrict__ sink, int H, int ld,
-                                    int pos_first, float scale, int rows_per_batch, float sink_const, int key_first, int window) {
+                                    int pos_first, float scale, int rows_per_batch, float sink_const, int key_first, KeyMask mask) {
   __shared__ float red[33];
   const int r = blockIdx.x, batch = r / rows_per_batch, rb = r - batch * rows_per_batch;
   const int h = rb % H, pos = pos_first + rb / H;
   const int n = pos - key_first + 1;                                             // columns [j0, n) are the keys this row sees
-  const int j0 = window > 0 ? max(0, pos - window + 1 - key_first) : 0;
+  const int j0 = max(0, mask.first(pos) - key_first);
   const float* srow = sc + (size_t)r * ld;
   const float sk = sink ? ld_f<T>(sink + batch * H + h) : (sink_const > 0.f ? logf(sink_const) : -INFINITY);
   float mx = sk;
@@ -154,12 +166,12 @@ struct LatentDecodeArgs {
   int H, KR, W, splits;
   int pool_aligned;   // the pool starts on a 16-byte boundary
   float scale;
-  int window;         // the token at position p sees the keys at max(0, p - window + 1) .. p; 0: all of 0 .. p
+  KeyMask mask;       // first key the token sees
 };
 
 // keys [k_lo, k_hi) of split j (of `splits`) for a single token at position ctx - 1
-SSDK_DEVINL void decode_split(int ctx, int window, int j, int splits, int* k_lo, int* k_hi) {
-  const int first = window > 0 ? max(0, ctx - window) : 0, per = (ctx - first + splits - 1) / splits;
+SSDK_DEVINL void decode_split(int ctx, const KeyMask& mask, int j, int splits, int* k_lo, int* k_hi) {
+  const int first = mask.first(ctx - 1), per = (ctx - first + splits - 1) / splits;
   *k_lo = first + j * per;
   *k_hi = min(ctx, *k_lo + per);
 }
@@ -196,7 +208,7 @@ __global__ void __launch_bounds__(kDecThreads) latent_decode_partial_kernel(cons
   T* ct = (T*)(rs + H);                    // [kDecTile, W] key rows
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   int k_lo, k_hi;
-  decode_split(rg.pos0[s] + 1, p.window, j, p.splits, &k_lo, &k_hi);
+  decode_split(rg.pos0[s] + 1, p.mask, j, p.splits, &k_lo, &k_hi);
   const T* q = (const T*)p.qcat + (size_t)row * H * W;
   constexpr int kPerVec = 16 / (int)sizeof(T);
   const size_t ct_off = ((size_t)kDecTile * Hp + (size_t)H * W + (size_t)H * KR + 3 * (size_t)H) * 4;
@@ -326,7 +338,7 @@ __global__ void __launch_bounds__(kDmThreads) latent_decode_mma_kernel(const Lat
   float* rs = ls + 16;                                         // [16] rescale of this tile
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
   int k_lo, k_hi;
-  decode_split(rg.pos0[s] + 1, p.window, j, p.splits, &k_lo, &k_hi);
+  decode_split(rg.pos0[s] + 1, p.mask, j, p.splits, &k_lo, &k_hi);
   const int vpr = W / 8;   // 16-byte vectors per row
   const __nv_bfloat16* cache = (const __nv_bfloat16*)p.cache;
   auto load_tile = [&](int k0, int buf) {

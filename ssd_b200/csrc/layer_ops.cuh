@@ -1,6 +1,6 @@
 // layer_ops.cuh — the element-wise steps of a layered (hybrid) model's block.  The residual stream, every norm
 // statistic and every gate are fp32; T (bf16 or float) is the storage type of the activations that feed a linear layer.
-//   embed_rows_kernel         x = embed[token] * scale                          (fp32 residual; optional T copy)
+//   embed_rows_kernel         x = embed[token] * scale                          (fp32 residual, `copies` streams; optional T copy)
 //   offset_rmsnorm_kernel     y = x / sqrt(mean(x^2) + eps) * (offset + w)       (offset 1: unit-offset weight, 0: plain);
 //                             optionally a second output with a second weight from the same statistic (two-norm blocks)
 //   postnorm_residual_kernel  x += mult * norm(s1 y1 + s2 y2): the norm sits on a sublayer's OUTPUT (serial blocks)
@@ -12,6 +12,11 @@
 //   head_rmsnorm_gate_kernel  per-head unit RMS, times a channel weight, times silu / sigmoid of a gate pre-activation
 //   clamped_glu_kernel        y = g * sigmoid(1.702 g) * (u + 1) with g = min(g, lim), u = clamp(u, -lim, lim)
 //   unary_kernel              tanh (decay low-rank bottleneck)
+//   stream_norm_kernel        y = norm(sum_s in_s x_s) * mult over the residual streams of a row (in = 1 without coefficients)
+//   stream_step_kernel        one pass over the streams between two sublayers: the old sublayer's result (one tensor, or two with
+//                             an RMS norm and a factor each) is written back, x_t = sum_s mix[s, t] x_s + out[t] y, and the next
+//                             sublayer's input norm(sum_t in[t] x_t) is made from the new streams while they are in registers
+//   stream_sum_kernel         the sum of the streams
 //   block_combine_kernel      parallel block: x += ls1 * g1 * mixer + ls2 * g2 * (sum_k w_k expert_k + sigmoid(sg) * shared + b);
 //                             ls1, ls2, sg, b are optional (1, 1, no gate, 0), and so are the per-token, per-channel residual
 //                             gates g = sigmoid(pre-activation + bias); an identity expert's output is the feed-forward's
@@ -83,13 +88,13 @@ SSDK_DEVINL void st_contig(T* p, const float* f) {
 
 template <typename T>
 __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restrict__ embed, float* __restrict__ x, int width,
-                                  int vocab, float scale, T* __restrict__ xt) {
+                                  int vocab, float scale, T* __restrict__ xt, int copies) {
   const int m = blockIdx.x;
   int id = ids[m];
   id = min(max(id, 0), vocab - 1);
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     const float v = ld_f<T>(embed + (size_t)id * width + c) * scale;
-    x[(size_t)m * width + c] = v;
+    for (int s = 0; s < copies; ++s) x[((size_t)m * copies + s) * width + c] = v;
     if (xt) st_f<T>(xt + (size_t)m * width + c, v);
   }
 }
@@ -307,6 +312,153 @@ __global__ void block_combine_kernel(const CombineArgs p) {
       y = p.ls2 ? fmaf(ld_f<T>((const T*)p.ls2 + c), f, y) : y + f;
     }
     p.x[(size_t)m * p.width + c] += y;
+  }
+}
+
+// ---------------------------------------------------------------------------------------------- residual streams
+// x [M, S, width] fp32: the S streams of a row lie side by side.
+
+// y[r] = mult * norm(sum_s in[s] x[rows[r]][s]); rows (optional): gather.  dynamic shared memory: width floats
+template <typename T>
+__global__ void stream_norm_kernel(const float* __restrict__ x, int S, const T* __restrict__ in, const T* __restrict__ w, T* __restrict__ y,
+                                   const int* __restrict__ rows, int width, float eps, float offset, float mult) {
+  extern __shared__ float sn_u[];
+  __shared__ float red[33];
+  const int r = blockIdx.x;
+  const float* xr = x + (size_t)(rows ? rows[r] : r) * S * width;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    float u = 0.f;
+    for (int s = 0; s < S; ++s) u = fmaf(in ? ld_f<T>(in + s) : 1.f, xr[(size_t)s * width + c], u);
+    sn_u[c] = u;
+    ss = fmaf(u, u, ss);
+  }
+  ss = block_sum(ss, red);
+  const float inv = mult / sqrtf(ss / (float)width + eps);
+  for (int c = threadIdx.x; c < width; c += blockDim.x) st_f<T>(y + (size_t)r * width + c, sn_u[c] * inv * (offset + ld_f<T>(w + c)));
+}
+
+__global__ void stream_sum_kernel(const float* __restrict__ x, float* __restrict__ y, int S, int width) {
+  const float* xr = x + (size_t)blockIdx.x * S * width;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    float u = 0.f;
+    for (int s = 0; s < S; ++s) u += xr[(size_t)s * width + c];
+    y[(size_t)blockIdx.x * width + c] = u;
+  }
+}
+
+constexpr int kMaxStreams = 32;
+
+struct StreamStepArgs {
+  float* x;               // [M, S, width], updated in place
+  const float* y1;        // [M, width] the sublayer's result, or its first part
+  const float* y2;        // [M, width] second part, or nullptr
+  float s1, s2;           // factors of the parts
+  const void* w1;         // [width] T weights of the parts' norms (plain), or nullptr: parts as they are
+  const void* w2;
+  const void* mix;        // [S (from), S (to)] T, or nullptr (S = 1): x += y
+  const void* out;        // [S] T
+  const void* in;         // [S] T of the next sublayer, or nullptr: 1
+  const void* nw;         // [width] T norm weight of the next sublayer
+  void* h;                // [M, width] T the next sublayer's input, or nullptr: the row has no next sublayer here
+  int S, width;
+  float eps, offset;
+};
+
+// VEC channels per thread and step
+template <int VEC> SSDK_DEVINL void ld_vec(const float* p, float* f) {
+  if constexpr (VEC == 4) { const float4 v = *reinterpret_cast<const float4*>(p); f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
+  else f[0] = *p;
+}
+template <int VEC> SSDK_DEVINL void st_vec(float* p, const float* f) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
+
+// grid (M).  SM >= S: streams held in registers; VEC = 4 needs a width that is a multiple of 4.  dynamic shared memory: width floats
+template <typename T, int SM, int VEC>
+__global__ void stream_step_kernel(const StreamStepArgs p) {
+  extern __shared__ float ss_u[];
+  __shared__ float red[33], cmix[SM * SM], cout[SM], cin[SM];
+  const int S = p.S, W = p.width;
+  for (int i = threadIdx.x; i < S * S; i += blockDim.x) cmix[i / S * SM + i % S] = p.mix ? ld_f<T>((const T*)p.mix + i) : 1.f;
+  for (int i = threadIdx.x; i < S; i += blockDim.x) {
+    cout[i] = p.out ? ld_f<T>((const T*)p.out + i) : 1.f;
+    cin[i] = p.in ? ld_f<T>((const T*)p.in + i) : 1.f;
+  }
+  const size_t row = (size_t)blockIdx.x * W;
+  float* xr = p.x + row * S;
+  float f1 = p.s1, f2 = p.s2;
+  if (p.w1) {
+    float a = 0.f, b = 0.f;
+    for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+      float v[VEC];
+      ld_vec<VEC>(p.y1 + row + c, v);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) a = fmaf(v[e], v[e], a);
+      if (p.y2) {
+        ld_vec<VEC>(p.y2 + row + c, v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) b = fmaf(v[e], v[e], b);
+      }
+    }
+    a = block_sum(a, red);
+    f1 /= sqrtf(a / (float)W + p.eps);
+    if (p.y2) { b = block_sum(b, red); f2 /= sqrtf(b / (float)W + p.eps); }
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float y[VEC], xo[SM][VEC], u[VEC];
+    ld_vec<VEC>(p.y1 + row + c, y);
+#pragma unroll
+    for (int s = 0; s < SM; ++s)
+      if (s < S) ld_vec<VEC>(xr + (size_t)s * W + c, xo[s]);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) { y[e] *= f1 * (p.w1 ? ld_f<T>((const T*)p.w1 + c + e) : 1.f); u[e] = 0.f; }
+    if (p.y2) {
+      float y2[VEC];
+      ld_vec<VEC>(p.y2 + row + c, y2);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = fmaf(y2[e], f2 * (p.w2 ? ld_f<T>((const T*)p.w2 + c + e) : 1.f), y[e]);
+    }
+#pragma unroll
+    for (int t = 0; t < SM; ++t) {
+      if (t < S) {
+        float xn[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) xn[e] = cout[t] * y[e];
+#pragma unroll
+        for (int s = 0; s < SM; ++s)
+          if (s < S) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) xn[e] = fmaf(cmix[s * SM + t], xo[s][e], xn[e]);
+          }
+        st_vec<VEC>(xr + (size_t)t * W + c, xn);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) u[e] = fmaf(cin[t], xn[e], u[e]);
+      }
+    }
+    if (p.h) {
+      st_vec<VEC>(ss_u + c, u);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss = fmaf(u[e], u[e], ss);
+    }
+  }
+  if (!p.h) return;
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)W + p.eps);
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {   // the thread's own entries of u
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss_u[c + e] *= inv * (p.offset + ld_f<T>((const T*)p.nw + c + e));
+    T* h = (T*)p.h + row + c;
+    if constexpr (VEC == 4 && sizeof(T) == 2) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(ss_u[c], ss_u[c + 1]), hi = __floats2bfloat162_rn(ss_u[c + 2], ss_u[c + 3]);
+      *reinterpret_cast<uint2*>(h) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st_f<T>(h + e, ss_u[c + e]);
+    }
   }
 }
 

@@ -1,4 +1,4 @@
-"""Layered ("hybrid") models: a program of layers, each one token mixer + an optional feed-forward.  Four designs are
+"""Layered ("hybrid") models: a program of layers, each one token mixer + an optional feed-forward.  Five designs are
 served through this module, told apart by config.json's `"architecture"`:
 
     Pikavik   parallel pre-norm blocks (mixer and mixture-of-experts feed-forward read the same normed input, unit-offset
@@ -19,6 +19,12 @@ served through this module, told apart by config.json's `"architecture"`:
               without positions (sliding window, plain softmax); feed-forward dense with a PolyNorm activation or a
               mixture of squared-relu experts whose weights are the softmax over the chosen logits, plus a gated shared
               expert
+    Vatolorn  serial pre-norm blocks over several residual streams (a sublayer reads a weighted sum of the streams; the
+              new streams are a mixture of the old ones plus a share each of its result); mixer `parallel`:
+              grouped-query attention over chunks of positions (biased q | k | v behind a short convolution, RMS norm over
+              the whole query and key projection, YaRN-scaled interleaved rotation, plain softmax) beside a gated delta
+              rule with a decay per key channel (low-rank decay and output-gate projections), both results RMS-normed
+              and averaged; dense silu-GLU feed-forward; scaled logits
 
     HybridSpec     what config.json (and, for sizes it does not list, the checkpoint's tensor shapes) says
     load_hybrid_weights   safetensors -> device tensors in the packed layout libssdk's ssdk_hyb_bind expects
@@ -47,7 +53,7 @@ DESIGNS = {
     "Pikavik": {"mixers": ("wkv", "mlstm", "latent_attention"), "mlp": ("moe",), "block": L.BLOCK_PARALLEL_PRENORM,
                 "norm_offset": 1.0},
     "Kefurax": {"mixers": ("rglru", "mamba1", "parallel"), "mlp": ("dense",), "block": L.BLOCK_SERIAL_POSTNORM,
-                "norm_offset": 0.0},
+                "norm_offset": 0.0, "pair": {"qk_norm": 1, "sink": 1.0, "pair_gate": 1}, "ffn": {"ff_act": L.ACT_GELU_TANH}},
     # constants the design fixes, as the arguments the shared mechanisms take
     "Lisenex": {"mixers": ("latent_attention",), "mlp": ("dense", "moe"), "block": L.BLOCK_PARALLEL_TWO_NORMS,
                 "norm_offset": 0.0, "dense": "ffn", "tied_head": True,
@@ -61,8 +67,17 @@ DESIGNS = {
                 "latent": {"rot_interleaved": 0, "out_gate": 0, "learned_sink": 0},
                 "moe": {"route_top_softmax": 1, "group_best": 1, "expert_act": L.ACT_RELU2, "expert_glu": 0, "shared_gate": 1},
                 "ffn": {"ff_act": L.ACT_POLYNORM}},
+    "Vatolorn": {"mixers": ("parallel",), "mlp": ("dense",), "block": L.BLOCK_SERIAL_PRENORM, "norm_offset": 0.0,
+                 "pair": {"qk_norm": 2, "pair_norm": 1, "d_gate_act": 1, "left_scale": 0.5, "right_scale": 0.5},
+                 "pair_low_rank": True, "ffn": {"ff_act": L.ACT_SILU}},
 }
 RGLRU_DECAY_MULT = 8.0  # log a = -8 r softplus(lam)
+
+
+def whole8(n: int) -> int:
+    """Bottleneck ranks are bound padded with zero rows to a multiple of 8: the second product then always has rows of whole
+    16-byte vectors."""
+    return -(-n // 8) * 8
 
 
 @dataclass
@@ -133,6 +148,16 @@ class LayerSpec:
     rot_half: int = 0
     expert_glu: int = 1
     route_top_softmax: int = 0
+    # attention over chunks of positions (0: none); variants of the `parallel` mixer: sigmoid gate on the attention's heads,
+    # convolution taps of its q | k | v (0: none), norms on both results, ranks of the delta rule's decay and output-gate
+    # bottlenecks (0: one decay per head / the gate straight from the input), output gate 0 silu, 1 sigmoid
+    chunk: int = 0
+    pair_gate: int = 0
+    pair_conv: int = 0
+    pair_norm: int = 0
+    d_decay_rank: int = 0
+    d_gate_rank: int = 0
+    d_gate_act: int = 0
 
     def cfg(self) -> L.HybLayerCfg:
         mlp = {"moe": L.MLP_MOE, "dense": L.MLP_GLU, "ffn": L.MLP_FFN, None: L.MLP_NONE}[self.mlp]
@@ -146,7 +171,8 @@ class LayerSpec:
                              self.rot_interleaved, self.kv_from, self.out_gate, self.learned_sink, self.identity,
                              self.route_softmax, self.route_bias, self.group_best, self.route_renorm, self.expert_act,
                              self.shared_gate, self.ff_act, self.window, self.rot_half, self.expert_glu,
-                             self.route_top_softmax)
+                             self.route_top_softmax, self.chunk, self.pair_gate, self.pair_conv, self.pair_norm,
+                             whole8(self.d_decay_rank), whole8(self.d_gate_rank), self.d_gate_act)
 
 
 @dataclass
@@ -159,6 +185,8 @@ class HybridSpec:
     embed_scale: float = 1.0
     residual_mult: float = 1.0
     canon_taps: int = 0       # one-norm blocks: taps of the sublayers' input convolutions (0: none)
+    streams: int = 0          # serial pre-norm blocks: residual streams (0: one plain residual)
+    logit_scale: float = 1.0
 
     @property
     def gated_residual(self) -> bool:
@@ -210,14 +238,23 @@ class HybridSpec:
                 a, d = m["left"], m["right"]
                 rot = a.get("rot") or {}
                 sc = rot.get("scaling") or {}
-                ls = LayerSpec(mixer=kind, heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]),
-                               vdim=int(a["vdim"]), attn_scale=float(a["scale"]), qk_norm=1, sink=1.0,
+                ls = LayerSpec(mixer=kind, heads=int(a["heads"]), kv_heads=int(a.get("kv_heads", a["heads"])), dim=int(a["dim"]),
+                               vdim=int(a.get("vdim", a["dim"])), attn_scale=float(a["scale"]), pair_conv=int(a.get("conv") or 0),
+                               chunk=int((a.get("mask") or {}).get("size", 0)),
                                rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)),
                                yarn_factor=float(sc.get("factor", 0.0)), yarn_original=float(sc.get("original", 0.0)),
                                yarn_fast=float(sc.get("fast", 0.0)), yarn_slow=float(sc.get("slow", 0.0)),
-                               d_heads=int(d["heads"]), d_kv_heads=int(d["kv_heads"]), d_dim=int(d["dim"]),
-                               d_vdim=int(d["vdim"]), conv=int(d["conv"]), left_scale=float(m["left_scale"]),
-                               right_scale=float(m["right_scale"]))
+                               d_heads=int(d["heads"]), d_kv_heads=int(d.get("kv_heads", d["heads"])), d_dim=int(d["dim"]),
+                               d_vdim=int(d.get("vdim", d["dim"])), conv=int(d.get("conv") or 1),
+                               left_scale=float(m.get("left_scale", 1.0)), right_scale=float(m.get("right_scale", 1.0)))
+                for key, val in (design.get("pair") or {}).items():
+                    setattr(ls, key, val)
+                if design.get("pair_low_rank"):   # ranks of the two bottlenecks: only the tensors' shapes give them
+                    for field_, name in (("d_decay_rank", "a1"), ("d_gate_rank", "g1")):
+                        rank = int(shapes[f"l{i}.mix.right.{name}"][0]) if shapes is not None else int(d.get(name, 0))
+                        if rank < 1:
+                            raise ValueError(f"layer {i}: the rank of the delta rule's {name} is unknown")
+                        setattr(ls, field_, rank)
             elif kind == "attention":
                 rot = m.get("rot") or {}
                 ls = LayerSpec(mixer=kind, heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=int(m["dim"]),
@@ -272,7 +309,9 @@ class HybridSpec:
         return cls(width=int(cfg["width"]), vocab=int(cfg["vocab"]), eps=float(cfg["norm"]["eps"]), layers=layers,
                    architecture=arch, embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
                    residual_mult=float(cfg.get("residual_mult", 1.0)),
-                   canon_taps=int((cfg.get("canon") or {}).get("taps", 0)) if design["block"] == L.BLOCK_PARALLEL_ONE_NORM else 0)
+                   canon_taps=int((cfg.get("canon") or {}).get("taps", 0)) if design["block"] == L.BLOCK_PARALLEL_ONE_NORM else 0,
+                   streams=int(cfg.get("streams") or 0) if design["block"] == L.BLOCK_SERIAL_PRENORM else 0,
+                   logit_scale=float(cfg.get("logit_scale", 1.0)))
 
     @classmethod
     def from_dir(cls, path: str) -> "HybridSpec":
@@ -323,7 +362,8 @@ def pack_hybrid_weights(spec: HybridSpec, raw: dict[str, torch.Tensor], dtype: t
     w["HEAD"] = w["EMBED"] if spec.tied_head else dev(t("head"))   # a tied head reads the table itself (without its scale)
     two_norms = spec.block == L.BLOCK_PARALLEL_TWO_NORMS
     one_norm = spec.block == L.BLOCK_PARALLEL_ONE_NORM
-    scales = not two_norms and not one_norm
+    serial_pre = spec.block == L.BLOCK_SERIAL_PRENORM
+    scales = not two_norms and not one_norm and not serial_pre
     for i, ls in enumerate(spec.layers):
         p, mx = f"l{i}.", f"l{i}.mix."
         lw = {"NORM": dev(t(p + "norm1"))}
@@ -334,6 +374,10 @@ def pack_hybrid_weights(spec: HybridSpec, raw: dict[str, torch.Tensor], dtype: t
             if spec.gated_residual:
                 lw["RES_GATE"] = dev(torch.cat([t(p + "rg" + k) for k in subs]))
                 lw["RES_GATE_B"] = dev(torch.cat([t(p + "rg" + k + ".b") for k in subs]))
+        if serial_pre and spec.streams:   # per sublayer: how the streams are read, mixed and written
+            subs = ("1", "2") if ls.mlp else ("1",)
+            for name, key in (("HC_IN", "in"), ("HC_OUT", "out"), ("HC_MIX", "mix")):
+                lw[name] = dev(torch.stack([t(f"{p}hc{k}.{key}") for k in subs]))
         if ls.mixer in ("wkv", "mlstm", "latent_attention"):
             lw["MIX_OUT"] = dev(t(mx + "o"))
             if scales:
@@ -353,8 +397,26 @@ def pack_hybrid_weights(spec: HybridSpec, raw: dict[str, torch.Tensor], dtype: t
             lw["SEL_ALOG"], lw["SEL_D"], lw["MIX_OUT"] = dev(t(mx + "A_log")), dev(t(mx + "D")), dev(t(mx + "o"))
         elif ls.mixer == "parallel":
             a, d = mx + "left.", mx + "right."
-            lw["PAIR_IN"] = dev(torch.cat([t(a + "q"), t(a + "k"), t(a + "v"), t(a + "g"),
-                                           t(d + "q"), t(d + "k"), t(d + "v"), t(d + "g"), t(d + "b"), t(d + "a")]))
+            def pad_rank(x, dim):   # zero rows (dim 0) or columns (dim 1) up to a whole multiple of 8
+                n = whole8(x.shape[dim]) - x.shape[dim]
+                return torch.nn.functional.pad(x, (0, 0, 0, n) if dim == 0 else (0, n))
+            rows = [t(a + "q"), t(a + "k"), t(a + "v")] + ([t(a + "g")] if ls.pair_gate else [])
+            rows += [t(d + "q"), t(d + "k"), t(d + "v")] + ([] if ls.d_gate_rank else [t(d + "g")]) + [t(d + "b")]
+            rows += [pad_rank(t(d + "a1"), 0)] if ls.d_decay_rank else [t(d + "a")]
+            rows += [pad_rank(t(d + "g1"), 0)] if ls.d_gate_rank else []
+            lw["PAIR_IN"] = dev(torch.cat(rows))
+            if ls.d_decay_rank:
+                lw["DELTA_A2"] = dev(pad_rank(t(d + "a2"), 1))
+            if ls.d_gate_rank:
+                lw["DELTA_G2"] = dev(pad_rank(t(d + "g2"), 1))
+            if a + "q.b" in raw:
+                lw["ATTN_IN_B"] = dev(torch.cat([t(a + "q.b"), t(a + "k.b"), t(a + "v.b")]))
+            if ls.pair_conv:
+                lw["ATTN_CONV_W"] = dev(torch.cat([t(a + "q.conv"), t(a + "k.conv"), t(a + "v.conv")]))
+            if ls.qk_norm == 2:
+                lw["ATTN_QK_NORM"] = dev(torch.cat([t(a + "q.norm"), t(a + "k.norm")]))
+            if ls.pair_norm:
+                lw["PAIR_NORM"] = dev(torch.stack([t(a + "out"), t(d + "out")]))
             lw["ATTN_OUT"], lw["MIX_OUT"] = dev(t(a + "o")), dev(t(d + "o"))
             lw["CONV_W"] = dev(torch.cat([t(d + "q.conv"), t(d + "k.conv"), t(d + "v.conv")]))
             lw["DELTA_ALOG"], lw["DELTA_DT_B"] = dev(t(d + "A_log")), dev(t(d + "dt_bias"))
@@ -593,7 +655,7 @@ class HybridRunner:
         self.max_logit_rows = max_logit_rows or max(1, min(max_tokens, (1 << 30) // spec.vocab))
         cfg = L.HybCfg(spec.width, spec.vocab, len(spec.layers), L.DT_BF16 if self.dtype == torch.bfloat16 else L.DT_F32,
                        spec.eps, max_tokens, max_seqs, self.max_logit_rows, block_size, self.max_blocks, spec.block, spec.norm_offset,
-                       spec.embed_scale, spec.residual_mult, spec.canon_taps, int(spec.gated_residual))
+                       spec.embed_scale, spec.residual_mult, spec.canon_taps, int(spec.gated_residual), spec.streams, spec.logit_scale)
         layer_cfgs = (L.HybLayerCfg * len(spec.layers))(*[l.cfg() for l in spec.layers])
         h = C.c_void_p()
         L.check(self.lib.ssdk_hyb_create(C.byref(cfg), layer_cfgs, C.byref(h)), "ssdk_hyb_create")

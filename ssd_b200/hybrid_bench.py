@@ -51,7 +51,7 @@ def pikavik_spec(z):
 def kefurax_spec(z):
     """Layers that resemble a real model's: 128-wide heads, four query heads per key/value head, a delta rule with
     128 x 128 heads, a selective scan of twice the width with 16 states, a recurrence as wide as the model."""
-    from .hybrid import RGLRU_DECAY_MULT, HybridSpec, LayerSpec
+    from .hybrid import DESIGNS, RGLRU_DECAY_MULT, HybridSpec, LayerSpec
     W = z["width"]
     heads, ff = W // 128, z["top"] * z["ff"] + z["sff"]
     layers = []
@@ -59,13 +59,15 @@ def kefurax_spec(z):
         kind = ("parallel", "mamba1", "rglru", "parallel")[i % 4]
         if kind == "parallel":
             layers.append(LayerSpec("parallel", heads, 128, 128, rot_dims=64, rot_base=10000.0, attn_scale=128 ** -0.5,
-                                    kv_heads=max(1, heads // 4), qk_norm=1, sink=1.0, yarn_factor=4.0, yarn_original=4096.0,
+                                    kv_heads=max(1, heads // 4), yarn_factor=4.0, yarn_original=4096.0,
                                     yarn_fast=16.0, yarn_slow=2.0, conv=4, d_heads=heads, d_kv_heads=max(1, heads // 2), d_dim=128,
-                                    d_vdim=128, left_scale=1.0, right_scale=1.0, mlp="dense", ff=ff))
+                                    d_vdim=128, left_scale=1.0, right_scale=1.0, mlp="dense", ff=ff, **DESIGNS["Kefurax"]["pair"],
+                                    **DESIGNS["Kefurax"]["ffn"]))
         elif kind == "mamba1":
-            layers.append(LayerSpec("mamba1", 1, 1, inner=2 * W, state=16, dt_rank=W // 16, conv=4, mlp="dense", ff=ff))
+            layers.append(LayerSpec("mamba1", 1, 1, inner=2 * W, state=16, dt_rank=W // 16, conv=4, mlp="dense", ff=ff, **DESIGNS["Kefurax"]["ffn"]))
         else:
-            layers.append(LayerSpec("rglru", 1, 1, inner=W, blocks=heads, conv=4, decay_mult=RGLRU_DECAY_MULT, mlp="dense", ff=ff))
+            layers.append(LayerSpec("rglru", 1, 1, inner=W, blocks=heads, conv=4, decay_mult=RGLRU_DECAY_MULT, mlp="dense", ff=ff,
+                                    **DESIGNS["Kefurax"]["ffn"]))
     return HybridSpec(W, z["vocab"], 1e-6, layers, architecture="Kefurax", embed_scale=1.0, residual_mult=0.7)
 
 
