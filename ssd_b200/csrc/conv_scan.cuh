@@ -10,8 +10,9 @@
 //                         no bias; input_conv_state_kernel saves the last taps - 1 rows of h
 //   rglru_scan_kernel     S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t,  a_t = exp(-c r_t softplus(lam)),  out = S_t gelu(y_t)
 //   selective_scan_kernel S[c,n] = exp(dt_c A[c,n]) S[c,n] + dt_c x_c B_n,  y_c = sum_n S[c,n] C_n + D_c x_c,  out = y silu(z)
-//   delta_prep_kernel     convolution + SiLU of q | k | v, unit vectors per head for q and k, beta and the head decay
-//   delta_scan_kernel     gated delta rule: S = g S; u = beta (v - S^T k); S += k u^T; o = S^T q
+//   delta_chunk_prep_kernel  gated delta rule, everything that does not depend on the state: convolution + SiLU of q | k | v,
+//                         unit vectors per head, beta, decays per head or per key channel, and per chunk of rows their products
+//   delta_chunk_scan_kernel  the walk over the chunks: S = g S; u = beta (v - S^T k); S += k u^T; o = S^T q
 //
 // A state slot is never cleared: a sequence whose portion starts at position 0 ignores what the slot holds.
 #pragma once
@@ -366,254 +367,428 @@ __global__ void selective_scan_kernel(const SelScanArgs p, const Ragged rg) {
 }
 
 // ---------------------------------------------------------------------------------------------- gated delta rule
+// Per head, S [D, V]:  S = diag(g_t) S;  u_t = beta_t (v_t - S^T k_t);  S += k_t u_t^T;  o_t = S^T q_t.
+// C consecutive rows (a chunk) are taken together.  With S the state before the chunk, G_i = g_1 .. g_i (per key channel) and
+// G_(j,i] = g_(j+1) .. g_i, unrolling the recurrence gives
+//     u_i = beta_i (v_i - (G_i k_i)^T S - sum_{j<i} A_ij u_j),         A_ij = sum_d k_i G_(j,i] k_j
+//     o_i = (G_i q_i)^T S + sum_{j<=i} B_ij u_j,                       B_ij = sum_d q_i G_(j,i] k_j
+//     S  <- S + (G_C - 1) S + sum_i (G_(i,C] k_i) u_i^T
+// A, B and every scaled k and q are independent of the state, and so is X = (I + diag(beta) A)^-1 diag(beta) (unit triangular
+// inverse): u = X r and o = (G q)^T S + (B X) r with r_i = v_i - (G_i k_i)^T S.  delta_chunk_prep_kernel makes them for all
+// chunks at once, delta_chunk_scan_kernel walks the chunks.  No quotient of decays is formed, so any decay in (0, 1] is safe;
+// the factor that survives from chunk to chunk, G_C - 1, comes from expm1 of the summed log decays.  All fp32.
+//
+// Record of one (chunk, head), DP >= D padded with zeros:  G k [C][DP] | G_(.,C] k [C][DP] | G q [C][DP] | G_C - 1 [DP] |
+// X [C][C] | B X [C][C] (C = 1: padded to 4 floats).  Rows behind the portion's end are zero.
+inline __host__ __device__ int delta_record(int DP, int C) { return (3 * C + 1) * DP + (C > 1 ? 2 * C * C : 4); }
+
+constexpr int kDeltaChunk = 8;   // rows of a chunk (1 in calls that bring one row per sequence)
+constexpr int kDeltaTaps = 8;    // convolutions up to this length keep their rows in registers
+
 struct DeltaPrepArgs {
   ConvArgs conv;          // over the q | k | v columns (C = 2 G D + H V); out / out_t unused
   const float* b; int ld_b;    // [M, ...]: beta pre-activations in columns [0, H)
   const float* a; int ld_a;    // decay pre-activations: [M, ...] columns [0, H), or (per_channel) [M, H D]
   const void* A_log;      // [H] T
   const void* dt_bias;    // [H] T, or (per_channel) [H D]
-  float* q;               // [M, G D] unit vectors * q_scale
-  float* k;               // [M, G D] unit vectors
   float* v;               // [M, H V]
-  float* beta;            // [M, H]
-  float* decay;           // g - 1 (exact also where the decay g is within an ulp of 1): [M, H], or (per_channel) [M, H D]; may be `a` itself
-  int H, G, D, V, per_channel;
+  float* rec;             // records, (chunk index, head)
+  int H, G, D, V, DP, per_channel;
   float q_scale, unit_eps;
 };
 
-// grid (M, 2 G + H (+ H when per_channel)): unit u < G is a query head, u < 2 G a key head, then value heads, then the decays of
-// the heads' key channels; one CTA convolves the unit's channels (SiLU), and makes a query or key head a unit vector.
-// dynamic shared memory: max(D, V) floats.
-template <typename T>
-__global__ void delta_prep_kernel(const DeltaPrepArgs p, const Ragged rg) {
+// chunk ci of sequence s: records of different sequences never overlap (a portion of n rows has at most n / C + 1 chunks)
+SSDK_DEVINL size_t delta_chunk_index(const Ragged& rg, int s, int ci, int C) { return (size_t)(rg.cu[s] / C + s + ci); }
+
+// channel c of the convolution at C consecutive rows t0 .. of sequence s (rows from nr on: zero), then SiLU
+template <typename T, int C>
+SSDK_DEVINL void conv_silu_rows(const ConvArgs& p, const Ragged& rg, int s, int t0, int nr, int c, float* y) {
+  const int r0 = rg.cu[s];
+  if (p.taps > kDeltaTaps) {
+#pragma unroll
+    for (int i = 0; i < C; ++i) y[i] = i < nr ? silu_f(conv_at<T>(p, rg, r0 + t0 + i, s, t0 + i, c)) : 0.f;
+    return;
+  }
+  const bool carried = rg.pos0[s] > 0;
+  const float* hist = p.hist + (size_t)rg.slot[s] * p.slot_stride;
+  float w[kDeltaTaps], x[C + kDeltaTaps - 1];   // w[b]: weight of the row b steps back; x[i + kDeltaTaps - 1]: row t0 + i
+#pragma unroll
+  for (int b = 0; b < kDeltaTaps; ++b) w[b] = b < p.taps ? ld_f<T>((const T*)p.w + (size_t)c * p.taps + (p.taps - 1 - b)) : 0.f;
+#pragma unroll
+  for (int i = 1 - kDeltaTaps; i < C; ++i) {
+    const int t = t0 + i;
+    float v = 0.f;
+    if (i > -p.taps && i < nr) {
+      if (t >= 0) v = p.in[(size_t)(r0 + t) * p.ld_in + c];
+      else if (carried) v = hist[(size_t)(p.taps - 1 + t) * p.C + c];
+    }
+    x[i + kDeltaTaps - 1] = v;
+  }
+#pragma unroll
+  for (int i = 0; i < C; ++i) {
+    float acc = 0.f;
+#pragma unroll
+    for (int b = kDeltaTaps - 1; b >= 0; --b) acc = fmaf(w[b], x[i - b + kDeltaTaps - 1], acc);
+    y[i] = i < nr ? silu_f(acc) : 0.f;
+  }
+}
+
+inline size_t delta_prep_smem(int D, int C) { return ((size_t)3 * C * D + 3 * C * C + 3 * C + 4) * 4; }
+
+// grid (chunks of the longest portion, n_seqs, H), 128 threads
+template <typename T, int C>
+__global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaPrepArgs p, const Ragged rg) {
   extern __shared__ float dp_sm[];
-  __shared__ float red[33];
-  const int m = blockIdx.x, unit = blockIdx.y, s = rg.tok_seq[m], t = m - rg.cu[s];
-  const int GD = p.G * p.D, HV = p.H * p.V;
-  if (unit == 0) {
-    for (int h = threadIdx.x; h < p.H; h += blockDim.x) {
-      p.beta[(size_t)m * p.H + h] = sigmoid_f(p.b[(size_t)m * p.ld_b + h]);
-      if (!p.per_channel) {
-        const float sp = softplus_f(p.a[(size_t)m * p.ld_a + h] + ld_f<T>((const T*)p.dt_bias + h));
-        p.decay[(size_t)m * p.H + h] = expm1f(-expf(ld_f<T>((const T*)p.A_log + h)) * sp);
+  constexpr int kThreads = 128, kSlices = kThreads / C;
+  const int ci = blockIdx.x, s = blockIdx.y, h = blockIdx.z, t0 = ci * C, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int m0 = rg.cu[s] + t0, nr = min(C, rg.cu[s + 1] - m0);
+  if (nr <= 0) return;
+  const int D = p.D, V = p.V, DP = p.DP, GD = p.G * D, g = h / (p.H / p.G);
+  float* kk = dp_sm;                // [C][D] keys, then unit keys
+  float* qq = kk + C * D;           // [C][D]
+  float* ll = qq + C * D;           // [C][D] log decays, then decays
+  float* A = ll + C * D;            // [C][C]
+  float* B = A + C * C;             // [C][C]
+  float* X = B + C * C;             // [C][C]
+  float* sc = X + C * C;            // [2 C] 1 / length of the keys, then of the queries
+  float* beta = sc + 2 * C;         // [C]
+  float* rec = p.rec + (delta_chunk_index(rg, s, ci, C) * p.H + h) * delta_record(DP, C);
+  const float rate = -expf(ld_f<T>((const T*)p.A_log + h));
+  for (int d = tid; d < D; d += kThreads) {
+    float y[C];
+    conv_silu_rows<T, C>(p.conv, rg, s, t0, nr, g * D + d, y);
+#pragma unroll
+    for (int i = 0; i < C; ++i) qq[i * D + d] = y[i];
+    conv_silu_rows<T, C>(p.conv, rg, s, t0, nr, GD + g * D + d, y);
+    const int c = p.per_channel ? h * D + d : h;
+    const float bias = ld_f<T>((const T*)p.dt_bias + c);
+#pragma unroll
+    for (int i = 0; i < C; ++i) {
+      kk[i * D + d] = y[i];
+      ll[i * D + d] = i < nr ? rate * softplus_f(p.a[(size_t)(m0 + i) * p.ld_a + c] + bias) : 0.f;
+    }
+  }
+  for (int d = tid; d < V; d += kThreads) {
+    float y[C];
+    conv_silu_rows<T, C>(p.conv, rg, s, t0, nr, 2 * GD + h * V + d, y);
+#pragma unroll
+    for (int i = 0; i < C; ++i)
+      if (i < nr) p.v[((size_t)(m0 + i) * p.H + h) * V + d] = y[i];
+  }
+  if (tid < C) beta[tid] = tid < nr ? sigmoid_f(p.b[(size_t)(m0 + tid) * p.ld_b + h]) : 0.f;
+  __syncthreads();
+  for (int x = warp; x < 2 * C; x += kThreads / 32) {   // (kk and qq are adjacent: row x of the two)
+    float ss = 0.f;
+    for (int d = lane; d < D; d += 32) { const float v = kk[x * D + d]; ss = fmaf(v, v, ss); }
+    ss = warp_sum(ss);
+    if (lane == 0) sc[x] = (x < C ? 1.0f : p.q_scale) / sqrtf(ss + p.unit_eps);
+  }
+  __syncthreads();
+  for (int d = tid; d < DP; d += kThreads) {
+    float k[C], e[C], L = 0.f, G = 1.f;
+#pragma unroll
+    for (int i = 0; i < C; ++i) {
+      float q = 0.f;
+      k[i] = 0.f; e[i] = 1.f;
+      if (d < D) {
+        const float l = ll[i * D + d];
+        k[i] = kk[i * D + d] * sc[i]; q = qq[i * D + d] * sc[C + i]; e[i] = expf(l);
+        kk[i * D + d] = k[i]; qq[i * D + d] = q; ll[i * D + d] = e[i];
+        L += l;
+      }
+      G *= e[i];
+      rec[i * DP + d] = k[i] * G;
+      rec[(2 * C + i) * DP + d] = q * G;
+    }
+    G = 1.f;
+#pragma unroll
+    for (int i = C - 1; i >= 0; --i) { rec[(C + i) * DP + d] = k[i] * G; G *= e[i]; }
+    rec[3 * C * DP + d] = expm1f(L);
+  }
+  __syncthreads();
+  {
+    const int jj = tid / kSlices, sl = tid % kSlices;   // key row jj, channels sl, sl + kSlices, ..
+    float a[C], b[C];
+#pragma unroll
+    for (int i = 0; i < C; ++i) a[i] = b[i] = 0.f;
+    for (int d = sl; d < D; d += kSlices) {
+      float run = kk[jj * D + d];
+#pragma unroll
+      for (int i = 0; i < C; ++i) {
+        if (i > jj) { run *= ll[i * D + d]; a[i] = fmaf(kk[i * D + d], run, a[i]); }
+        if (i >= jj) b[i] = fmaf(qq[i * D + d], run, b[i]);
+      }
+    }
+    if constexpr (C == 1) {
+      b[0] = warp_sum(b[0]);
+      if (lane == 0) A[0] = 0.f;
+      __syncthreads();                 // (sc is free now: the warps' parts of B meet there and in X, A)
+      if (lane == 0) dp_sm[warp] = b[0];
+      __syncthreads();
+      if (tid == 0) {
+        float* x = rec + (3 * C + 1) * DP;
+        x[0] = beta[0]; x[1] = ((dp_sm[0] + dp_sm[1]) + (dp_sm[2] + dp_sm[3])) * beta[0]; x[2] = x[3] = 0.f;
+      }
+      return;
+    } else {
+#pragma unroll
+      for (int o = kSlices >> 1; o > 0; o >>= 1) {
+#pragma unroll
+        for (int i = 0; i < C; ++i) {
+          a[i] += __shfl_xor_sync(0xffffffffu, a[i], o);
+          b[i] += __shfl_xor_sync(0xffffffffu, b[i], o);
+        }
+      }
+      if (sl == 0) {
+#pragma unroll
+        for (int i = 0; i < C; ++i) { A[i * C + jj] = a[i]; B[i * C + jj] = b[i]; }
       }
     }
   }
-  if (unit >= 2 * p.G + p.H) {  // the decays of one head's key channels
-    const int h = unit - 2 * p.G - p.H;
-    const float rate = -expf(ld_f<T>((const T*)p.A_log + h));
-    for (int d = threadIdx.x; d < p.D; d += blockDim.x) {
-      const int c = h * p.D + d;
-      p.decay[(size_t)m * p.H * p.D + c] = expm1f(rate * softplus_f(p.a[(size_t)m * p.ld_a + c] + ld_f<T>((const T*)p.dt_bias + c)));
+  __syncthreads();
+  if (tid < C) {                       // column tid of X: forward substitution, then the row's beta
+    float x[C];
+#pragma unroll
+    for (int i = 0; i < C; ++i) {
+      float acc = 0.f;
+#pragma unroll
+      for (int l = 0; l < C; ++l)
+        if (l < i) acc = fmaf(A[i * C + l], x[l], acc);
+      x[i] = i == tid ? 1.f : (i > tid ? -beta[i] * acc : 0.f);
     }
-    return;
+#pragma unroll
+    for (int i = 0; i < C; ++i) X[i * C + tid] = x[i] * beta[tid];
   }
-  if (unit >= 2 * p.G) {  // a value head: convolution and SiLU only
-    const int c0 = 2 * GD + (unit - 2 * p.G) * p.V;
-    for (int d = threadIdx.x; d < p.V; d += blockDim.x)
-      p.v[(size_t)m * HV + (size_t)(unit - 2 * p.G) * p.V + d] = silu_f(conv_at<T>(p.conv, rg, m, s, t, c0 + d));
-    return;
+  __syncthreads();
+  float* xo = rec + (3 * C + 1) * DP;
+  for (int x = tid; x < C * C; x += kThreads) {
+    const int i = x / C, jc = x % C;
+    float acc = 0.f;
+#pragma unroll
+    for (int l = 0; l < C; ++l) acc = fmaf(l <= i ? B[i * C + l] : 0.f, X[l * C + jc], acc);
+    xo[x] = X[x];
+    xo[C * C + x] = acc;
   }
-  const int c0 = unit * p.D;  // q heads, then k heads, in the order of the convolution's channels
-  float ss = 0.f;
-  for (int d = threadIdx.x; d < p.D; d += blockDim.x) {
-    const float v = silu_f(conv_at<T>(p.conv, rg, m, s, t, c0 + d));
-    dp_sm[d] = v;
-    ss = fmaf(v, v, ss);
-  }
-  ss = block_sum(ss, red);
-  const bool is_q = unit < p.G;
-  const float inv = (is_q ? p.q_scale : 1.0f) / sqrtf(ss + p.unit_eps);
-  float* dst = (is_q ? p.q : p.k) + (size_t)m * GD + (size_t)(is_q ? unit : unit - p.G) * p.D;
-  for (int d = threadIdx.x; d < p.D; d += blockDim.x) dst[d] = dp_sm[d] * inv;
 }
 
 struct DeltaArgs {
-  const float* q; const float* k;    // [M, G D]
+  const float* rec;                  // records of delta_chunk_prep_kernel
   const float* v;                    // [M, H V]
-  const float* beta;                 // [M, H]
-  const float* decay;                // g - 1: [M, H], or one per key channel [M, H D]
   float* o;                          // [M, H V]
   float* S; size_t slot_stride;      // [H, V, D] per slot: a column of the state (one value channel) is contiguous
-  int H, G, D, V;
-  int vec;                           // D, V, row offsets and the slot are whole 16-byte pieces
+  int H, D, V, DP;
+  int vec;                           // D and the slot's columns are whole 16-byte pieces
 };
 
-constexpr int kDeltaRows = 16;   // rows staged together (two such buffers: the next chunk arrives under the current one's walk)
+// two fp32 products and sums at once
+SSDK_DEVINL uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+SSDK_DEVINL uint64_t pack2(float x, float y) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(x), "f"(y));
+  return d;
+}
+SSDK_DEVINL void unpack2(uint64_t v, float* x, float* y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(*x), "=f"(*y) : "l"(v)); }
+
 constexpr int kDeltaWarps = 4;
+inline __host__ __device__ int delta_cols(int LC) { return kDeltaWarps * 64 / LC; }   // value columns of a CTA
+inline size_t delta_scan_smem(int DP, int LC, int C) { return (size_t)2 * (delta_record(DP, C) + C * delta_cols(LC)) * 4; }
 
-// floats of one staged row: k | q (| decay per channel), DP entries each, then value columns, beta, decay per head (padded to 4)
-inline __host__ __device__ int delta_row_floats(int DP, int cols, bool per_channel) {
-  return (per_channel ? 3 : 2) * DP + (cols + 2 + 3) / 4 * 4;
-}
-inline size_t delta_scan_smem(int DP, int cols, bool per_channel) {
-  return (size_t)2 * kDeltaRows * delta_row_floats(DP, cols, per_channel) * 4;
-}
-
-// The walk over a sequence's rows.  grid (n_seqs, H, ceil(V / cols)), kDeltaWarps warps, cols = kDeltaWarps * 32 / LC.
-// The columns of the state (value channels) are independent of one another: LC neighbouring lanes share one column, lane r
-// of them holds the key channels 4 (r + LC i) .. + 3, i < NQ, in registers (D <= 4 LC NQ; padded channels meet k = q = 0).
-// Both contractions over D (S^T k and S^T q) are thread-local sums followed by a shuffle tree over the LC lanes: no CTA
-// barrier inside a row.  Rows arrive by cp.async, sixteen at a time, under the walk of the previous sixteen.  CH: one decay
-// per key channel instead of one per head.  Everything is fp32 whatever the model's storage type.
-template <int LC, int NQ, bool CH>
-__global__ void __launch_bounds__(kDeltaWarps * 32) delta_scan_kernel(const DeltaArgs p, const Ragged rg) {
+// The walk over a sequence's chunks.  grid (n_seqs, H, ceil(V / delta_cols)), kDeltaWarps warps.  The columns of the state are
+// independent of one another: LC neighbouring lanes share TWO columns, lane r of them holds their key channels
+// 4 (r + LC i) .. + 3, i < NQ, in registers (DP = 4 LC NQ), so one load of a scaled key serves both.  Sums over D are
+// thread-local packed products followed by a shuffle tree over the LC lanes; C rows' trees run together.  The next chunk's
+// record arrives by cp.async under the current one's arithmetic.
+template <int LC, int NQ, int C>
+__global__ void __launch_bounds__(kDeltaWarps * 32) delta_chunk_scan_kernel(const DeltaArgs p, const Ragged rg) {
   extern __shared__ __align__(16) float ds_sm[];
-  constexpr int DP = 4 * LC * NQ, kCols = kDeltaWarps * 32 / LC, kR = kDeltaRows, kThreads = kDeltaWarps * 32;
-  const int RF = delta_row_floats(DP, kCols, CH), off_v = (CH ? 3 : 2) * DP, off_b = off_v + kCols;
-  const int s = blockIdx.x, hd = blockIdx.y, g = hd / (p.H / p.G), tid = threadIdx.x;
-  const int lr = tid % LC, jl = tid / LC, j = blockIdx.z * kCols + jl;
-  const int D = p.D, V = p.V, GD = p.G * D, HV = p.H * V, HDk = p.H * D;
-  const bool col = j < V, carried = rg.pos0[s] > 0;
-  float* Sg = p.S + (size_t)rg.slot[s] * p.slot_stride + ((size_t)hd * V + (col ? j : 0)) * D;
-  float4 S[NQ];
+  constexpr int DP = 4 * LC * NQ, kCols = kDeltaWarps * 64 / LC, kThreads = kDeltaWarps * 32, kVals = 2 * C;
+  constexpr int kRec = (3 * C + 1) * DP + (C > 1 ? 2 * C * C : 4), kBuf = kRec + C * kCols;
+  const int s = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x, lr = tid % LC, jl = 2 * (tid / LC), c0 = blockIdx.z * kCols, j = c0 + jl;
+  const int D = p.D, V = p.V, HV = p.H * V, vcols = min(kCols, V - c0);
+  const bool carried = rg.pos0[s] > 0;
+  float* Sg = p.S + (size_t)rg.slot[s] * p.slot_stride + ((size_t)hd * V + j) * D;
+  uint64_t S[2][NQ][2];
 #pragma unroll
-  for (int i = 0; i < NQ; ++i) {
-    const int d = 4 * (lr + LC * i);
-    S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (col && carried) {
-      if (p.vec) {
-        if (d < D) S[i] = *reinterpret_cast<const float4*>(Sg + d);
-      } else {
-        if (d < D) S[i].x = Sg[d];
-        if (d + 1 < D) S[i].y = Sg[d + 1];
-        if (d + 2 < D) S[i].z = Sg[d + 2];
-        if (d + 3 < D) S[i].w = Sg[d + 3];
+  for (int c = 0; c < 2; ++c)
+#pragma unroll
+    for (int i = 0; i < NQ; ++i) {
+      const int d = 4 * (lr + LC * i);
+      const float* src = Sg + (size_t)c * D;
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+      if (j + c < V && carried) {
+        if (p.vec) {
+          if (d < D) { const float4 f = *reinterpret_cast<const float4*>(src + d); x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w; }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (d + e < D) x[e] = src[d + e];
+        }
       }
+      S[c][i][0] = pack2(x[0], x[1]); S[c][i][1] = pack2(x[2], x[3]);
     }
-  }
-  // padding (channels from D up to DP, value columns beyond V) is zero in both buffers and never written again
-  for (int i = tid; i < 2 * kR * RF; i += kThreads) ds_sm[i] = 0.f;
+  for (int i = tid; i < 2 * kBuf; i += kThreads) ds_sm[i] = 0.f;   // value rows and columns outside the portion stay finite
   __syncthreads();
-  const int r0 = rg.cu[s], r1 = rg.cu[s + 1];
-  const int c0 = blockIdx.z * kCols, vcols = min(kCols, V - c0);
-  auto issue = [&](int m0, float* buf) {
-    const int nr = min(kR, r1 - m0);
-    if (p.vec) {
-      const int dq = D >> 2, per = (CH ? 3 : 2) * dq, vq = vcols >> 2;
-      for (int i = tid; i < nr * per; i += kThreads) {
-        const int r = i / per, x = i - r * per, part = x / dq, d = (x - part * dq) * 4;
-        const size_t m = m0 + r;
-        const float* src = part == 0 ? p.k + m * GD + g * D + d : part == 1 ? p.q + m * GD + g * D + d : p.decay + m * HDk + hd * D + d;
-        cp_async16(buf + r * RF + part * DP + d, src, true);
-      }
-      for (int i = tid; i < nr * vq; i += kThreads) {
-        const int r = i / vq, c = (i - r * vq) * 4;
-        cp_async16(buf + r * RF + off_v + c, p.v + (size_t)(m0 + r) * HV + hd * V + c0 + c, true);
-      }
-    } else {   // 4-byte copies: no alignment rule beyond the element's own
-      for (int i = tid; i < nr * D; i += kThreads) {
-        const int r = i / D, d = i - r * D;
-        const size_t m = m0 + r;
-        cp_async4(buf + r * RF + d, p.k + m * GD + g * D + d);
-        cp_async4(buf + r * RF + DP + d, p.q + m * GD + g * D + d);
-        if (CH) cp_async4(buf + r * RF + 2 * DP + d, p.decay + m * HDk + hd * D + d);
-      }
-      for (int i = tid; i < nr * vcols; i += kThreads) {
-        const int r = i / vcols, c = i - r * vcols;
-        cp_async4(buf + r * RF + off_v + c, p.v + (size_t)(m0 + r) * HV + hd * V + c0 + c);
-      }
-    }
-    if (tid < nr) {
-      cp_async4(buf + tid * RF + off_b, p.beta + (size_t)(m0 + tid) * p.H + hd);
-      if (!CH) cp_async4(buf + tid * RF + off_b + 1, p.decay + (size_t)(m0 + tid) * p.H + hd);
+  const int r0 = rg.cu[s], r1 = rg.cu[s + 1], n_chunks = (r1 - r0 + C - 1) / C;
+  const float* rec0 = p.rec + (delta_chunk_index(rg, s, 0, C) * p.H + hd) * kRec;
+  auto issue = [&](int ci, float* buf) {
+    const float* src = rec0 + (size_t)ci * p.H * kRec;
+    for (int i = tid; i < kRec / 4; i += kThreads) cp_async16(buf + 4 * i, src + 4 * i, true);
+    const int m0 = r0 + ci * C, nr = min(C, r1 - m0);
+    for (int i = tid; i < C * kCols; i += kThreads) {
+      const int r = i / kCols, c = i % kCols;
+      if (r < nr && c < vcols) cp_async4(buf + kRec + i, p.v + (size_t)(m0 + r) * HV + hd * V + c0 + c);
     }
     cp_async_commit();
   };
-  issue(r0, ds_sm);
-  int cur = 0;
-  for (int m0 = r0; m0 < r1; m0 += kR, cur ^= 1) {
-    const int nr = min(kR, r1 - m0);
-    if (m0 + kR < r1) {
-      issue(m0 + kR, ds_sm + (cur ^ 1) * kR * RF);
+  issue(0, ds_sm);
+  for (int ci = 0; ci < n_chunks; ++ci) {
+    if (ci + 1 < n_chunks) {
+      issue(ci + 1, ds_sm + ((ci + 1) & 1) * kBuf);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
     }
     __syncthreads();
-    const float* buf = ds_sm + cur * kR * RF;
-#pragma unroll 2
-    for (int r = 0; r < nr; ++r) {
-      const float* row = buf + r * RF;
-      const float4* k4 = reinterpret_cast<const float4*>(row) + lr;
-      const float beta = row[off_b], v = row[off_v + jl];
-      float dec = 0.f;
-      if (!CH) dec = row[off_b + 1];
-      float4 kk[NQ];
-      float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
+    const float* buf = ds_sm + (ci & 1) * kBuf;
+    const float* Xs = buf + (3 * C + 1) * DP;
+    const float* vs = buf + kRec + jl;
+    auto piece = [&](int row, int i) { return *reinterpret_cast<const ulonglong2*>(buf + row * DP + 4 * (lr + LC * i)); };
+    // row sums of the scaled keys and queries with the state before the chunk
+    float P[C][2], O[kVals];
 #pragma unroll
-      for (int i = 0; i < NQ; ++i) {
-        kk[i] = k4[LC * i];
-        const float4 gg = CH ? k4[DP / 2 + LC * i] : make_float4(dec, dec, dec, dec);
-        S[i].x = fmaf(S[i].x, gg.x, S[i].x); S[i].y = fmaf(S[i].y, gg.y, S[i].y);   // S g = S + S (g - 1), rounded once
-        S[i].z = fmaf(S[i].z, gg.z, S[i].z); S[i].w = fmaf(S[i].w, gg.w, S[i].w);
-        a0 = fmaf(S[i].x, kk[i].x, a0); a1 = fmaf(S[i].y, kk[i].y, a1);
-        a2 = fmaf(S[i].z, kk[i].z, a2); a3 = fmaf(S[i].w, kk[i].w, a3);
+    for (int i = 0; i < C; ++i) {
+      uint64_t a[2] = {0ull, 0ull}, b[2] = {0ull, 0ull};
+#pragma unroll
+      for (int x = 0; x < NQ; ++x) {
+        const ulonglong2 k = piece(i, x), q = piece(2 * C + i, x);
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          a[c] = fma2(S[c][x][0], k.x, a[c]); a[c] = fma2(S[c][x][1], k.y, a[c]);
+          b[c] = fma2(S[c][x][0], q.x, b[c]); b[c] = fma2(S[c][x][1], q.y, b[c]);
+        }
       }
-      float dot = (a0 + a1) + (a2 + a3);
 #pragma unroll
-      for (int o = LC >> 1; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-      const float u = beta * (v - dot);
-      a0 = a1 = a2 = a3 = 0.f;
-#pragma unroll
-      for (int i = 0; i < NQ; ++i) {
-        const float4 qq = k4[DP / 4 + LC * i];
-        S[i].x = fmaf(kk[i].x, u, S[i].x); S[i].y = fmaf(kk[i].y, u, S[i].y);
-        S[i].z = fmaf(kk[i].z, u, S[i].z); S[i].w = fmaf(kk[i].w, u, S[i].w);
-        a0 = fmaf(S[i].x, qq.x, a0); a1 = fmaf(S[i].y, qq.y, a1);
-        a2 = fmaf(S[i].z, qq.z, a2); a3 = fmaf(S[i].w, qq.w, a3);
+      for (int c = 0; c < 2; ++c) {
+        float lo, hi;
+        unpack2(a[c], &lo, &hi); P[i][c] = lo + hi;
+        unpack2(b[c], &lo, &hi); O[2 * i + c] = lo + hi;
       }
-      float o = (a0 + a1) + (a2 + a3);
+    }
 #pragma unroll
-      for (int x = LC >> 1; x > 0; x >>= 1) o += __shfl_xor_sync(0xffffffffu, o, x);
-      if (col && lr == 0) p.o[(size_t)(m0 + r) * HV + hd * V + j] = o;
+    for (int o = LC >> 1; o > 0; o >>= 1) {
+#pragma unroll
+      for (int i = 0; i < C; ++i)
+#pragma unroll
+        for (int c = 0; c < 2; ++c) P[i][c] += __shfl_xor_sync(0xffffffffu, P[i][c], o);
+    }
+    float r[C][2];
+#pragma unroll
+    for (int i = 0; i < C; ++i) { r[i][0] = vs[i * kCols] - P[i][0]; r[i][1] = vs[i * kCols + 1] - P[i][1]; }
+    // the state: decay of the whole chunk, then every row's write
+#pragma unroll
+    for (int x = 0; x < NQ; ++x) {
+      const ulonglong2 g = piece(3 * C, x);
+#pragma unroll
+      for (int c = 0; c < 2; ++c) { S[c][x][0] = fma2(S[c][x][0], g.x, S[c][x][0]); S[c][x][1] = fma2(S[c][x][1], g.y, S[c][x][1]); }
+    }
+#pragma unroll
+    for (int i = 0; i < C; ++i) {
+      float u0 = 0.f, u1 = 0.f;
+#pragma unroll
+      for (int l = 0; l <= i; ++l) { const float x = Xs[i * C + l]; u0 = fmaf(x, r[l][0], u0); u1 = fmaf(x, r[l][1], u1); }
+      const uint64_t uu[2] = {pack2(u0, u0), pack2(u1, u1)};
+#pragma unroll
+      for (int x = 0; x < NQ; ++x) {
+        const ulonglong2 k = piece(C + i, x);
+#pragma unroll
+        for (int c = 0; c < 2; ++c) { S[c][x][0] = fma2(k.x, uu[c], S[c][x][0]); S[c][x][1] = fma2(k.y, uu[c], S[c][x][1]); }
+      }
+    }
+    // the read-out: the lanes' parts are summed so that every lane ends with its own value(s), index 2 row + column
+    const int m0 = r0 + ci * C, nr = min(C, r1 - m0);
+    if constexpr (C == 1) {
+#pragma unroll
+      for (int o = LC >> 1; o > 0; o >>= 1) { O[0] += __shfl_xor_sync(0xffffffffu, O[0], o); O[1] += __shfl_xor_sync(0xffffffffu, O[1], o); }
+      if (lr < 2 && j + lr < V) p.o[(size_t)m0 * HV + hd * V + j + lr] = lr ? fmaf(Xs[1], r[0][1], O[1]) : fmaf(Xs[1], r[0][0], O[0]);
+    } else {
+      static_assert(C == 1 || 2 * C >= LC, "every lane ends with at least one value");
+#pragma unroll
+      for (int st = 0, n = C; st < (LC == 16 ? 4 : 3); ++st, n >>= 1) {
+        const int o = (LC >> 1) >> st;
+        const bool up = (lr & o) != 0;
+#pragma unroll
+        for (int t = 0; t < C; ++t)
+          if (t < n) {
+            const float send = up ? O[t] : O[t + n], keep = up ? O[t + n] : O[t];
+            O[t] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+          }
+      }
+      constexpr int kEach = kVals / LC;
+#pragma unroll
+      for (int t = 0; t < kEach; ++t) {
+        const int idx = lr * kEach + t, i = idx >> 1, c = idx & 1;
+        float acc = O[t];
+        const float4* bx = reinterpret_cast<const float4*>(Xs + C * C + i * C);
+#pragma unroll
+        for (int l = 0; l < C; l += 4) {
+          const float4 f = bx[l / 4];
+          acc = fmaf(f.x, c ? r[l][1] : r[l][0], acc); acc = fmaf(f.y, c ? r[l + 1][1] : r[l + 1][0], acc);
+          acc = fmaf(f.z, c ? r[l + 2][1] : r[l + 2][0], acc); acc = fmaf(f.w, c ? r[l + 3][1] : r[l + 3][0], acc);
+        }
+        if (i < nr && j + c < V) p.o[(size_t)(m0 + i) * HV + hd * V + j + c] = acc;
+      }
     }
     __syncthreads();  // every thread is done with this buffer before the chunk after next is copied into it
   }
-  if (col) {
 #pragma unroll
-    for (int i = 0; i < NQ; ++i) {
-      const int d = 4 * (lr + LC * i);
-      if (p.vec) {
-        if (d < D) *reinterpret_cast<float4*>(Sg + d) = S[i];
-      } else {
-        if (d < D) Sg[d] = S[i].x;
-        if (d + 1 < D) Sg[d + 1] = S[i].y;
-        if (d + 2 < D) Sg[d + 2] = S[i].z;
-        if (d + 3 < D) Sg[d + 3] = S[i].w;
+  for (int c = 0; c < 2; ++c)
+    if (j + c < V) {
+#pragma unroll
+      for (int i = 0; i < NQ; ++i) {
+        const int d = 4 * (lr + LC * i);
+        float* dst = Sg + (size_t)c * D;
+        float x[4];
+        unpack2(S[c][i][0], x, x + 1); unpack2(S[c][i][1], x + 2, x + 3);
+        if (p.vec) {
+          if (d < D) *reinterpret_cast<float4*>(dst + d) = make_float4(x[0], x[1], x[2], x[3]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (d + e < D) dst[d + e] = x[e];
+        }
       }
     }
-  }
 }
 
-// Any D: one thread per column, the column in shared memory ([D][blockDim], dynamic), operands read from global memory.
-// grid (n_seqs, H, ceil(V / blockDim))
-template <bool CH>
+// Any D: one thread per column, the column in shared memory ([D][blockDim], dynamic), records of single rows (C = 1) read from
+// global memory.  grid (n_seqs, H, ceil(V / blockDim))
 __global__ void delta_scan_any_kernel(const DeltaArgs p, const Ragged rg) {
   extern __shared__ __align__(16) float ds_sm[];
-  const int s = blockIdx.x, hd = blockIdx.y, g = hd / (p.H / p.G), jl = threadIdx.x, Vr = blockDim.x, j = blockIdx.z * Vr + jl;
-  const int D = p.D, V = p.V;
+  const int s = blockIdx.x, hd = blockIdx.y, jl = threadIdx.x, Vr = blockDim.x, j = blockIdx.z * Vr + jl;
+  const int D = p.D, V = p.V, DP = p.DP, kRec = delta_record(DP, 1);
   if (j >= V) return;
   float* Sg = p.S + (size_t)rg.slot[s] * p.slot_stride + ((size_t)hd * V + j) * D;
   const bool carried = rg.pos0[s] > 0;
   for (int d = 0; d < D; ++d) ds_sm[(size_t)d * Vr + jl] = carried ? Sg[d] : 0.f;
-  for (int m = rg.cu[s]; m < rg.cu[s + 1]; ++m) {
-    const float* k = p.k + (size_t)m * p.G * D + g * D;
-    const float* q = p.q + (size_t)m * p.G * D + g * D;
-    const float* gc = p.decay + (CH ? ((size_t)m * p.H + hd) * D : (size_t)m * p.H + hd);
+  for (int ci = 0; ci < rg.cu[s + 1] - rg.cu[s]; ++ci) {
+    const float* rec = p.rec + (delta_chunk_index(rg, s, ci, 1) * p.H + hd) * kRec;
+    const size_t at = ((size_t)(rg.cu[s] + ci) * p.H + hd) * V + j;
     float dot = 0.f, o = 0.f;
     for (int d = 0; d < D; ++d) {
-      const float so = ds_sm[(size_t)d * Vr + jl], sv = fmaf(so, gc[CH ? d : 0], so);
-      ds_sm[(size_t)d * Vr + jl] = sv;
-      dot = fmaf(sv, k[d], dot);
+      const float sv = ds_sm[(size_t)d * Vr + jl];
+      dot = fmaf(sv, rec[d], dot);
+      o = fmaf(sv, rec[2 * DP + d], o);
     }
-    const float u = p.beta[(size_t)m * p.H + hd] * (p.v[((size_t)m * p.H + hd) * V + j] - dot);
+    const float r = p.v[at] - dot, u = rec[4 * DP] * r;
     for (int d = 0; d < D; ++d) {
-      const float sv = fmaf(k[d], u, ds_sm[(size_t)d * Vr + jl]);
-      ds_sm[(size_t)d * Vr + jl] = sv;
-      o = fmaf(sv, q[d], o);
+      const float sv = ds_sm[(size_t)d * Vr + jl];
+      ds_sm[(size_t)d * Vr + jl] = fmaf(rec[DP + d], u, fmaf(sv, rec[3 * DP + d], sv));
     }
-    p.o[((size_t)m * p.H + hd) * V + j] = o;
+    p.o[at] = fmaf(rec[4 * DP + 1], r, o);
   }
   for (int d = 0; d < D; ++d) Sg[d] = ds_sm[(size_t)d * Vr + jl];
 }

@@ -54,6 +54,7 @@ struct ssdk_hyb_engine {
   int max_tiles = 0;
   // widths of the shared buffers (elements per row)
   int w_p0 = 0, w_p1 = 0, w_p2 = 0, w_t0 = 0, w_t1 = 0, w_e = 0, w_top = 0, w_ff2 = 0, w_ff = 0, w_sff2 = 0, w_sff = 0;
+  size_t delta_floats = 0; float* delta_rec = nullptr;   // chunk records of the delta rule
   bool any_wkv = false, any_pair = false, any_ffn = false;
   int* h_meta = nullptr;     // pinned staging of the step's integers
   // tcgen05 path of the dense bf16 products: TMA descriptors by (pointer, rows, K, box rows), split-K partials
@@ -80,19 +81,29 @@ struct ssdk_hyb_engine {
   bool smem_attr_done = false;
 };
 
-// delta rule: lanes per state column (LC) and 16-byte pieces per lane (NQ) of delta_scan_kernel, 4 LC NQ >= D; few columns in
-// flight spread each over more lanes.  LC = 0: no register form, the column lives in shared memory (delta_scan_any_kernel)
+// delta rule: lanes per pair of state columns (LC) and 16-byte pieces per lane and column (NQ) of delta_chunk_scan_kernel,
+// 4 LC NQ >= D; few columns in flight spread each over more lanes.  LC = 0: no register form, the column lives in shared
+// memory (delta_scan_any_kernel)
 static void delta_shape(int D, bool few, int* LC, int* NQ) {
   auto set = [&](int lc, int nq) { *LC = lc; *NQ = nq; };
-  if (D <= 16) set(4, 1);
-  else if (D <= 32) set(4, 2);
-  else if (D <= 64) few ? set(8, 2) : set(4, 4);
-  else if (D <= 128) few ? set(8, 4) : set(4, 8);
-  else if (D <= 256) set(8, 8);
+  if (D <= 32) set(8, 1);
+  else if (D <= 64) few ? set(16, 1) : set(8, 2);
+  else if (D <= 128) few ? set(16, 2) : set(8, 4);
+  else if (D <= 256) set(16, 4);
   else if (D <= 512) set(16, 8);
   else set(0, 0);
 }
 constexpr int kDeltaAnyCols = 32;  // columns per CTA of the shared-memory form
+// padded key size of a record, and the floats of all records of a call with `rows` rows in `seqs` sequences
+static int delta_padded(int D) {
+  int LC = 0, NQ = 0;
+  delta_shape(D, false, &LC, &NQ);
+  return LC ? 4 * LC * NQ : (D + 3) / 4 * 4;
+}
+static size_t delta_record_floats(int D, int H, size_t rows, size_t seqs) {
+  const int DP = delta_padded(D), C = D <= 512 ? ssdk::kDeltaChunk : 1;
+  return std::max((rows / C + seqs) * H * ssdk::delta_record(DP, C), 2 * std::min(rows, seqs) * H * ssdk::delta_record(DP, 1));
+}
 
 static int hyb_derive(ssdk_hyb_engine* e) {
   const ssdk_hyb_cfg& g = e->cfg;
@@ -186,7 +197,8 @@ static int hyb_derive(ssdk_hyb_engine* e) {
       up(e->w_p0, Ca + (c.pair_gate ? (long long)H * V : 0) + Cd + (c.d_gate_rank ? c.d_gate_rank : (long long)Hd * Vd) + Hd +
                       (c.d_decay_rank ? c.d_decay_rank : Hd));
       up(e->w_p1, std::max((long long)H * V, (long long)Hd * Vd));
-      up(e->w_p2, Cd + Hd + (c.d_decay_rank ? (long long)Hd * Dd : Hd) + (c.d_gate_rank ? (long long)Hd * Vd : 0));
+      up(e->w_p2, (long long)Hd * Vd + (c.d_decay_rank ? (long long)Hd * Dd : 0) + (c.d_gate_rank ? (long long)Hd * Vd : 0));
+      e->delta_floats = std::max(e->delta_floats, delta_record_floats(Dd, Hd, g.max_tokens, g.max_seqs));
       up(e->w_t0, (long long)H * V); up(e->w_t1, std::max((long long)Hd * Vd, (long long)c.d_decay_rank + c.d_gate_rank));
       up(e->w_qcat, (long long)H * D); up(e->w_key, (long long)G * D); up(e->w_kr, (long long)G * V); up(e->w_lh, H);
       e->any_pair = true;
@@ -261,6 +273,7 @@ static int64_t hyb_carve(ssdk_hyb_engine* e, uint8_t* base) {
   e->p0 = (float*)take(cap * e->w_p0 * 4);
   e->p1 = (float*)take(cap * e->w_p1 * 4);
   e->p2 = (float*)take(cap * e->w_p2 * 4);
+  e->delta_rec = (float*)take(e->delta_floats * 4);
   e->t0 = take(cap * e->w_t0 * es);
   e->t1 = take(cap * e->w_t1 * es);
   e->mix_out = (float*)take(cap * g.width * 4);
@@ -946,13 +959,9 @@ struct HybRun {
     ssdk::DeltaPrepArgs dp = {};
     dp.conv.in = e->p0 + o_dq; dp.conv.ld_in = Ntot; dp.conv.w = Lr.t[SSDK_HT_CONV_W].p; dp.conv.hist = st + (size_t)Hd * Dd * Vd;
     dp.conv.slot_stride = e->slot_floats; dp.conv.C = Cd; dp.conv.taps = taps;
-    dp.q = e->p2; dp.k = dp.q + (size_t)M * dGD; dp.v = dp.k + (size_t)M * dGD;
-    float* rest = dp.v + (size_t)M * dHV;          // (per-channel decays first: they stay on 16-byte boundaries)
-    float* dz = rest;
-    if (Ra) rest += (size_t)M * Hd * Dd;
-    float* gz = rest;
-    if (Rg) rest += (size_t)M * dHV;
-    dp.beta = rest; dp.decay = Ra ? dz : rest + (size_t)M * Hd;
+    dp.v = e->p2; dp.rec = e->delta_rec;
+    float* dz = dp.v + (size_t)M * dHV;                            // decay pre-activations [M, Hd Dd]
+    float* gz = dz + (Ra ? (size_t)M * Hd * Dd : 0);               // gate pre-activations [M, Hd Vd]
     dp.b = e->p0 + o_b; dp.ld_b = Ntot;
     if (Ra || Rg) {   // second halves of the low-rank projections
       const void *za = e->p0 + o_a, *zg = e->p0 + o_g1;
@@ -968,14 +977,12 @@ struct HybRun {
     }
     dp.a = Ra ? dz : e->p0 + o_a; dp.ld_a = Ra ? Hd * Dd : Ntot; dp.per_channel = Ra > 0;
     dp.A_log = Lr.t[SSDK_HT_DELTA_ALOG].p; dp.dt_bias = Lr.t[SSDK_HT_DELTA_DT_B].p;
-    dp.H = Hd; dp.G = Gd; dp.D = Dd; dp.V = Vd; dp.q_scale = 1.0f / sqrtf((float)Dd); dp.unit_eps = 1e-6f;
-    CKI(L.go(ssdk::delta_prep_kernel<T>, dim3(M, 2 * Gd + Hd + (Ra ? Hd : 0)), dim3(std::min(256, (std::max(Dd, Vd) + 31) / 32 * 32)),
-             (size_t)std::max(Dd, Vd) * 4, dp, rg));
-    if (taps > 1) CKI(L.go(ssdk::conv_state_kernel<T>, dim3(rg.n_seqs, (Cd + 255) / 256), dim3(256), 0, dp.conv, rg));
+    dp.H = Hd; dp.G = Gd; dp.D = Dd; dp.V = Vd; dp.DP = delta_padded(Dd); dp.q_scale = 1.0f / sqrtf((float)Dd); dp.unit_eps = 1e-6f;
     ssdk::DeltaArgs da;
-    da.q = dp.q; da.k = dp.k; da.v = dp.v; da.beta = dp.beta; da.decay = dp.decay; da.o = e->p1; da.S = st; da.slot_stride = e->slot_floats;
-    da.H = Hd; da.G = Gd; da.D = Dd; da.V = Vd; da.vec = Dd % 4 == 0 && Vd % 4 == 0;
-    CKI(Ra ? delta_scan<true>(da) : delta_scan<false>(da));
+    da.rec = e->delta_rec; da.v = dp.v; da.o = e->p1; da.S = st; da.slot_stride = e->slot_floats; da.H = Hd; da.D = Dd; da.V = Vd; da.DP = dp.DP;
+    da.vec = Dd % 4 == 0;
+    CKI(delta_rule(dp, da));
+    if (taps > 1) CKI(L.go(ssdk::conv_state_kernel<T>, dim3(rg.n_seqs, (Cd + 255) / 256), dim3(256), 0, dp.conv, rg));
     const dim3 ngrid(M, Hd), nblock(std::min(256, (Vd + 31) / 32 * 32));
     const float* gate = Rg ? gz : e->p0 + o_dg;
     const int ld_gate = Rg ? dHV : Ntot;
@@ -985,27 +992,36 @@ struct HybRun {
     return lin(e->t1, dHV, Lr.t[SSDK_HT_MIX_OUT].p, dHV, e->mix2, W, M, W, dHV);
   }
 
-  // the walk of the delta rule over this step's rows; CH: one decay per key channel
-  template <bool CH>
-  int delta_scan(const ssdk::DeltaArgs& da) {
-    // fewer columns than the machine's schedulers hold warps for at four lanes each: twice the lanes per column
-    const bool few = (long long)rg.n_seqs * da.H * da.V * 4 / 32 < 4LL * num_sms();
+  // the delta rule over this step's rows: state-independent products per chunk, then the walk
+  int delta_rule(const ssdk::DeltaPrepArgs& dp, const ssdk::DeltaArgs& da) {
+    int n_max = 0;
+    for (int s = 0; s < rg.n_seqs; ++s) n_max = std::max(n_max, h_cu[s + 1] - h_cu[s]);
+    // a warp walks 64 / LC columns: fewer warps than the machine's schedulers at eight lanes each take sixteen
+    const bool few = (long long)rg.n_seqs * da.H * da.V / 8 < 4LL * num_sms();
     int LC = 0, NQ = 0;
     delta_shape(da.D, few, &LC, &NQ);
+    const int C = n_max == 1 || LC == 0 ? 1 : ssdk::kDeltaChunk;
+    const dim3 pgrid((n_max + C - 1) / C, rg.n_seqs, da.H), pblock(128);
+    if (C == 1) CKI(L.go(ssdk::delta_chunk_prep_kernel<T, 1>, pgrid, pblock, ssdk::delta_prep_smem(da.D, 1), dp, rg));
+    else CKI(L.go(ssdk::delta_chunk_prep_kernel<T, ssdk::kDeltaChunk>, pgrid, pblock, ssdk::delta_prep_smem(da.D, C), dp, rg));
     if (LC == 0)
-      return L.go(ssdk::delta_scan_any_kernel<CH>, dim3(rg.n_seqs, da.H, (da.V + kDeltaAnyCols - 1) / kDeltaAnyCols), dim3(kDeltaAnyCols),
+      return L.go(ssdk::delta_scan_any_kernel, dim3(rg.n_seqs, da.H, (da.V + kDeltaAnyCols - 1) / kDeltaAnyCols), dim3(kDeltaAnyCols),
                   (size_t)da.D * kDeltaAnyCols * 4, da, rg);
-    const int cols = ssdk::kDeltaWarps * 32 / LC;
+    if (C == 1) return delta_walk<1>(da, LC, NQ);
+    return delta_walk<ssdk::kDeltaChunk>(da, LC, NQ);
+  }
+  template <int C>
+  int delta_walk(const ssdk::DeltaArgs& da, int LC, int NQ) {
+    const int cols = ssdk::delta_cols(LC);
     const dim3 grid(rg.n_seqs, da.H, (da.V + cols - 1) / cols), block(ssdk::kDeltaWarps * 32);
-    const size_t smem = ssdk::delta_scan_smem(4 * LC * NQ, cols, CH);
-    if (LC == 4 && NQ == 1) return L.go(ssdk::delta_scan_kernel<4, 1, CH>, grid, block, smem, da, rg);
-    if (LC == 4 && NQ == 2) return L.go(ssdk::delta_scan_kernel<4, 2, CH>, grid, block, smem, da, rg);
-    if (LC == 8 && NQ == 2) return L.go(ssdk::delta_scan_kernel<8, 2, CH>, grid, block, smem, da, rg);
-    if (LC == 4 && NQ == 4) return L.go(ssdk::delta_scan_kernel<4, 4, CH>, grid, block, smem, da, rg);
-    if (LC == 8 && NQ == 4) return L.go(ssdk::delta_scan_kernel<8, 4, CH>, grid, block, smem, da, rg);
-    if (LC == 4 && NQ == 8) return L.go(ssdk::delta_scan_kernel<4, 8, CH>, grid, block, smem, da, rg);
-    if (LC == 8 && NQ == 8) return L.go(ssdk::delta_scan_kernel<8, 8, CH>, grid, block, smem, da, rg);
-    return L.go(ssdk::delta_scan_kernel<16, 8, CH>, grid, block, smem, da, rg);
+    const size_t smem = ssdk::delta_scan_smem(da.DP, LC, C);
+    if (LC == 8 && NQ == 1) return L.go(ssdk::delta_chunk_scan_kernel<8, 1, C>, grid, block, smem, da, rg);
+    if (LC == 16 && NQ == 1) return L.go(ssdk::delta_chunk_scan_kernel<16, 1, C>, grid, block, smem, da, rg);
+    if (LC == 8 && NQ == 2) return L.go(ssdk::delta_chunk_scan_kernel<8, 2, C>, grid, block, smem, da, rg);
+    if (LC == 16 && NQ == 2) return L.go(ssdk::delta_chunk_scan_kernel<16, 2, C>, grid, block, smem, da, rg);
+    if (LC == 8 && NQ == 4) return L.go(ssdk::delta_chunk_scan_kernel<8, 4, C>, grid, block, smem, da, rg);
+    if (LC == 16 && NQ == 4) return L.go(ssdk::delta_chunk_scan_kernel<16, 4, C>, grid, block, smem, da, rg);
+    return L.go(ssdk::delta_chunk_scan_kernel<16, 8, C>, grid, block, smem, da, rg);
   }
 
   int run_mixer(HybLayer& Lr) {
@@ -1192,13 +1208,12 @@ static int hyb_smem_attrs(ssdk_hyb_engine* e) {
   CK(cudaFuncSetAttribute(ssdk::latent_decode_mma_kernel<5, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::latent_decode_mma_kernel<9, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
 #define SSDK_DELTA_ATTR(LC, NQ) \
-  CK(cudaFuncSetAttribute(ssdk::delta_scan_kernel<LC, NQ, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
-  CK(cudaFuncSetAttribute(ssdk::delta_scan_kernel<LC, NQ, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  SSDK_DELTA_ATTR(4, 1) SSDK_DELTA_ATTR(4, 2) SSDK_DELTA_ATTR(8, 2) SSDK_DELTA_ATTR(4, 4) SSDK_DELTA_ATTR(8, 4) SSDK_DELTA_ATTR(4, 8)
-  SSDK_DELTA_ATTR(8, 8) SSDK_DELTA_ATTR(16, 8)
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_scan_kernel<LC, NQ, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_scan_kernel<LC, NQ, ssdk::kDeltaChunk>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  SSDK_DELTA_ATTR(8, 1) SSDK_DELTA_ATTR(16, 1) SSDK_DELTA_ATTR(8, 2) SSDK_DELTA_ATTR(16, 2) SSDK_DELTA_ATTR(8, 4) SSDK_DELTA_ATTR(16, 4)
+  SSDK_DELTA_ATTR(16, 8)
 #undef SSDK_DELTA_ATTR
-  CK(cudaFuncSetAttribute(ssdk::delta_scan_any_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::delta_scan_any_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::delta_scan_any_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
 #define SSDK_STREAM_ATTR(SM, VEC) \
@@ -1208,8 +1223,10 @@ static int hyb_smem_attrs(ssdk_hyb_engine* e) {
 #undef SSDK_STREAM_ATTR
   CK(cudaFuncSetAttribute(ssdk::stream_norm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::stream_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::delta_prep_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::delta_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_prep_kernel<bf16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_prep_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_prep_kernel<bf16, ssdk::kDeltaChunk>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_prep_kernel<float, ssdk::kDeltaChunk>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   e->smem_attr_done = true;
   return 0;
 }

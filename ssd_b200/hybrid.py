@@ -506,7 +506,7 @@ def random_hybrid_weights(spec: HybridSpec, dtype: torch.dtype, device, seed: in
     def uni(lo, hi, *shape):
         return (lo + (hi - lo) * torch.rand(*shape, generator=g, device=device)).to(dtype)
 
-    if spec.block == L.BLOCK_SERIAL_POSTNORM:
+    if spec.block in (L.BLOCK_SERIAL_POSTNORM, L.BLOCK_SERIAL_PRENORM):
         w["FINAL_NORM"] = vec(W, 1.0)
     if spec.block == L.BLOCK_PARALLEL_ONE_NORM:
         w["FINAL_NORM"] = vec(W, 1.0)
@@ -593,13 +593,28 @@ def random_hybrid_weights(spec: HybridSpec, dtype: torch.dtype, device, seed: in
                 lw["SEL_ALOG"], lw["SEL_D"], lw["MIX_OUT"] = torch.log(uni(0.3, 4.0, I, N).float()).to(dtype), vec(I, 1.0, 0.2), lin(W, I)
             else:
                 G, Hd, Gd, Dd, Vd = ls.kv_heads, ls.d_heads, ls.d_kv_heads, ls.d_dim, ls.d_vdim
-                Cd = 2 * Gd * Dd + Hd * Vd
-                lw["PAIR_IN"] = lin(H * D + G * D + G * V + H * V + Cd + Hd * Vd + 2 * Hd, W)
+                Cd, Ca, Ra, Rg = 2 * Gd * Dd + Hd * Vd, H * D + G * (D + V), whole8(ls.d_decay_rank), whole8(ls.d_gate_rank)
+                lw["PAIR_IN"] = lin(Ca + (H * V if ls.pair_gate else 0) + Cd + (0 if Rg else Hd * Vd) + Hd + (Ra or Hd) + Rg, W)
                 lw["ATTN_OUT"], lw["MIX_OUT"] = lin(W, H * V), lin(W, Hd * Vd)
                 lw["CONV_W"] = (torch.randn(Cd, taps, generator=g, device=device) * 0.6).to(dtype)
-                lw["DELTA_ALOG"], lw["DELTA_DT_B"], lw["MIX_NORM"] = uni(-2.0, 0.5, Hd), uni(-2.0, 1.0, Hd), vec(Hd * Vd, 1.0)
+                lw["DELTA_ALOG"], lw["DELTA_DT_B"], lw["MIX_NORM"] = uni(-2.0, 0.5, Hd), uni(-2.0, 1.0, Hd * (Dd if Ra else 1)), vec(Hd * Vd, 1.0)
+                if Ra:
+                    lw["DELTA_A2"] = lin(Hd * Dd, Ra)
+                if Rg:
+                    lw["DELTA_G2"] = lin(Hd * Vd, Rg)
+                if ls.pair_conv:
+                    lw["ATTN_IN_B"] = vec(Ca, 0.0, 0.3)
+                    lw["ATTN_CONV_W"] = (torch.randn(Ca, ls.pair_conv, generator=g, device=device) * 0.5).to(dtype)
+                if ls.qk_norm == 2:
+                    lw["ATTN_QK_NORM"] = vec((H + G) * D, 1.0)
+                if ls.pair_norm:
+                    lw["PAIR_NORM"] = torch.stack([vec(W, 1.0), vec(W, 1.0)])
             if ls.mlp == "dense":
                 lw["NORM2"], lw["GLU_IN"], lw["GLU_OUT"] = vec(W, 1.0), lin(2 * ls.ff, W), lin(W, ls.ff)
+            if spec.streams:
+                n, S = 2 if ls.mlp else 1, spec.streams
+                lw["HC_IN"], lw["HC_OUT"] = vec(n * S, 1.0 / S, 0.1).view(n, S), vec(n * S, 1.0, 0.1).view(n, S)
+                lw["HC_MIX"] = (torch.eye(S, device=device) + 0.05 * torch.randn(n, S, S, generator=g, device=device)).to(dtype)
             w["layers"].append(lw)
             continue
         lw = {"NORM": vec(W), "LS_MIX": vec(W, 1.0), "MIX_OUT": lin(W, H * V)}

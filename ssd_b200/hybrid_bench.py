@@ -1,4 +1,4 @@
-"""Throughput of the hybrid families (bench.py --arch pikavik | kefurax | lisenex | kokatar).
+"""Throughput of the hybrid families (bench.py --arch pikavik | kefurax | lisenex | kokatar | vatolorn).
 
 --arch pikavik: a Pikavik stack beside the closest dense model of the framework (below).
 --arch kefurax: a Kefurax stack (attention + delta-rule pair with a dense feed-forward, selective scan, rglru, ...) beside
@@ -10,6 +10,10 @@ shared expert) beside the same Pikavik stack.
 attention with a learned sink and windowed latent attention without positions; a dense PolyNorm feed-forward or
 squared-relu experts with a gated shared expert) beside the closest existing model of the framework, a Lisenex stack of the
 same width, depth, vocabulary and feed-forward / expert sizes.
+--arch vatolorn: a Vatolorn stack (serial pre-norm blocks over four residual streams; chunked attention behind a convolution
+beside a delta rule with a decay per key channel; dense silu-GLU feed-forward) beside the closest existing model of the
+framework, a Kefurax stack whose every layer is the attention + delta-rule pair, of the same width, depth, vocabulary, head
+counts and sizes and feed-forward size.
 
 For every size: a Pikavik stack (mLSTM, wkv, wkv, latent attention, ... each with a grouped mixture of experts and a
 shared expert) with random weights, and a Llama stack of the same width, depth and ACTIVE feed-forward size
@@ -48,7 +52,27 @@ def pikavik_spec(z):
     return HybridSpec(z["width"], z["vocab"], 1e-6, layers)
 
 
-def kefurax_spec(z):
+def kefurax_pairs_spec(z):
+    """A Kefurax stack of attention + delta-rule pairs only."""
+    return kefurax_spec(z, ("parallel",))
+
+
+def vatolorn_spec(z, chunk=1024):
+    """Layers that resemble a real model's: attention with 128-wide heads, four query heads per key/value head, half of a head
+    rotated, 4 taps on q | k | v, chunks of `chunk` positions; a delta rule with 128 x 128 heads, two heads per query/key head,
+    4 taps, rank-128 decay and output-gate projections; four residual streams; the feed-forward of the Kefurax arm."""
+    from .hybrid import DESIGNS, HybridSpec, LayerSpec
+    d = DESIGNS["Vatolorn"]
+    W = z["width"]
+    heads, ff = W // 128, z["top"] * z["ff"] + z["sff"]
+    layers = [LayerSpec("parallel", heads, 128, 128, rot_dims=64, rot_base=10000.0, attn_scale=128 ** -0.5, kv_heads=max(1, heads // 4),
+                        yarn_factor=4.0, yarn_original=4096.0, yarn_fast=16.0, yarn_slow=2.0, pair_conv=4, chunk=chunk, conv=4,
+                        d_heads=heads, d_kv_heads=max(1, heads // 2), d_dim=128, d_vdim=128, d_decay_rank=128, d_gate_rank=128,
+                        mlp="dense", ff=ff, **d["pair"], **d["ffn"]) for _ in range(z["layers"])]
+    return HybridSpec(W, z["vocab"], 1e-6, layers, architecture="Vatolorn", streams=4, logit_scale=0.5)
+
+
+def kefurax_spec(z, kinds=("parallel", "mamba1", "rglru", "parallel")):
     """Layers that resemble a real model's: 128-wide heads, four query heads per key/value head, a delta rule with
     128 x 128 heads, a selective scan of twice the width with 16 states, a recurrence as wide as the model."""
     from .hybrid import DESIGNS, RGLRU_DECAY_MULT, HybridSpec, LayerSpec
@@ -56,7 +80,7 @@ def kefurax_spec(z):
     heads, ff = W // 128, z["top"] * z["ff"] + z["sff"]
     layers = []
     for i in range(z["layers"]):
-        kind = ("parallel", "mamba1", "rglru", "parallel")[i % 4]
+        kind = kinds[i % len(kinds)]
         if kind == "parallel":
             layers.append(LayerSpec("parallel", heads, 128, 128, rot_dims=64, rot_base=10000.0, attn_scale=128 ** -0.5,
                                     kv_heads=max(1, heads // 4), yarn_factor=4.0, yarn_original=4096.0,
@@ -265,7 +289,28 @@ def run_kokatar(args):
     return out
 
 
+def run_vatolorn(args):
+    out = {"metric": "prefill and decode tokens/s, Vatolorn beside Kefurax pairs at equal width / depth / head and feed-forward sizes",
+           "dtype": "bf16", "data": "synthetic (random weights, random token ids)", "n_gpus": 1, "steps": args.steps,
+           "warmup": args.warmup, "timing": "CUDA events around the public forward call, median; every pass streams the stack's "
+           "weights (> 126 MB L2 for size m; size s partly L2-resident, stated here)", "sizes": {}}
+    names = [args.hybrid_size] if args.hybrid_size != "all" else list(SIZES)
+    for name in names:
+        z = SIZES[name]
+        row = {"config": {k: z[k] for k in ("width", "layers", "vocab")}, "prompt": args.prompt_len_hybrid, "decode_batch": args.hybrid_batch,
+               "chunk": 1024, "streams": 4}
+        row["vatolorn"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, spec_fn=vatolorn_spec)
+        if not args.no_dense_arm:
+            row["kefurax_pairs"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, spec_fn=kefurax_pairs_spec)
+        if args.hybrid_fp32:
+            row["vatolorn_fp32"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, "float32", vatolorn_spec)
+        out["sizes"][name] = row
+    return out
+
+
 def run(args):
+    if getattr(args, "arch", "pikavik") == "vatolorn":
+        return run_vatolorn(args)
     if getattr(args, "arch", "pikavik") == "kokatar":
         return run_kokatar(args)
     if getattr(args, "arch", "pikavik") == "kefurax":
