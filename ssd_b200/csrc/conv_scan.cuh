@@ -594,26 +594,26 @@ SSDK_DEVINL uint64_t pack2(float x, float y) {
 SSDK_DEVINL void unpack2(uint64_t v, float* x, float* y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(*x), "=f"(*y) : "l"(v)); }
 
 constexpr int kDeltaWarps = 4;
-inline __host__ __device__ int delta_cols(int LC) { return kDeltaWarps * 64 / LC; }   // value columns of a CTA
-inline size_t delta_scan_smem(int DP, int LC, int C) { return (size_t)2 * (delta_record(DP, C) + C * delta_cols(LC)) * 4; }
+inline __host__ __device__ int delta_cols(int LC, int NC) { return kDeltaWarps * 32 / LC * NC; }   // value columns of a CTA
+inline size_t delta_scan_smem(int DP, int LC, int NC, int C) { return (size_t)2 * (delta_record(DP, C) + C * delta_cols(LC, NC)) * 4; }
 
 // The walk over a sequence's chunks.  grid (n_seqs, H, ceil(V / delta_cols)), kDeltaWarps warps.  The columns of the state are
-// independent of one another: LC neighbouring lanes share TWO columns, lane r of them holds their key channels
-// 4 (r + LC i) .. + 3, i < NQ, in registers (DP = 4 LC NQ), so one load of a scaled key serves both.  Sums over D are
+// independent of one another: LC neighbouring lanes share NC columns (1 or 2), lane r of them holds their key
+// channels 4 (r + LC i) .. + 3, i < NQ, in registers (DP = 4 LC NQ); with two columns one load of a scaled key serves both.  Sums over D are
 // thread-local packed products followed by a shuffle tree over the LC lanes; C rows' trees run together.  The next chunk's
 // record arrives by cp.async under the current one's arithmetic.
-template <int LC, int NQ, int C>
-__global__ void __launch_bounds__(kDeltaWarps * 32) delta_chunk_scan_kernel(const DeltaArgs p, const Ragged rg) {
+template <int LC, int NQ, int NC, int C>
+__global__ void __launch_bounds__(kDeltaWarps * 32, 1) delta_chunk_scan_kernel(const DeltaArgs p, const Ragged rg) {
   extern __shared__ __align__(16) float ds_sm[];
-  constexpr int DP = 4 * LC * NQ, kCols = kDeltaWarps * 64 / LC, kThreads = kDeltaWarps * 32, kVals = 2 * C;
+  constexpr int DP = 4 * LC * NQ, kCols = kDeltaWarps * 32 / LC * NC, kThreads = kDeltaWarps * 32, kVals = NC * C;
   constexpr int kRec = (3 * C + 1) * DP + (C > 1 ? 2 * C * C : 4), kBuf = kRec + C * kCols;
-  const int s = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x, lr = tid % LC, jl = 2 * (tid / LC), c0 = blockIdx.z * kCols, j = c0 + jl;
+  const int s = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x, lr = tid % LC, jl = NC * (tid / LC), c0 = blockIdx.z * kCols, j = c0 + jl;
   const int D = p.D, V = p.V, HV = p.H * V, vcols = min(kCols, V - c0);
   const bool carried = rg.pos0[s] > 0;
   float* Sg = p.S + (size_t)rg.slot[s] * p.slot_stride + ((size_t)hd * V + j) * D;
-  uint64_t S[2][NQ][2];
+  uint64_t S[NC][NQ][2];
 #pragma unroll
-  for (int c = 0; c < 2; ++c)
+  for (int c = 0; c < NC; ++c)
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
       const int d = 4 * (lr + LC * i);
@@ -656,96 +656,130 @@ __global__ void __launch_bounds__(kDeltaWarps * 32) delta_chunk_scan_kernel(cons
     const float* buf = ds_sm + (ci & 1) * kBuf;
     const float* Xs = buf + (3 * C + 1) * DP;
     const float* vs = buf + kRec + jl;
-    auto piece = [&](int row, int i) { return *reinterpret_cast<const ulonglong2*>(buf + row * DP + 4 * (lr + LC * i)); };
-    // row sums of the scaled keys and queries with the state before the chunk
-    float P[C][2], O[kVals];
+    // 16-byte pieces of a record row.  All pieces of a phase are requested together and ahead of the arithmetic before it (the
+    // walk is bound by the latency of shared memory and of the exchanges, not by their number): kAll keeps a phase in registers
+    const uint32_t at = smem_u32(buf) + 16u * lr;
+    constexpr bool kAll = NQ * C <= 16;
+    constexpr int kAhead = kAll ? C : (NQ <= 4 && C >= 4 ? 4 : 1);   // rows requested together
+    typedef ulonglong2 Rows[kAhead][NQ];
+    auto fetch = [&](int row0, Rows& k) {
 #pragma unroll
-    for (int i = 0; i < C; ++i) {
-      uint64_t a[2] = {0ull, 0ull}, b[2] = {0ull, 0ull};
+      for (int i = 0; i < kAhead; ++i)
 #pragma unroll
-      for (int x = 0; x < NQ; ++x) {
-        const ulonglong2 k = piece(i, x), q = piece(2 * C + i, x);
+        for (int x = 0; x < NQ; ++x)
+          asm volatile("ld.shared.v2.u64 {%0, %1}, [%2];" : "=l"(k[i][x].x), "=l"(k[i][x].y) : "r"(at + (uint32_t)((row0 + i) * DP + 4 * LC * x) * 4u) : "memory");
+    };
+    float P[C][NC], O[kVals];
+    auto sums = [&](const Rows& k, int i0, auto put) {   // products of the fetched rows with the state before the chunk
 #pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          a[c] = fma2(S[c][x][0], k.x, a[c]); a[c] = fma2(S[c][x][1], k.y, a[c]);
-          b[c] = fma2(S[c][x][0], q.x, b[c]); b[c] = fma2(S[c][x][1], q.y, b[c]);
+      for (int i = 0; i < kAhead; ++i) {
+        uint64_t a[NC] = {};
+#pragma unroll
+        for (int x = 0; x < NQ; ++x)
+#pragma unroll
+          for (int c = 0; c < NC; ++c) { a[c] = fma2(S[c][x][0], k[i][x].x, a[c]); a[c] = fma2(S[c][x][1], k[i][x].y, a[c]); }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          float lo, hi;
+          unpack2(a[c], &lo, &hi);
+          put(i0 + i, c, lo + hi);
         }
       }
+    };
+    auto put_p = [&](int i, int c, float v) { P[i][c] = v; };
+    auto put_o = [&](int i, int c, float v) { O[NC * i + c] = v; };
+    Rows kr;
+    if constexpr (kAll) {
+      Rows kg, qg;
+      fetch(0, kg);
+      fetch(2 * C, qg);
+      sums(kg, 0, put_p);
+      fetch(C, kr);
+      sums(qg, 0, put_o);
+    } else {
 #pragma unroll
-      for (int c = 0; c < 2; ++c) {
-        float lo, hi;
-        unpack2(a[c], &lo, &hi); P[i][c] = lo + hi;
-        unpack2(b[c], &lo, &hi); O[2 * i + c] = lo + hi;
-      }
+      for (int i0 = 0; i0 < C; i0 += kAhead) { fetch(i0, kr); sums(kr, i0, put_p); }
+#pragma unroll
+      for (int i0 = 0; i0 < C; i0 += kAhead) { fetch(2 * C + i0, kr); sums(kr, i0, put_o); }
+      fetch(C, kr);
     }
+    float xr[C][(C + 3) / 4 * 4];
+#pragma unroll
+    for (int i = 0; i < C; ++i)
+#pragma unroll
+      for (int l = 0; l <= i; l += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(Xs + i * C + l);
+        xr[i][l] = f.x; xr[i][l + 1] = f.y; xr[i][l + 2] = f.z; xr[i][l + 3] = f.w;
+      }
 #pragma unroll
     for (int o = LC >> 1; o > 0; o >>= 1) {
+      float t[C][NC];   // all exchanges of a step are in flight together
 #pragma unroll
       for (int i = 0; i < C; ++i)
 #pragma unroll
-        for (int c = 0; c < 2; ++c) P[i][c] += __shfl_xor_sync(0xffffffffu, P[i][c], o);
-    }
-    float r[C][2];
+        for (int c = 0; c < NC; ++c) t[i][c] = __shfl_xor_sync(0xffffffffu, P[i][c], o);
 #pragma unroll
-    for (int i = 0; i < C; ++i) { r[i][0] = vs[i * kCols] - P[i][0]; r[i][1] = vs[i * kCols + 1] - P[i][1]; }
-    // the state: decay of the whole chunk, then every row's write
+      for (int i = 0; i < C; ++i)
+#pragma unroll
+        for (int c = 0; c < NC; ++c) P[i][c] += t[i][c];
+    }
+    float r[C][NC];
+#pragma unroll
+    for (int i = 0; i < C; ++i)
+#pragma unroll
+      for (int c = 0; c < NC; ++c) r[i][c] = vs[i * kCols + c] - P[i][c];
+    // the state: decay of the whole chunk, then every row's write u_i = sum_l X_il r_l
 #pragma unroll
     for (int x = 0; x < NQ; ++x) {
-      const ulonglong2 g = piece(3 * C, x);
+      const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(buf + 3 * C * DP + 4 * (lr + LC * x));
 #pragma unroll
-      for (int c = 0; c < 2; ++c) { S[c][x][0] = fma2(S[c][x][0], g.x, S[c][x][0]); S[c][x][1] = fma2(S[c][x][1], g.y, S[c][x][1]); }
+      for (int c = 0; c < NC; ++c) { S[c][x][0] = fma2(S[c][x][0], g.x, S[c][x][0]); S[c][x][1] = fma2(S[c][x][1], g.y, S[c][x][1]); }
     }
 #pragma unroll
-    for (int i = 0; i < C; ++i) {
-      float u0 = 0.f, u1 = 0.f;
+    for (int i0 = 0; i0 < C; i0 += kAhead) {
+      if (i0 > 0) fetch(C + i0, kr);
 #pragma unroll
-      for (int l = 0; l <= i; ++l) { const float x = Xs[i * C + l]; u0 = fmaf(x, r[l][0], u0); u1 = fmaf(x, r[l][1], u1); }
-      const uint64_t uu[2] = {pack2(u0, u0), pack2(u1, u1)};
+      for (int i = 0; i < kAhead; ++i) {
 #pragma unroll
-      for (int x = 0; x < NQ; ++x) {
-        const ulonglong2 k = piece(C + i, x);
+        for (int c = 0; c < NC; ++c) {
+          float u = 0.f;
 #pragma unroll
-        for (int c = 0; c < 2; ++c) { S[c][x][0] = fma2(k.x, uu[c], S[c][x][0]); S[c][x][1] = fma2(k.y, uu[c], S[c][x][1]); }
-      }
-    }
-    // the read-out: the lanes' parts are summed so that every lane ends with its own value(s), index 2 row + column
-    const int m0 = r0 + ci * C, nr = min(C, r1 - m0);
-    if constexpr (C == 1) {
+          for (int l = 0; l <= i0 + i; ++l) u = fmaf(xr[i0 + i][l], r[l][c], u);
+          const uint64_t uu = pack2(u, u);
 #pragma unroll
-      for (int o = LC >> 1; o > 0; o >>= 1) { O[0] += __shfl_xor_sync(0xffffffffu, O[0], o); O[1] += __shfl_xor_sync(0xffffffffu, O[1], o); }
-      if (lr < 2 && j + lr < V) p.o[(size_t)m0 * HV + hd * V + j + lr] = lr ? fmaf(Xs[1], r[0][1], O[1]) : fmaf(Xs[1], r[0][0], O[0]);
-    } else {
-      static_assert(C == 1 || 2 * C >= LC, "every lane ends with at least one value");
-#pragma unroll
-      for (int st = 0, n = C; st < (LC == 16 ? 4 : 3); ++st, n >>= 1) {
-        const int o = (LC >> 1) >> st;
-        const bool up = (lr & o) != 0;
-#pragma unroll
-        for (int t = 0; t < C; ++t)
-          if (t < n) {
-            const float send = up ? O[t] : O[t + n], keep = up ? O[t + n] : O[t];
-            O[t] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-          }
-      }
-      constexpr int kEach = kVals / LC;
-#pragma unroll
-      for (int t = 0; t < kEach; ++t) {
-        const int idx = lr * kEach + t, i = idx >> 1, c = idx & 1;
-        float acc = O[t];
-        const float4* bx = reinterpret_cast<const float4*>(Xs + C * C + i * C);
-#pragma unroll
-        for (int l = 0; l < C; l += 4) {
-          const float4 f = bx[l / 4];
-          acc = fmaf(f.x, c ? r[l][1] : r[l][0], acc); acc = fmaf(f.y, c ? r[l + 1][1] : r[l + 1][0], acc);
-          acc = fmaf(f.z, c ? r[l + 2][1] : r[l + 2][0], acc); acc = fmaf(f.w, c ? r[l + 3][1] : r[l + 3][0], acc);
+          for (int x = 0; x < NQ; ++x) { S[c][x][0] = fma2(kr[i][x].x, uu, S[c][x][0]); S[c][x][1] = fma2(kr[i][x].y, uu, S[c][x][1]); }
         }
-        if (i < nr && j + c < V) p.o[(size_t)(m0 + i) * HV + hd * V + j + c] = acc;
       }
+    }
+    // the read-out: the lanes' parts are summed so that a lane ends with its own value(s), index NC row + column (lanes share one
+    // when there are fewer values than lanes)
+    const int m0 = r0 + ci * C, nr = min(C, r1 - m0);
+#pragma unroll
+    for (int o = LC >> 1, n = kVals >> 1; o > 0; o >>= 1, n >>= 1) {
+      const bool up = (lr & o) != 0;
+      float got[kVals];
+#pragma unroll
+      for (int x = 0; x < kVals; ++x)
+        if (x < n) got[x] = __shfl_xor_sync(0xffffffffu, up ? O[x] : O[x + n], o);
+        else if (n == 0 && x == 0) got[0] = __shfl_xor_sync(0xffffffffu, O[0], o);
+#pragma unroll
+      for (int x = 0; x < kVals; ++x)
+        if (x < n) O[x] = (up ? O[x + n] : O[x]) + got[x];
+        else if (n == 0 && x == 0) O[0] += got[0];
+    }
+    constexpr int kEach = kVals > LC ? kVals / LC : 1, kShare = kVals < LC ? LC / kVals : 1;
+#pragma unroll
+    for (int x = 0; x < kEach; ++x) {
+      const int idx = lr / kShare * kEach + x, i = idx / NC, c = idx % NC;
+      float acc = O[x];
+#pragma unroll
+      for (int l = 0; l < C; ++l) acc = fmaf(Xs[(C > 1 ? C * C : 1) + i * C + l], NC == 2 && c ? r[l][NC - 1] : r[l][0], acc);
+      if (lr % kShare == 0 && i < nr && j + c < V) p.o[(size_t)(m0 + i) * HV + hd * V + j + c] = acc;
     }
     __syncthreads();  // every thread is done with this buffer before the chunk after next is copied into it
   }
 #pragma unroll
-  for (int c = 0; c < 2; ++c)
+  for (int c = 0; c < NC; ++c)
     if (j + c < V) {
 #pragma unroll
       for (int i = 0; i < NQ; ++i) {

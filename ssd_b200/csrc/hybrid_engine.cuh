@@ -996,8 +996,10 @@ struct HybRun {
   int delta_rule(const ssdk::DeltaPrepArgs& dp, const ssdk::DeltaArgs& da) {
     int n_max = 0;
     for (int s = 0; s < rg.n_seqs; ++s) n_max = std::max(n_max, h_cu[s + 1] - h_cu[s]);
-    // a warp walks 64 / LC columns: fewer warps than the machine's schedulers at eight lanes each take sixteen
-    const bool few = (long long)rg.n_seqs * da.H * da.V / 8 < 4LL * num_sms();
+    // a warp walks 32 NC / LC columns.  Sixteen lanes share one column, then two, while every warp still finds a scheduler of its
+    // own (a second one doubles the walk's latency more than it saves); beyond, eight lanes share two
+    const long long cols = (long long)rg.n_seqs * da.H * da.V, schedulers = 4LL * num_sms();
+    const bool one = cols / 2 <= schedulers, few = cols / 4 <= 2 * schedulers;
     int LC = 0, NQ = 0;
     delta_shape(da.D, few, &LC, &NQ);
     const int C = n_max == 1 || LC == 0 ? 1 : ssdk::kDeltaChunk;
@@ -1007,21 +1009,21 @@ struct HybRun {
     if (LC == 0)
       return L.go(ssdk::delta_scan_any_kernel, dim3(rg.n_seqs, da.H, (da.V + kDeltaAnyCols - 1) / kDeltaAnyCols), dim3(kDeltaAnyCols),
                   (size_t)da.D * kDeltaAnyCols * 4, da, rg);
-    if (C == 1) return delta_walk<1>(da, LC, NQ);
-    return delta_walk<ssdk::kDeltaChunk>(da, LC, NQ);
+    if (C == 1) return delta_walk<1, 2>(da, LC, NQ);
+    return one ? delta_walk<ssdk::kDeltaChunk, 1>(da, LC, NQ) : delta_walk<ssdk::kDeltaChunk, 2>(da, LC, NQ);
   }
-  template <int C>
+  template <int C, int NC>
   int delta_walk(const ssdk::DeltaArgs& da, int LC, int NQ) {
-    const int cols = ssdk::delta_cols(LC);
+    const int cols = ssdk::delta_cols(LC, NC);
     const dim3 grid(rg.n_seqs, da.H, (da.V + cols - 1) / cols), block(ssdk::kDeltaWarps * 32);
-    const size_t smem = ssdk::delta_scan_smem(da.DP, LC, C);
-    if (LC == 8 && NQ == 1) return L.go(ssdk::delta_chunk_scan_kernel<8, 1, C>, grid, block, smem, da, rg);
-    if (LC == 16 && NQ == 1) return L.go(ssdk::delta_chunk_scan_kernel<16, 1, C>, grid, block, smem, da, rg);
-    if (LC == 8 && NQ == 2) return L.go(ssdk::delta_chunk_scan_kernel<8, 2, C>, grid, block, smem, da, rg);
-    if (LC == 16 && NQ == 2) return L.go(ssdk::delta_chunk_scan_kernel<16, 2, C>, grid, block, smem, da, rg);
-    if (LC == 8 && NQ == 4) return L.go(ssdk::delta_chunk_scan_kernel<8, 4, C>, grid, block, smem, da, rg);
-    if (LC == 16 && NQ == 4) return L.go(ssdk::delta_chunk_scan_kernel<16, 4, C>, grid, block, smem, da, rg);
-    return L.go(ssdk::delta_chunk_scan_kernel<16, 8, C>, grid, block, smem, da, rg);
+    const size_t smem = ssdk::delta_scan_smem(da.DP, LC, NC, C);
+    if (LC == 8 && NQ == 1) return L.go(ssdk::delta_chunk_scan_kernel<8, 1, NC, C>, grid, block, smem, da, rg);
+    if (LC == 16 && NQ == 1) return L.go(ssdk::delta_chunk_scan_kernel<16, 1, NC, C>, grid, block, smem, da, rg);
+    if (LC == 8 && NQ == 2) return L.go(ssdk::delta_chunk_scan_kernel<8, 2, NC, C>, grid, block, smem, da, rg);
+    if (LC == 16 && NQ == 2) return L.go(ssdk::delta_chunk_scan_kernel<16, 2, NC, C>, grid, block, smem, da, rg);
+    if (LC == 8 && NQ == 4) return L.go(ssdk::delta_chunk_scan_kernel<8, 4, NC, C>, grid, block, smem, da, rg);
+    if (LC == 16 && NQ == 4) return L.go(ssdk::delta_chunk_scan_kernel<16, 4, NC, C>, grid, block, smem, da, rg);
+    return L.go(ssdk::delta_chunk_scan_kernel<16, 8, NC, C>, grid, block, smem, da, rg);
   }
 
   int run_mixer(HybLayer& Lr) {
@@ -1208,8 +1210,9 @@ static int hyb_smem_attrs(ssdk_hyb_engine* e) {
   CK(cudaFuncSetAttribute(ssdk::latent_decode_mma_kernel<5, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   CK(cudaFuncSetAttribute(ssdk::latent_decode_mma_kernel<9, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
 #define SSDK_DELTA_ATTR(LC, NQ) \
-  CK(cudaFuncSetAttribute(ssdk::delta_chunk_scan_kernel<LC, NQ, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
-  CK(cudaFuncSetAttribute(ssdk::delta_chunk_scan_kernel<LC, NQ, ssdk::kDeltaChunk>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_scan_kernel<LC, NQ, 2, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_scan_kernel<LC, NQ, 1, ssdk::kDeltaChunk>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::delta_chunk_scan_kernel<LC, NQ, 2, ssdk::kDeltaChunk>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   SSDK_DELTA_ATTR(8, 1) SSDK_DELTA_ATTR(16, 1) SSDK_DELTA_ATTR(8, 2) SSDK_DELTA_ATTR(16, 2) SSDK_DELTA_ATTR(8, 4) SSDK_DELTA_ATTR(16, 4)
   SSDK_DELTA_ATTR(16, 8)
 #undef SSDK_DELTA_ATTR
