@@ -472,6 +472,7 @@ def main():
     ap.add_argument("--hybrid-size", default="all", choices=["all", "s", "m"])
     ap.add_argument("--prompt-len-hybrid", type=int, default=2048)
     ap.add_argument("--hybrid-batch", type=int, default=8)
+    ap.add_argument("--hybrid-chunk", type=int, default=4096, help="vatolorn: positions per attention chunk")
     ap.add_argument("--hybrid-fp32", action="store_true", help="also time the float32 storage mode")
     ap.add_argument("--no-dense-arm", action="store_true")
     args = ap.parse_args()

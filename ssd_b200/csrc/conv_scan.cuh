@@ -383,7 +383,7 @@ __global__ void selective_scan_kernel(const SelScanArgs p, const Ragged rg) {
 inline __host__ __device__ int delta_record(int DP, int C) { return (3 * C + 1) * DP + (C > 1 ? 2 * C * C : 4); }
 
 constexpr int kDeltaChunk = 8;   // rows of a chunk (1 in calls that bring one row per sequence)
-constexpr int kDeltaTaps = 8;    // convolutions up to this length keep their rows in registers
+constexpr int kDeltaTaps = 4;    // convolutions up to this length keep their rows in registers
 
 struct DeltaPrepArgs {
   ConvArgs conv;          // over the q | k | v columns (C = 2 G D + H V); out / out_t unused

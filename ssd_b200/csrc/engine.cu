@@ -176,19 +176,19 @@ static int launch_gemm_inst(Launcher& L, const CUtensorMap& tmW, const CUtensorM
     CK(cudaFuncSetAttribute(gemm_ws_kernel<UN, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
     attr_set = true;
   }
-  if (row_chunks > 1 && EPI != EPI_PARTIAL) return fail("row chunks are an EPI_PARTIAL feature");
+  if (row_chunks > 1 && EPI != EPI_PARTIAL && EPI != EPI_GLU) return fail("row chunks are a feature of EPI_PARTIAL and EPI_GLU");
   return L.go(gemm_ws_kernel<UN, EPI>, dim3(tiles, splits, row_chunks), dim3(kGemmThreads), (size_t)Cfg::kSmemBytes, tmW, tmX, p);
 }
-// row_chunks > 1 (EPI_PARTIAL): p.M rows in chunks of umma_n along gridDim.z, tmX covering all of them
+// row_chunks > 1 (EPI_PARTIAL, EPI_GLU): p.M rows in chunks of umma_n along gridDim.z, tmX covering all of them
 static int launch_gemm(Launcher& L, int umma_n, int epi, const CUtensorMap& tmW, const CUtensorMap& tmX,
                        const GemmParams& p, int tiles, int splits, int row_chunks = 1) {
 #define SSDK_GEMM_CASE(UN, EP) \
   if (umma_n == UN && epi == EP) return launch_gemm_inst<UN, EP>(L, tmW, tmX, p, tiles, splits, row_chunks);
-  SSDK_GEMM_CASE(16, EPI_BF16) SSDK_GEMM_CASE(16, EPI_PARTIAL) SSDK_GEMM_CASE(16, EPI_SILU) SSDK_GEMM_CASE(16, EPI_PUBLISH)
-  SSDK_GEMM_CASE(32, EPI_BF16) SSDK_GEMM_CASE(32, EPI_PARTIAL) SSDK_GEMM_CASE(32, EPI_SILU) SSDK_GEMM_CASE(32, EPI_PUBLISH)
-  SSDK_GEMM_CASE(64, EPI_BF16) SSDK_GEMM_CASE(64, EPI_PARTIAL) SSDK_GEMM_CASE(64, EPI_SILU) SSDK_GEMM_CASE(64, EPI_PUBLISH)
-  SSDK_GEMM_CASE(128, EPI_BF16) SSDK_GEMM_CASE(128, EPI_PARTIAL) SSDK_GEMM_CASE(128, EPI_SILU)
-  SSDK_GEMM_CASE(256, EPI_BF16) SSDK_GEMM_CASE(256, EPI_PARTIAL) SSDK_GEMM_CASE(256, EPI_SILU)
+  SSDK_GEMM_CASE(16, EPI_BF16) SSDK_GEMM_CASE(16, EPI_PARTIAL) SSDK_GEMM_CASE(16, EPI_SILU) SSDK_GEMM_CASE(16, EPI_GLU) SSDK_GEMM_CASE(16, EPI_PUBLISH)
+  SSDK_GEMM_CASE(32, EPI_BF16) SSDK_GEMM_CASE(32, EPI_PARTIAL) SSDK_GEMM_CASE(32, EPI_SILU) SSDK_GEMM_CASE(32, EPI_GLU) SSDK_GEMM_CASE(32, EPI_PUBLISH)
+  SSDK_GEMM_CASE(64, EPI_BF16) SSDK_GEMM_CASE(64, EPI_PARTIAL) SSDK_GEMM_CASE(64, EPI_SILU) SSDK_GEMM_CASE(64, EPI_GLU) SSDK_GEMM_CASE(64, EPI_PUBLISH)
+  SSDK_GEMM_CASE(128, EPI_BF16) SSDK_GEMM_CASE(128, EPI_PARTIAL) SSDK_GEMM_CASE(128, EPI_SILU) SSDK_GEMM_CASE(128, EPI_GLU)
+  SSDK_GEMM_CASE(256, EPI_BF16) SSDK_GEMM_CASE(256, EPI_PARTIAL) SSDK_GEMM_CASE(256, EPI_SILU) SSDK_GEMM_CASE(256, EPI_GLU)
 #undef SSDK_GEMM_CASE
   return fail("no GEMM instance for umma_n=%d epi=%d", umma_n, epi);
 }
@@ -1081,11 +1081,11 @@ static int get_spec_graph(ssdk_engine* e, int B, bool host_io, bool stream_draft
 static int init_kernel_attrs() {
 #define SSDK_ATTR_G(UN, EP) \
   CK(cudaFuncSetAttribute(gemm_ws_kernel<UN, EP>, cudaFuncAttributeMaxDynamicSharedMemorySize, GemmCfg<UN>::kSmemBytes));
-  SSDK_ATTR_G(16, EPI_BF16) SSDK_ATTR_G(16, EPI_PARTIAL) SSDK_ATTR_G(16, EPI_SILU) SSDK_ATTR_G(16, EPI_PUBLISH)
-  SSDK_ATTR_G(32, EPI_BF16) SSDK_ATTR_G(32, EPI_PARTIAL) SSDK_ATTR_G(32, EPI_SILU) SSDK_ATTR_G(32, EPI_PUBLISH)
-  SSDK_ATTR_G(64, EPI_BF16) SSDK_ATTR_G(64, EPI_PARTIAL) SSDK_ATTR_G(64, EPI_SILU) SSDK_ATTR_G(64, EPI_PUBLISH)
-  SSDK_ATTR_G(128, EPI_BF16) SSDK_ATTR_G(128, EPI_PARTIAL) SSDK_ATTR_G(128, EPI_SILU)
-  SSDK_ATTR_G(256, EPI_BF16) SSDK_ATTR_G(256, EPI_PARTIAL) SSDK_ATTR_G(256, EPI_SILU)
+  SSDK_ATTR_G(16, EPI_BF16) SSDK_ATTR_G(16, EPI_PARTIAL) SSDK_ATTR_G(16, EPI_SILU) SSDK_ATTR_G(16, EPI_GLU) SSDK_ATTR_G(16, EPI_PUBLISH)
+  SSDK_ATTR_G(32, EPI_BF16) SSDK_ATTR_G(32, EPI_PARTIAL) SSDK_ATTR_G(32, EPI_SILU) SSDK_ATTR_G(32, EPI_GLU) SSDK_ATTR_G(32, EPI_PUBLISH)
+  SSDK_ATTR_G(64, EPI_BF16) SSDK_ATTR_G(64, EPI_PARTIAL) SSDK_ATTR_G(64, EPI_SILU) SSDK_ATTR_G(64, EPI_GLU) SSDK_ATTR_G(64, EPI_PUBLISH)
+  SSDK_ATTR_G(128, EPI_BF16) SSDK_ATTR_G(128, EPI_PARTIAL) SSDK_ATTR_G(128, EPI_SILU) SSDK_ATTR_G(128, EPI_GLU)
+  SSDK_ATTR_G(256, EPI_BF16) SSDK_ATTR_G(256, EPI_PARTIAL) SSDK_ATTR_G(256, EPI_SILU) SSDK_ATTR_G(256, EPI_GLU)
 #undef SSDK_ATTR_G
 #define SSDK_ATTR_A(HD, MT) \
   CK(cudaFuncSetAttribute(paged_attn_kernel<HD, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * 2 * kAttChunk * (HD + 8) * 2));

@@ -19,7 +19,8 @@
 //     an fp32 [S, M, N] buffer which the *consumer* kernel (norm / rope / silu) reduces
 //     in a fixed order, so results are deterministic.
 //   * epilogues: bf16 store, fp32 split-K partial, or fused SiLU(gate)*up where a tile is
-//     64 gate rows + 64 up rows of the packed gate|up matrix (layers/activation.py:11-14).
+//     64 gate rows + 64 up rows of the packed gate|up matrix (layers/activation.py:11-14); EPI_GLU is its form for the layered
+//     models: any number of row chunks, silu or gelu_tanh, gate and up kept in fp32 up to the product.
 //   * PDL: weight tiles of the first kStages are requested BEFORE griddepcontrol.wait, so
 //     the HBM stream of this GEMM starts under the tail of the previous kernel.
 #pragma once
@@ -32,7 +33,7 @@ constexpr int kBlockK = 64;    // bf16 per k-block = 128 B = one swizzle row
 constexpr int kTileRows = 128; // weight rows per CTA = UMMA_M
 constexpr int kGemmThreads = 192;
 
-enum GemmEpi { EPI_BF16 = 0, EPI_PARTIAL = 1, EPI_SILU = 2, EPI_PUBLISH = 3 };
+enum GemmEpi { EPI_BF16 = 0, EPI_PARTIAL = 1, EPI_SILU = 2, EPI_PUBLISH = 3, EPI_GLU = 4 };
 
 // EPI_PUBLISH — row-parallel linear + the first half of the one-shot tensor-parallel all-reduce in ONE kernel
 // (layers/linear.py:195-199: y = x W^T, then dist.all_reduce).  Every split-K CTA stores its fp32 partial tile and takes a
@@ -74,6 +75,7 @@ struct GemmParams {
   const int* g_tile_rows = nullptr;
   const int* g_n_tiles = nullptr;
   int g_expert_rows = 0;
+  int glu_gelu = 0;       // EPI_GLU: 0 silu, 1 gelu_tanh
 };
 
 // Split-K ticket reduction run by the 4 epilogue warps (threads 64..191).  `col` = this thread's column in the partial
@@ -162,7 +164,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
     m_valid = min(UMMA_N, p.g_tile_rows[blockIdx.z]);
     w_row0 = p.g_tile_expert[blockIdx.z] * p.g_expert_rows;
   }
-  const int col_lo = (EPI == EPI_SILU) ? tile * 64 : tile * kTileRows;   // first output column of the tile
+  const int col_lo = (EPI == EPI_SILU || EPI == EPI_GLU) ? tile * 64 : tile * kTileRows;   // first output column of the tile
   const int row_lo = col_lo + w_row0;                                    // its first weight row in the W map
   const int row_hi = row_lo + p.hi_row_offset;
 
@@ -272,6 +274,24 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         for (int m = 0; m < CW; ++m)
           if (m0 + m < m_valid) out[(size_t)(m0 + m) * p.N + n] = __uint_as_float(r[m]);
       }
+    } else if (EPI == EPI_GLU) {
+      // act(gate) * up: rows 0..63 = gate, 64..127 = up of the same 64 output columns; the retired pipeline stages hold the exchange
+      float* ex = reinterpret_cast<float*>(smem);
+      constexpr int LD = CW + 1;
+#pragma unroll
+      for (int m = 0; m < CW; ++m) ex[row * LD + m] = __uint_as_float(r[m]);
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out);
+      const int mc = min(CW, m_valid - m0);
+      for (int idx = threadIdx.x - 64; idx < 64 * mc; idx += 128) {
+        const int j = idx & 63, m = idx >> 6, n = col_lo + j;
+        if (n < p.N) {
+          const float g = ex[j * LD + m], u = ex[(64 + j) * LD + m];
+          const float a = p.glu_gelu ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : __fdividef(g, 1.0f + __expf(-g));
+          out[(size_t)(m_base + m0 + m) * p.ldo + n] = f2bf(a * u);
+        }
+      }
+      if (UMMA_N > CW) asm volatile("bar.sync 1, 128;" ::: "memory");  // the next pass overwrites the exchange buffer
     } else if (EPI == EPI_PUBLISH) {
       const PublishParams& pb = p.pub;
       const int n = row_lo + row;

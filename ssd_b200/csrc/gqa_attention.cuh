@@ -88,11 +88,47 @@ struct GqaConvPrepArgs {
 
 inline size_t gqa_conv_prep_smem(int C, int rot_dims) { return ((size_t)C + rot_dims + 4) * 4; }
 
+// VEC consecutive channels of a row after the convolution.  VEC = 4: channel count, row stride and pointers are whole 16-byte
+// pieces and the taps are 2 or 4 (a channel group's taps then are too)
+template <typename T, int VEC, int TAPS>
+SSDK_DEVINL void conv_group(const ConvArgs& p, const Ragged& rg, int m, int s, int t, int c, float* y) {
+  if constexpr (VEC == 1) {
+    y[0] = conv_at<T>(p, rg, m, s, t, c);
+  } else {
+    const bool carried = rg.pos0[s] > 0;
+    const float* hist = p.hist + (size_t)rg.slot[s] * p.slot_stride;
+    float w[VEC * TAPS], ib[VEC];   // w[e * TAPS + j]: channel c + e, tap j
+    ld_contig<T, VEC * TAPS>((const T*)p.w + (size_t)c * TAPS, w);
+    if (p.in_bias) ld_contig<T, VEC>((const T*)p.in_bias + c, ib);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) y[e] = 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      const int back = TAPS - 1 - j;
+      float x[VEC];
+      if (back <= t) {
+        const float4 f = *reinterpret_cast<const float4*>(p.in + (size_t)(m - back) * p.ld_in + c);
+        x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w;
+        if (p.in_bias) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) x[e] += ib[e];
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] = carried ? hist[(size_t)(TAPS - 1 - (back - t)) * p.C + c + e] : 0.f;
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = fmaf(w[e * TAPS + j], x[e], y[e]);
+    }
+  }
+}
+
 // grid (M): a CTA convolves the row's q | k | v channels into shared memory, norms the whole query and the whole key
 // projection there, turns the first rot_dims entries of every head and stores queries (group-major) and the token's page row.
-template <typename T>
+// VEC = 4: as conv_group, and D, V and the rotated part are multiples of 4 with adjacent pairs.
+template <typename T, int VEC, int TAPS>
 __global__ void gqa_conv_prep_kernel(const GqaConvPrepArgs p, const Ragged rg) {
-  extern __shared__ float gc_sm[];
+  extern __shared__ __align__(16) float gc_sm[];
   __shared__ float red[33];
   const int m = blockIdx.x, s = rg.tok_seq[m], t = m - rg.cu[s], pos = rg.pos0[s] + t;
   const int H = p.g.H, G = p.g.G, D = p.g.D, V = p.g.V, HD = H * D, QK = (H + G) * D, C = QK + G * V;
@@ -105,39 +141,64 @@ __global__ void gqa_conv_prep_kernel(const GqaConvPrepArgs p, const Ragged rg) {
     cs[i] = c * p.g.rot_mult; cs[half + i] = sn * p.g.rot_mult;
   }
   float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) {
-    const float v = conv_at<T>(p.conv, rg, m, s, t, c);
-    y[c] = v;
-    if (c < HD) sq = fmaf(v, v, sq);
-    else if (c < QK) sk = fmaf(v, v, sk);
+  for (int c = threadIdx.x * VEC; c < C; c += blockDim.x * VEC) {
+    float v[VEC], ss = 0.f;
+    conv_group<T, VEC, TAPS>(p.conv, rg, m, s, t, c, v);
+    st_vec<VEC>(y + c, v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(v[e], v[e], ss);
+    if (c < HD) sq += ss;      // (a group of VEC channels never spans q and k: their sizes are multiples of VEC)
+    else if (c < QK) sk += ss;
   }
-  if (p.g.qk_norm == 2) {
+  float iq = 1.f, ik = 1.f;
+  const bool norm = p.g.qk_norm == 2;
+  if (norm) {
     sq = block_sum(sq, red);
     sk = block_sum(sk, red);
-    const float iq = 1.0f / sqrtf(sq / (float)HD + p.g.eps), ik = 1.0f / sqrtf(sk / (float)(G * D) + p.g.eps);
-    for (int c = threadIdx.x; c < QK; c += blockDim.x) y[c] *= (c < HD ? iq : ik) * ld_f<T>((const T*)p.norm_w + c);
+    iq = 1.0f / sqrtf(sq / (float)HD + p.g.eps);
+    ik = 1.0f / sqrtf(sk / (float)(G * D) + p.g.eps);
   }
   __syncthreads();
   T* row = (T*)p.g.cache + page_row(rg, s, pos) * (size_t)(G * (D + V));
   const int hpg = H / G;
-  for (int c = threadIdx.x; c < C; c += blockDim.x) {
-    float v = y[c];
+  const T* nw = (const T*)p.norm_w;
+  for (int c = threadIdx.x * VEC; c < C; c += blockDim.x * VEC) {
+    float v[VEC];
+    ld_vec<VEC>(y + c, v);
+    T* dst = row + (c - HD);   // keys of all heads, then values: the page row's own order
     if (c < QK) {
       const int hd = c / D, d = c - hd * D;
+      if (norm) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] *= (c < HD ? iq : ik) * ld_f<T>(nw + c + e);
+      }
       if (d < rd) {
-        const int i = p.g.rot_half ? (d < half ? d : d - half) : d >> 1;
-        const bool first = p.g.rot_half ? d < half : (d & 1) == 0;
-        const int step = p.g.rot_half ? half : 1;
-        const float o = y[first ? c + step : c - step];   // the other entry of the pair
-        v = first ? v * cs[i] - o * cs[half + i] : v * cs[i] + o * cs[half + i];
+        if constexpr (VEC == 4) {
+#pragma unroll
+          for (int e = 0; e < VEC; e += 2) {
+            const float co = cs[(d + e) >> 1], sn = cs[half + ((d + e) >> 1)], a = v[e], b = v[e + 1];
+            v[e] = a * co - b * sn; v[e + 1] = b * co + a * sn;
+          }
+        } else {
+          const int i = p.g.rot_half ? (d < half ? d : d - half) : d >> 1, step = p.g.rot_half ? half : 1;
+          const bool first = p.g.rot_half ? d < half : (d & 1) == 0;
+          const int co = first ? c + step : c - step;
+          const float o = y[co] * (norm ? (c < HD ? iq : ik) * ld_f<T>(nw + co) : 1.f);   // the other entry of the pair
+          v[0] = first ? v[0] * cs[i] - o * cs[half + i] : v[0] * cs[i] + o * cs[half + i];
+        }
       }
       if (c < HD) {
         const int g = hd / hpg;
-        st_f<T>((T*)p.g.q + (((size_t)g * rg.M + m) * hpg + (hd - g * hpg)) * D + d, v);
-        continue;
+        dst = (T*)p.g.q + (((size_t)g * rg.M + m) * hpg + (hd - g * hpg)) * D + d;
       }
     }
-    st_f<T>(row + (c - HD), v);   // keys of all heads, then values: the page row's own order
+    if constexpr (VEC == 4 && sizeof(T) == 2) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+      *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st_f<T>(dst + e, v[e]);
+    }
   }
 }
 

@@ -62,6 +62,7 @@ struct ssdk_hyb_engine {
   bool use_decode_attn = true;  // fused single-token latent attention (SSDK_HYB_DECODE_ATTN=0: GEMM path for every row)
   bool use_tc_experts = true;   // routed experts of calls with many rows on the grouped tcgen05 GEMM (SSDK_HYB_TC_EXPERTS=0: mma.sync tile)
   bool use_tc_scores = true;    // score GEMM of latent-attention portions on the tcgen05 GEMM (SSDK_HYB_TC_SCORES=0: mma.sync tile)
+  bool use_tc_glu = true;       // gated feed-forward's activation in the epilogue of the tcgen05 GEMM (SSDK_HYB_TC_GLU=0: a kernel of its own)
   bool use_decode_mma = true;   // its tensor-core form for bf16 storage (SSDK_HYB_DECODE_MMA=0: the CUDA-core form)
   std::map<std::tuple<const void*, int64_t, int, int, int>, CUtensorMap> tmaps;
   float* partials = nullptr; size_t partial_floats = 0;
@@ -368,6 +369,19 @@ struct HybRun {
       CKI(L.go(ssdk::splitk_sum_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, (const float*)e->partials, C, S, n));
     }
     return 0;
+  }
+  // y [m, ff] (bf16) = act(x Wg^T) * (x Wu^T) in the GEMM's epilogue; W holds the gate rows, then the up rows
+  int lin_tc_glu(const void* A, const void* W, void* y, int m_total, int ff, int K, bool gelu) {
+    const CUtensorMap* tm;
+    CKI(e->tmap(W, 2 * ff, K, 64, &tm));
+    const CUtensorMap tmW = *tm;
+    const int un = umma_n_for(std::min(m_total, kMaxTokens)), chunks = (m_total + un - 1) / un;
+    CKI(e->tmap(A, m_total, K, un, &tm));
+    const CUtensorMap tmX = *tm;
+    GemmParams p;
+    p.M = m_total; p.N = ff; p.ldo = ff; p.num_kb = K / kBlockK; p.kb_per_split = p.num_kb; p.tile_rows = 64; p.hi_row_offset = ff;
+    p.sk_partials = nullptr; p.sk_counters = nullptr; p.sk_width = 0; p.out = y; p.glu_gelu = gelu;
+    return launch_gemm(L, un, EPI_GLU, tmW, tmX, p, (ff + 63) / 64, 1, chunks);
   }
   // grouped form: rows of X sorted by expert, tile list on the device (expert_plan_kernel with tiles of `un` rows);
   // C[r, :] = X[r, :] Wm[expert(r)]^T with Wm the experts' [N, K] matrices stacked by rows
@@ -745,14 +759,22 @@ struct HybRun {
   static constexpr bool kF32 = std::is_same<T, float>::value;
   const T* w_at(const HybTensor& t, size_t off) const { return (const T*)t.p + off; }
 
+  // rows x column slices of a row-wise activation: few rows are spread over the machine
+  static dim3 act_grid(int rows, int cols) { return dim3(rows, std::max(1, std::min((cols + 255) / 256, 4 * num_sms() / rows))); }
+
   int glu(HybLayer& Lr) {
     const int W = e->cfg.width, ff = Lr.c.ff;
     CKI(check_tensor(Lr, SSDK_HT_GLU_IN, 2 * ff, W, "mlp.gate|up")); CKI(check_tensor(Lr, SSDK_HT_GLU_OUT, W, ff, "mlp.down"));
+    // bf16 with whole k-blocks and enough 64-column tiles to stream the weights: activation and product in the GEMM's epilogue
+    if (e->use_tc_glu && (ff + 63) / 64 * ((M + kMaxTokens - 1) / kMaxTokens) >= 24 && tc_ok(hin, W, Lr.t[SSDK_HT_GLU_IN].p, W, 2 * ff, 2 * ff, W)) {
+      CKI(lin_tc_glu(hin, Lr.t[SSDK_HT_GLU_IN].p, e->t0, M, ff, W, Lr.c.ff_act == SSDK_ACT_GELU_TANH));
+      return lin(e->t0, ff, Lr.t[SSDK_HT_GLU_OUT].p, ff, e->mix_out, W, M, W, ff);
+    }
     CKI(lin(hin, W, Lr.t[SSDK_HT_GLU_IN].p, W, e->p0, 2 * ff, M, 2 * ff, W));
     if (Lr.c.ff_act == SSDK_ACT_SILU)
-      CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_SILU>, dim3(M), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
+      CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_SILU>, act_grid(M, ff), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
     else
-      CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_GELU_TANH>, dim3(M), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
+      CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_GELU_TANH>, act_grid(M, ff), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
     return lin(e->t0, ff, Lr.t[SSDK_HT_GLU_OUT].p, ff, e->mix_out, W, M, W, ff);
   }
 
@@ -852,8 +874,14 @@ struct HybRun {
     if (conv) {
       ssdk::GqaConvPrepArgs cp;
       cp.g = pa; cp.conv = *conv; cp.norm_w = norm_w;
-      // a CTA per row: few rows take more threads each
-      CKI(L.go(ssdk::gqa_conv_prep_kernel<T>, dim3(M), dim3(M < num_sms() ? 1024 : 256), ssdk::gqa_conv_prep_smem(conv->C, c.rot_dims), cp, rg));
+      // 16 bytes of channels per thread where sizes and pointers allow; a CTA per row, few rows take more threads each
+      const bool vec = (conv->taps == 2 || conv->taps == 4) && conv->w && D % 4 == 0 && V % 4 == 0 && c.rot_dims % 4 == 0 && !c.rot_half &&
+                       conv->ld_in % 4 == 0 && (((uintptr_t)conv->in | (uintptr_t)conv->w | (uintptr_t)conv->in_bias | (uintptr_t)pool | (uintptr_t)e->qcat) & 15) == 0;
+      const dim3 grid(M), block(M < num_sms() ? (vec ? 512 : 1024) : 256);
+      const size_t smem = ssdk::gqa_conv_prep_smem(conv->C, c.rot_dims);
+      if (vec && conv->taps == 4) CKI(L.go(ssdk::gqa_conv_prep_kernel<T, 4, 4>, grid, block, smem, cp, rg));
+      else if (vec) CKI(L.go(ssdk::gqa_conv_prep_kernel<T, 4, 2>, grid, block, smem, cp, rg));
+      else CKI(L.go(ssdk::gqa_conv_prep_kernel<T, 1, 1>, grid, block, smem, cp, rg));
       if (conv->taps > 1) CKI(L.go(ssdk::conv_state_kernel<T>, dim3(rg.n_seqs, (conv->C + 255) / 256), dim3(256), 0, *conv, rg));
     } else {
       CKI(L.go(ssdk::gqa_prep_kernel<T>, dim3(M, H + G), dim3(32), 0, pa, rg));
@@ -1217,8 +1245,11 @@ static int hyb_smem_attrs(ssdk_hyb_engine* e) {
   SSDK_DELTA_ATTR(16, 8)
 #undef SSDK_DELTA_ATTR
   CK(cudaFuncSetAttribute(ssdk::delta_scan_any_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+#define SSDK_PREP_ATTR(VEC, TAPS) \
+  CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<bf16, VEC, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<float, VEC, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  SSDK_PREP_ATTR(4, 4) SSDK_PREP_ATTR(4, 2) SSDK_PREP_ATTR(1, 1)
+#undef SSDK_PREP_ATTR
 #define SSDK_STREAM_ATTR(SM, VEC) \
   CK(cudaFuncSetAttribute(ssdk::stream_step_kernel<bf16, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
   CK(cudaFuncSetAttribute(ssdk::stream_step_kernel<float, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
@@ -1327,6 +1358,7 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
   e->use_tc = env_int("SSDK_HYB_TCGEN05", 1) != 0;
   e->use_decode_attn = env_int("SSDK_HYB_DECODE_ATTN", 1) != 0;
   e->use_decode_mma = env_int("SSDK_HYB_DECODE_MMA", 1) != 0;
+  e->use_tc_glu = env_int("SSDK_HYB_TC_GLU", 1) != 0;
   e->use_tc_scores = env_int("SSDK_HYB_TC_SCORES", 1) != 0;
   e->use_tc_experts = env_int("SSDK_HYB_TC_EXPERTS", 1) != 0;
   e->layers.resize(cfg->n_layers);

@@ -159,7 +159,7 @@ template <typename T, int ACT>
 __global__ void glu_act_kernel(const float* __restrict__ z, int ldz, T* __restrict__ y, int ff, const int* __restrict__ n_rows) {
   const int r = blockIdx.x;
   if (n_rows && r >= *n_rows) return;
-  for (int c = threadIdx.x; c < ff; c += blockDim.x)
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ff; c += gridDim.y * blockDim.x)   // (columns may be spread over gridDim.y)
     st_f<T>(y + (size_t)r * ff + c, act_f<ACT>(z[(size_t)r * ldz + c]) * z[(size_t)r * ldz + ff + c]);
 }
 

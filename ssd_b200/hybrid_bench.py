@@ -57,7 +57,7 @@ def kefurax_pairs_spec(z):
     return kefurax_spec(z, ("parallel",))
 
 
-def vatolorn_spec(z, chunk=1024):
+def vatolorn_spec(z, chunk=4096):
     """Layers that resemble a real model's: attention with 128-wide heads, four query heads per key/value head, half of a head
     rotated, 4 taps on q | k | v, chunks of `chunk` positions; a delta rule with 128 x 128 heads, two heads per query/key head,
     4 taps, rank-128 decay and output-gate projections; four residual streams; the feed-forward of the Kefurax arm."""
@@ -298,12 +298,13 @@ def run_vatolorn(args):
     for name in names:
         z = SIZES[name]
         row = {"config": {k: z[k] for k in ("width", "layers", "vocab")}, "prompt": args.prompt_len_hybrid, "decode_batch": args.hybrid_batch,
-               "chunk": 1024, "streams": 4}
-        row["vatolorn"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, spec_fn=vatolorn_spec)
+               "chunk": args.hybrid_chunk, "streams": 4}
+        spec_fn = lambda zz: vatolorn_spec(zz, args.hybrid_chunk)
+        row["vatolorn"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, spec_fn=spec_fn)
         if not args.no_dense_arm:
             row["kefurax_pairs"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, spec_fn=kefurax_pairs_spec)
         if args.hybrid_fp32:
-            row["vatolorn_fp32"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, "float32", vatolorn_spec)
+            row["vatolorn_fp32"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, "float32", spec_fn)
         out["sizes"][name] = row
     return out
 

@@ -54,15 +54,15 @@ FULL = [U.parallel(mlp=U.dense()),
                    U.delta(heads=3, kv_heads=3, dim=40, vdim=36, conv=2, decay_rank=3, gate_rank=16), mlp=U.dense(ff=33))]
 
 
-@pytest.mark.parametrize("left", [U.attention(), U.attention(heads=3, kv_heads=3, dim=12, vdim=12, conv=1, chunk=1000, dims=12),
+@pytest.mark.parametrize("left", [U.attention(), U.attention(heads=4, dim=12, vdim=8, conv=4, dims=8), U.attention(heads=4, dim=8, vdim=20, conv=2, dims=8), U.attention(heads=3, kv_heads=3, dim=12, vdim=12, conv=1, chunk=1000, dims=12),
                                   U.attention(heads=8, kv_heads=2, dim=4, vdim=7, conv=6, chunk=1, dims=2, scaling=None),
                                   U.attention(heads=2, kv_heads=1, dim=33, vdim=40, conv=2, chunk=16, dims=0),
                                   U.attention(heads=1, kv_heads=1, dim=7, vdim=1, conv=3, chunk=5, dims=6, base=10.0),
                                   U.attention(conv=0, chunk=0)],
-                         ids=["grouped", "no-groups-full-rotation-wide-chunk", "chunk-of-one", "no-rotation-wide-values", "one-head-odd-size", "no-conv-no-chunks"])
+                         ids=["grouped", "whole-vectors-4-taps", "whole-vectors-2-taps", "no-groups-full-rotation-wide-chunk", "chunk-of-one", "no-rotation-wide-values", "one-head-odd-size", "no-conv-no-chunks"])
 def test_attention_alone(tmp_path, left):
     """The delta rule's norm weight is zero, so the layer is the attention half behind the streams."""
-    cfg = U.config([U.parallel(left=left)], streams=2)
+    cfg = U.config([U.parallel(left=left, right=U.delta(heads=4, kv_heads=2, vdim=8))], streams=2)
     tensors = U.random_tensors(cfg, 1)
     tensors["l0.mix.right.out"].zero_()
     r, plain, _ = _runner(tmp_path, cfg, tensors=tensors)
@@ -400,6 +400,28 @@ def test_bfloat16_calls_of_many_rows(tmp_path):
         out.append(r.forward([(seqs[0][pos:pos + c], pos, 2, _pages(330, 16, 30), list(range(c)))])[0])
         pos += c
     assert U.rel_err(np.concatenate(out), lg[:330]) < 2e-2
+
+
+def test_gated_feed_forward_in_the_gemm(tmp_path, monkeypatch):
+    """bf16: the gated feed-forward whose activation runs in the epilogue of the tcgen05 GEMM (a width of whole 64-column tiles,
+    and one that ends inside a tile) against the separate activation kernel and the oracle: several row chunks, a short
+    portion, single tokens."""
+    cfg = U.config([U.parallel(mlp=U.dense(ff=1600)), U.parallel(mlp=U.dense(ff=1548))], width=128, streams=2)
+    tensors = U.random_tensors(cfg, 0)
+    path = U.write(str(tmp_path / "glu"), cfg, tensors)
+    toks = _tokens(310, cfg["vocab"], 5)
+    ref, got = PlainModel(cfg, tensors).run(toks).numpy(), {}
+    for glu in ("1", "0"):
+        monkeypatch.setenv("SSDK_HYB_TC_GLU", glu)
+        r = _load(path, "bfloat16")
+        out, pos = [], 0
+        for c in [290, 17, 1, 1, 1]:
+            out.append(r.forward([(toks[pos:pos + c], pos, 2, _pages(310, 16), list(range(c)))])[0])
+            pos += c
+        got[glu] = np.concatenate(out)
+        assert U.rel_err(got[glu], ref) < BF16_TOL
+        r.close()
+    assert U.rel_err(got["1"], got["0"]) < 5e-3
 
 
 def test_greedy_generation_through_llm(tmp_path):
