@@ -14,6 +14,7 @@
 //   portions (>= 2 rows) two batched GEMMs per query block around sink_softmax_kernel (HybRun::gqa_attention)
 //   single-token rows    gqa_decode_partial_kernel (all decoding sequences in one launch, context split flash-decoding
 //                        style, fp32 weights) + gqa_decode_merge_kernel
+//                        (bf16 storage with 16-byte rows: the tensor-core forms of gqa_mma.cuh take both kinds of rows)
 //   attn_gate_kernel     group-major fp32 output x sigmoid(gate pre-activation) -> [M, H V] (T) for the output projection
 #pragma once
 #include "conv_scan.cuh"  // ConvArgs, conv_at
@@ -219,7 +220,9 @@ struct GqaDecodeArgs {
   const void* q;      // [G, M, H/G, D] T
   const void* cache;  // [rows, G (D + V)] T
   float* part;        // [n_seqs, H, splits, V + 2] fp32: unnormalised P V | running maximum | running sum
-  float* out;         // [G, M, H/G, V] fp32
+  void* y;            // [M, H V] T
+  const float* gate;  // pre-activations of a sigmoid gate, gate[m * ld_gate + h V + v], or nullptr
+  int ld_gate;
   int H, G, D, V, splits;
   float scale, sink;
   const void* sinks;  // [H] T learned sink logits (they replace the constant), or nullptr
@@ -339,40 +342,43 @@ __global__ void __launch_bounds__(kGqaDecWarps * 32) gqa_decode_partial_kernel(c
   if (tid == 0) dst[V] = m;
 }
 
-// grid (n_seqs, H): out = sum_j e^(m_j - m) acc_j / (e^(s - m) + sum_j e^(m_j - m) l_j), s the sink's logit (ln of the
-// constant, or the head's learned one)
+constexpr int kGqaMaxSplits = 32;
+
+// grid (n_seqs, H): y = sum_j e^(m_j - m) acc_j / (e^(s - m) + sum_j e^(m_j - m) l_j), s the sink's logit (ln of the constant, or
+// the head's learned one), times the sigmoid of the gate's pre-activation if the layer has a gate
 template <typename T>
 __global__ void gqa_decode_merge_kernel(const GqaDecodeArgs p, const Ragged rg) {
+  __shared__ float w[kGqaMaxSplits];
   const int s = blockIdx.x, hd = blockIdx.y;
   const int row = rg.cu[s];
   if (rg.cu[s + 1] - row != 1) return;
-  const int V = p.V, hpg = p.H / p.G, g = hd / hpg;
+  const int V = p.V;
   const float* part = p.part + ((size_t)s * p.H + hd) * p.splits * (V + 2);
-  const float sk = p.sinks ? ld_f<T>((const T*)p.sinks + hd) : (p.sink > 0.f ? logf(p.sink) : -INFINITY);
-  float m = sk;
-  for (int j = 0; j < p.splits; ++j) m = fmaxf(m, part[(size_t)j * (V + 2) + V]);
-  float den = sk == -INFINITY ? 0.f : expf(sk - m);
-  for (int j = 0; j < p.splits; ++j) {
-    const float mj = part[(size_t)j * (V + 2) + V];
-    if (mj != -INFINITY) den += expf(mj - m) * part[(size_t)j * (V + 2) + V + 1];
+  if (threadIdx.x < 32) {   // a lane per split: its weight, normalised
+    const int j = threadIdx.x;
+    const float sk = p.sinks ? ld_f<T>((const T*)p.sinks + hd) : (p.sink > 0.f ? logf(p.sink) : -INFINITY);
+    const float mj = j < p.splits ? part[(size_t)j * (V + 2) + V] : -INFINITY;
+    const float m = fmaxf(sk, warp_max(mj));
+    const float e = mj == -INFINITY ? 0.f : expf(mj - m);
+    const float den = warp_sum(j < p.splits ? e * part[(size_t)j * (V + 2) + V + 1] : 0.f) + (sk == -INFINITY ? 0.f : expf(sk - m));
+    w[j] = e / den;
   }
-  const float inv = 1.0f / den;
-  float* out = p.out + (((size_t)g * rg.M + row) * hpg + (hd - g * hpg)) * V;
+  __syncthreads();
+  T* y = (T*)p.y + (size_t)row * p.H * V + (size_t)hd * V;
   for (int c = threadIdx.x; c < V; c += blockDim.x) {
     float a = 0.f;
-    for (int j = 0; j < p.splits; ++j) {
-      const float mj = part[(size_t)j * (V + 2) + V];
-      if (mj != -INFINITY) a = fmaf(expf(mj - m), part[(size_t)j * (V + 2) + c], a);
-    }
-    out[c] = a * inv;
+#pragma unroll 4
+    for (int j = 0; j < p.splits; ++j) a = fmaf(w[j], part[(size_t)j * (V + 2) + c], a);
+    if (p.gate) a *= sigmoid_f(p.gate[(size_t)row * p.ld_gate + (size_t)hd * V + c]);
+    st_f<T>(y + c, a);
   }
 }
 
-// o [G, M, H/G, V] fp32 (group-major) and gate pre-activations gz[m * ldg + h * V + v] -> y [M, H V] (T) = o * sigmoid(gz)
+// o [G, M, H/G, V] fp32 (group-major) and gate pre-activations gz[m * ldg + h * V + v] -> y [M, H V] (T) = o * sigmoid(gz), rows row0 ..
 template <typename T>
 __global__ void attn_gate_kernel(const float* __restrict__ o, const float* __restrict__ gz, int ldg, T* __restrict__ y, int M, int H,
-                                 int G, int V) {
-  const int m = blockIdx.x, hpg = H / G;
+                                 int G, int V, int row0) {
+  const int m = row0 + blockIdx.x, hpg = H / G;
   for (int i = threadIdx.x; i < H * V; i += blockDim.x) {
     const int hd = i / V, v = i - hd * V, g = hd / hpg;
     const float ov = o[(((size_t)g * M + m) * hpg + (hd - g * hpg)) * V + v];

@@ -5,6 +5,7 @@
 #pragma once
 #include "conv_scan.cuh"
 #include "gqa_attention.cuh"
+#include "gqa_mma.cuh"
 #include "latent_attention.cuh"
 #include "layer_ops.cuh"
 #include "linear.cuh"
@@ -62,6 +63,7 @@ struct ssdk_hyb_engine {
   bool use_decode_attn = true;  // fused single-token latent attention (SSDK_HYB_DECODE_ATTN=0: GEMM path for every row)
   bool use_tc_experts = true;   // routed experts of calls with many rows on the grouped tcgen05 GEMM (SSDK_HYB_TC_EXPERTS=0: mma.sync tile)
   bool use_tc_scores = true;    // score GEMM of latent-attention portions on the tcgen05 GEMM (SSDK_HYB_TC_SCORES=0: mma.sync tile)
+  bool use_gqa_mma = true;      // grouped-query attention on the tensor cores (SSDK_HYB_GQA_MMA=0: GEMMs around a softmax, CUDA-core decode)
   bool use_tc_glu = true;       // gated feed-forward's activation in the epilogue of the tcgen05 GEMM (SSDK_HYB_TC_GLU=0: a kernel of its own)
   bool use_decode_mma = true;   // its tensor-core form for bf16 storage (SSDK_HYB_DECODE_MMA=0: the CUDA-core form)
   std::map<std::tuple<const void*, int64_t, int, int, int>, CUtensorMap> tmaps;
@@ -661,7 +663,7 @@ struct HybRun {
     // the concatenated heads, if the layer has one: the product stays fp32 up to the gate)
     if (gate) {
       CKI(lin(e->t0, H * KR, Lr.t[SSDK_HT_LAT_UV].p, KR, e->p1, H * V, M, V, KR, false, H, KR, (long long)V * KR, V));
-      CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(M), dim3(256), 0, (const float*)e->p1, gate, ldq, (T*)e->t1, M, H, 1, V));
+      CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(M), dim3(256), 0, (const float*)e->p1, gate, ldq, (T*)e->t1, M, H, 1, V, 0));
     } else {
       CKI(lin(e->t0, H * KR, Lr.t[SSDK_HT_LAT_UV].p, KR, e->t1, H * V, M, V, KR, true, H, KR, (long long)V * KR, V));
     }
@@ -856,10 +858,11 @@ struct HybRun {
     return lin(e->t1, I, Lr.t[SSDK_HT_MIX_OUT].p, I, e->mix_out, W, M, W, I);
   }
 
-  // grouped-query attention over the layer's page pool: z holds q | k | v (fp32); og [G, M, H/G, V] fp32.  conv (optional): z's
+  // grouped-query attention over the layer's page pool: z holds q | k | v (fp32) -> y [M, H V] (T), times
+  // sigmoid(gate pre-activation) if gate is given; og [G, M, H/G, V] fp32 is scratch.  conv (optional): z's
   // columns pass through a bias and a short convolution over time first, norm_w: then through a norm over the whole query
   // and key projection
-  int gqa_attention(HybLayer& Lr, const float* z, int ldz, float* og, const void* sinks = nullptr, const ssdk::ConvArgs* conv = nullptr,
+  int gqa_attention(HybLayer& Lr, const float* z, int ldz, void* y, float* og, const float* gate, int ld_gate, const void* sinks = nullptr, const ssdk::ConvArgs* conv = nullptr,
                     const void* norm_w = nullptr) {
     const ssdk_hyb_layer_cfg& c = Lr.c;
     const int H = c.heads, G = c.kv_heads, D = c.dim, V = c.vdim, hpg = H / G;
@@ -886,33 +889,56 @@ struct HybRun {
     } else {
       CKI(L.go(ssdk::gqa_prep_kernel<T>, dim3(M, H + G), dim3(32), 0, pa, rg));
     }
+    // tensor-core forms: bf16, heads of whole 16-byte pieces up to 128 wide, up to 16 query heads per key/value head
+    const bool mma = !kF32 && e->use_gqa_mma && D % 8 == 0 && V % 8 == 0 && std::max(D, V) <= 128 && hpg <= 16 && ((uintptr_t)pool & 15) == 0;
+    const int ks = std::max(D, V) <= 32 ? 2 : (std::max(D, V) <= 64 ? 4 : 8), vt = 2 * ks;
     bool fused_decode = false;
     {
       int ctx_max = 0;
       const int n_dec = decode_rows(mask, &ctx_max);
       const int vpl = (V + 31) / 32;
-      if (n_dec > 0 && vpl <= 8 && e->use_decode_attn) {
-        int splits = std::max(1, std::min({32, 8 * num_sms() / std::max(1, n_dec * H), (ctx_max + 127) / 128}));  // ~8 four-warp CTAs per SM
+      if (n_dec > 0 && (mma || vpl <= 8) && e->use_decode_attn) {
+        // tensor cores: ~3 four-warp CTAs per SM, at least a tile of keys each; CUDA cores: ~8 per SM (a CTA per head)
+        int splits = mma ? std::min({ssdk::kGqaMaxSplits, 3 * num_sms() / std::max(1, n_dec * G), (ctx_max + ssdk::kGmKeys - 1) / ssdk::kGmKeys})
+                         : std::min({ssdk::kGqaMaxSplits, 8 * num_sms() / std::max(1, n_dec * H), (ctx_max + 127) / 128});
+        splits = std::max(1, splits);
         const size_t per_split = (size_t)rg.n_seqs * H * (V + 2);
         splits = (int)std::min<size_t>(splits, e->att_elems / per_split);
         if (splits >= 1) {
           ssdk::GqaDecodeArgs da;
-          da.q = e->qcat; da.cache = pool; da.part = e->att_s; da.out = og; da.H = H; da.G = G; da.D = D; da.V = V; da.splits = splits;
+          da.q = e->qcat; da.cache = pool; da.part = e->att_s; da.y = y; da.gate = gate; da.ld_gate = ld_gate; da.H = H; da.G = G; da.D = D; da.V = V; da.splits = splits;
           da.scale = c.attn_scale; da.sink = sink_const; da.sinks = sinks; da.mask = mask;
-          const dim3 grid(rg.n_seqs, H, splits), block(ssdk::kGqaDecWarps * 32);
-          const size_t smem = ssdk::gqa_decode_smem(D, V);
-          if (vpl <= 1) CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 1>, grid, block, smem, da, rg));
+          const dim3 grid(rg.n_seqs, H, splits), block(ssdk::kGqaDecWarps * 32), mgrid(rg.n_seqs, G, splits), mblock(128);
+          const size_t smem = ssdk::gqa_decode_smem(D, V), msmem = ssdk::gqa_decode_mma_smem(ks, vt, V);
+          if (mma && ks == 2) CKI(L.go(ssdk::gqa_decode_mma_kernel<2, 4>, mgrid, mblock, msmem, da, rg));
+          else if (mma && ks == 4) CKI(L.go(ssdk::gqa_decode_mma_kernel<4, 8>, mgrid, mblock, msmem, da, rg));
+          else if (mma) CKI(L.go(ssdk::gqa_decode_mma_kernel<8, 16>, mgrid, mblock, msmem, da, rg));
+          else if (vpl <= 1) CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 1>, grid, block, smem, da, rg));
           else if (vpl <= 2) CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 2>, grid, block, smem, da, rg));
           else if (vpl <= 4) CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 4>, grid, block, smem, da, rg));
           else CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 8>, grid, block, smem, da, rg));
-          CKI(L.go(ssdk::gqa_decode_merge_kernel<T>, dim3(rg.n_seqs, H), dim3(64), 0, da, rg));
+          CKI(L.go(ssdk::gqa_decode_merge_kernel<T>, dim3(rg.n_seqs, H), dim3(V <= 64 ? 64 : 128), 0, da, rg));
           fused_decode = true;
         }
       }
     }
+    if (mma) {   // all portions in one launch
+      int n_max = 0;
+      for (int s = 0; s < rg.n_seqs; ++s) n_max = std::max(n_max, h_cu[s + 1] - h_cu[s]);
+      if (n_max > 1) {
+        ssdk::GqaPortionArgs fa;
+        fa.q = e->qcat; fa.cache = pool; fa.y = y; fa.gate = gate; fa.ld_gate = ld_gate; fa.H = H; fa.G = G; fa.D = D; fa.V = V;
+        fa.scale = c.attn_scale; fa.sink = sink_const; fa.sinks = sinks; fa.mask = mask;
+        const dim3 grid((n_max * hpg + ssdk::kGpRows - 1) / ssdk::kGpRows, G, rg.n_seqs), block(ssdk::kGpWarps * 32);
+        const size_t smem = 2 * ssdk::gm_tile_bytes(ks, vt);
+        if (ks == 2) CKI(L.go(ssdk::gqa_portion_mma_kernel<2, 4>, grid, block, smem, fa, rg));
+        else if (ks == 4) CKI(L.go(ssdk::gqa_portion_mma_kernel<4, 8>, grid, block, smem, fa, rg));
+        else CKI(L.go(ssdk::gqa_portion_mma_kernel<8, 16>, grid, block, smem, fa, rg));
+      }
+    }
     for (int s = 0; s < rg.n_seqs; ++s) {
       const int r0 = h_cu[s], n = h_cu[s + 1] - r0, p0 = h_pos0[s];
-      if (fused_decode && n == 1) continue;
+      if (n == 1 ? fused_decode : mma) continue;
       const int lo = mask.first(p0), ctx = p0 + n - lo, ctx_pad = (ctx + 7) / 8 * 8;   // keys lo .. p0 + n - 1
       CKI(L.go(ssdk::kv_gather_kernel<T>, dim3(ctx_pad), dim3(128), 0, (const T*)pool, (T*)e->keys, (T*)e->lat_t, rg, s, lo, ctx, ctx_pad, G, D, V));
       const int qb = (int)std::max<size_t>(1, e->att_elems / ((size_t)H * ctx_pad));
@@ -928,6 +954,7 @@ struct HybRun {
         CKI(lin(e->att_p, cb, (const T*)e->lat_t + kb, ctx_pad, og + (size_t)(r0 + q0) * hpg * V, V, rows, V, cb, false, G, (long long)rows * cb,
                 (long long)V * ctx_pad, (long long)M * hpg * V, false));
       }
+      CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(n), dim3(256), 0, (const float*)og, gate, ld_gate, (T*)y, M, H, G, V, r0));
     }
     return 0;
   }
@@ -945,8 +972,7 @@ struct HybRun {
     ssdk::ConvArgs ca = {};
     ca.in = e->p0; ca.ld_in = Nqkv; ca.in_bias = Lr.t[SSDK_HT_ATTN_IN_B].p; ca.w = Lr.t[SSDK_HT_CONV_W].p;
     ca.hist = e->state + Lr.state_off; ca.slot_stride = e->slot_floats; ca.C = Nqkv; ca.taps = taps;
-    CKI(gqa_attention(Lr, e->p0, Nqkv, e->p2, c.learned_sink ? Lr.t[SSDK_HT_ATTN_SINK].p : nullptr, &ca));
-    CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(M), dim3(256), 0, (const float*)e->p2, (const float*)nullptr, 0, (T*)e->t0, M, H, G, V));
+    CKI(gqa_attention(Lr, e->p0, Nqkv, e->t0, e->p2, nullptr, 0, c.learned_sink ? Lr.t[SSDK_HT_ATTN_SINK].p : nullptr, &ca));
     return lin(e->t0, H * V, Lr.t[SSDK_HT_MIX_OUT].p, H * V, e->mix_out, W, M, W, H * V);
   }
 
@@ -970,17 +996,16 @@ struct HybRun {
     if (Rg) CKI(check_tensor(Lr, SSDK_HT_DELTA_G2, dHV, Rg, "right.g2"));
     CKI(lin(hin, W, Lr.t[SSDK_HT_PAIR_IN].p, W, e->p0, Ntot, M, Ntot, W));
     // left: attention
+    const float* agate = c.pair_gate ? e->p0 + o_g : nullptr;
     if (c.pair_conv || c.qk_norm == 2 || Lr.t[SSDK_HT_ATTN_IN_B].p) {
       if (c.qk_norm == 1) return fail("attention pair: the per-head unit norm is built for projections without a bias");
       ssdk::ConvArgs ca = {};
       ca.in = e->p0; ca.ld_in = Ntot; ca.in_bias = Lr.t[SSDK_HT_ATTN_IN_B].p; ca.w = c.pair_conv ? Lr.t[SSDK_HT_ATTN_CONV_W].p : nullptr;
       ca.hist = e->state + Lr.attn_hist_off; ca.slot_stride = e->slot_floats; ca.C = Ca; ca.taps = std::max(1, c.pair_conv);
-      CKI(gqa_attention(Lr, e->p0, Ntot, e->p1, nullptr, &ca, Lr.t[SSDK_HT_ATTN_QK_NORM].p));
+      CKI(gqa_attention(Lr, e->p0, Ntot, e->t0, e->p1, agate, Ntot, nullptr, &ca, Lr.t[SSDK_HT_ATTN_QK_NORM].p));
     } else {
-      CKI(gqa_attention(Lr, e->p0, Ntot, e->p1));
+      CKI(gqa_attention(Lr, e->p0, Ntot, e->t0, e->p1, agate, Ntot));
     }
-    CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(M), dim3(256), 0, (const float*)e->p1, (const float*)(c.pair_gate ? e->p0 + o_g : nullptr), Ntot,
-             (T*)e->t0, M, H, G, V));
     CKI(lin(e->t0, HV, Lr.t[SSDK_HT_ATTN_OUT].p, HV, e->mix_out, W, M, W, HV));
     // right: gated delta rule
     float* st = e->state + Lr.state_off;
@@ -1250,6 +1275,11 @@ static int hyb_smem_attrs(ssdk_hyb_engine* e) {
   CK(cudaFuncSetAttribute(ssdk::gqa_conv_prep_kernel<float, VEC, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   SSDK_PREP_ATTR(4, 4) SSDK_PREP_ATTR(4, 2) SSDK_PREP_ATTR(1, 1)
 #undef SSDK_PREP_ATTR
+#define SSDK_GQA_ATTR(KS, VT) \
+  CK(cudaFuncSetAttribute(ssdk::gqa_portion_mma_kernel<KS, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_decode_mma_kernel<KS, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  SSDK_GQA_ATTR(2, 4) SSDK_GQA_ATTR(4, 8) SSDK_GQA_ATTR(8, 16)
+#undef SSDK_GQA_ATTR
 #define SSDK_STREAM_ATTR(SM, VEC) \
   CK(cudaFuncSetAttribute(ssdk::stream_step_kernel<bf16, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
   CK(cudaFuncSetAttribute(ssdk::stream_step_kernel<float, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
@@ -1358,6 +1388,7 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
   e->use_tc = env_int("SSDK_HYB_TCGEN05", 1) != 0;
   e->use_decode_attn = env_int("SSDK_HYB_DECODE_ATTN", 1) != 0;
   e->use_decode_mma = env_int("SSDK_HYB_DECODE_MMA", 1) != 0;
+  e->use_gqa_mma = env_int("SSDK_HYB_GQA_MMA", 1) != 0;
   e->use_tc_glu = env_int("SSDK_HYB_TC_GLU", 1) != 0;
   e->use_tc_scores = env_int("SSDK_HYB_TC_SCORES", 1) != 0;
   e->use_tc_experts = env_int("SSDK_HYB_TC_EXPERTS", 1) != 0;

@@ -402,6 +402,41 @@ def test_bfloat16_calls_of_many_rows(tmp_path):
     assert U.rel_err(np.concatenate(out), lg[:330]) < 2e-2
 
 
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim,chunk", [(6, 2, 40, 64, 50), (8, 2, 128, 96, 130), (3, 3, 72, 128, 1000), (16, 1, 24, 8, 77), (5, 1, 64, 16, 0)])
+def test_attention_on_the_tensor_cores(tmp_path, monkeypatch, heads, kv_heads, dim, vdim, chunk):
+    """bf16: the fused portion and decode kernels (every tile size, groups of one to sixteen heads, heads that do not fill a
+    tile, chunks shorter and longer than a tile of keys) against the oracle and against the GEMM path.  Attention is sharp
+    enough that a key too many or too few at a chunk's edge shows far above bf16 rounding."""
+    att = U.attention(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, conv=2, chunk=chunk, scale=2.5 / dim ** 0.5, dims=8)
+    cfg = U.config([U.parallel(copy.deepcopy(att)), U.parallel(copy.deepcopy(att), mlp=U.dense(ff=64))], width=64, vocab=96)
+    tensors = U.random_tensors(cfg, 3)
+    path = U.write(str(tmp_path / "mma"), cfg, tensors)
+    n = 330
+    toks = _tokens(n, cfg["vocab"], 15)
+    ref, got = PlainModel(cfg, tensors).run(toks).numpy(), {}
+    for mma in ("1", "0"):
+        monkeypatch.setenv("SSDK_HYB_GQA_MMA", mma)
+        r = _load(path, "bfloat16", num_blocks=64)
+        pages = _pages(n, 16, 7)[::-1]
+        whole, _ = r.forward([(toks, 0, 0, pages, list(range(n)))])
+        out, pos = [], 0
+        for c in [67, 2, 150, 1, 1, 60, 9] + [1] * 40:   # beside a second sequence's portion and a third one's single token
+            ents = [(toks[pos:pos + c], pos, 1, pages, list(range(c))), (toks[:5], 0, 2, [40], [])]
+            out.append(r.forward(ents + [([toks[0]], 0, 3, [41], [])])[0])
+            pos += c
+        got[mma] = (whole, np.concatenate(out))
+        for g in got[mma]:
+            assert U.rel_err(g, ref) < BF16_TOL and _per_pos(g, ref).max() < 5 * BF16_TOL
+        r.close()
+    assert U.rel_err(got["1"][0], got["0"][0]) < 2e-2 and U.rel_err(got["1"][1], got["0"][1]) < 2e-2
+    if chunk:
+        other = copy.deepcopy(cfg)
+        for lc in other["layers"]:
+            lc["mixer"]["left"]["mask"]["size"] += 1
+        moved = _per_pos(PlainModel(other, tensors).run(toks).numpy(), ref)
+        assert chunk > n or moved.max() > 5 * BF16_TOL
+
+
 def test_gated_feed_forward_in_the_gemm(tmp_path, monkeypatch):
     """bf16: the gated feed-forward whose activation runs in the epilogue of the tcgen05 GEMM (a width of whole 64-column tiles,
     and one that ends inside a tile) against the separate activation kernel and the oracle: several row chunks, a short
