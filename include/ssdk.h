@@ -260,7 +260,7 @@ int ssdk_verify(const void* logits_p, const void* logits_q, const int64_t* specu
  * Block kinds (SSDK_BLOCK_*): mixer and mixture of experts read the SAME normed input and join the residual
  * stream through per-channel layer scales (parallel pre-norm); each sublayer reads the residual stream itself and
  * its OUTPUT is normed before it is added (serial post-norm); or mixer and feed-forward read the same residual row
- * through a norm weight of their own and are added unscaled (parallel, two norms); or both read one plain norm's rows, each
+ * through a norm weight of their own and are added unscaled (parallel, two norms); each sublayer's input AND output are normed (serial, norms on both sides); or both read one plain norm's rows, each
  * through a short input convolution of its own, and are gated per channel before they are added (parallel, one norm).  The reference has no such model; these entry
  * points follow the conventions of the ones above (caller-owned device memory, int return codes).
  * Storage type T of weights / activations / latent cache: bf16 (fp32 accumulation; residual stream, norms, routers,
@@ -270,8 +270,10 @@ enum { SSDK_MIX_WKV = 0, SSDK_MIX_MLSTM = 1, SSDK_MIX_LATENT_ATTN = 2,
        SSDK_MIX_RGLRU = 3,        /* gated diagonal linear recurrence behind a short convolution, times a gelu branch */
        SSDK_MIX_SELECTIVE = 4,    /* selective scan (input-dependent step, B, C) behind a short convolution, silu gate */
        SSDK_MIX_ATTN_DELTA = 5,   /* grouped-query attention and a gated delta rule side by side on the same input (variants: pair_* and d_* fields) */
-       SSDK_MIX_ATTENTION = 6 };  /* grouped-query attention alone: biased q | k | v projections behind a short convolution,
-                                   * rotate-half rotation of the first rot_dims entries, optional sliding window, learned sink */
+       SSDK_MIX_ATTENTION = 6,    /* grouped-query attention alone: biased q | k | v projections behind a short convolution,
+                                   * rotate-half rotation of the first rot_dims entries, optional sliding window, learned sink; or, without
+                                   * bias and convolution, a norm per head before the rotation (qk_norm 3) and two maps per head (maps 2) */
+       SSDK_MIX_RETENTION = 7 };  /* linear attention with a fixed decay per head (ssdk_hyb_retention_decay), norm per head, silu gate */
 enum { SSDK_MLP_NONE = 0, SSDK_MLP_MOE = 1, SSDK_MLP_GLU = 2, /* dense: down(act(gate h) * (up h)), act = ff_act (silu or gelu_tanh) */
        SSDK_MLP_FFN = 3 };        /* dense, not gated: down(act(up h + b_up)) + b_down, act = ff_act */
 /* activations of the feed-forward kernels; CLAMPED is the limited GLU g sigmoid(1.702 g) (u + 1) */
@@ -283,6 +285,7 @@ enum { SSDK_BLOCK_PARALLEL_PRENORM = 0,  /* x += ls1 * mixer(h) + ls2 * ff(h), h
        SSDK_BLOCK_PARALLEL_TWO_NORMS = 2, /* x += mixer(norm1(x)) + ff(norm2(x)): one statistic, two weights, no layer scales */
        SSDK_BLOCK_SERIAL_PRENORM = 4,    /* x += mixer(norm1(x)); x += ff(norm2(x)).  streams > 0: the residual is `streams` copies x_s, a
                                           * sublayer reads norm(sum_s in[s] x_s) and its result y enters as x_t = sum_s mix[s, t] x_s + out[t] y */
+       SSDK_BLOCK_SERIAL_SANDWICH = 5,   /* x += m * post1(mixer(norm1(x))); x += m * post2(ff(norm2(x))): a norm before AND after each sublayer */
        SSDK_BLOCK_PARALLEL_ONE_NORM = 3 }; /* h = norm(x); x += g1 * mixer(h + conv1(h)) + g2 * ff(h + conv2(h)): plain norm weight; the
                                             * input convolutions (canon_taps > 0) and the gates g = sigmoid(W_g h + b) (gated_residual) are optional */
 
@@ -370,7 +373,7 @@ enum {
   /* attention of the pair: taps of its convolution over q | k | v (pair_conv > 0; the bias is SSDK_HT_ATTN_IN_B) and the weights of the
    * RMS norms over the whole query and key projections (qk_norm = 2) */
   SSDK_HT_ATTN_CONV_W,   /* [H D + G D + G V, pair_conv] */
-  SSDK_HT_ATTN_QK_NORM,  /* [H D + G D]: query weight, then key weight */
+  SSDK_HT_ATTN_QK_NORM,  /* [H D + G D]: query weight, then key weight; qk_norm = 3: [2, D] */
   /* delta rule: second halves of the low-rank projections */
   SSDK_HT_DELTA_A2,      /* [Hd Dd, d_decay_rank] */
   SSDK_HT_DELTA_G2,      /* [Hd Vd, d_gate_rank] */
@@ -379,6 +382,11 @@ enum {
   SSDK_HT_HC_IN,         /* [1 or 2, streams] */
   SSDK_HT_HC_OUT,        /* [1 or 2, streams] */
   SSDK_HT_HC_MIX,        /* [1 or 2, streams (from), streams (to)] */
+  /* SSDK_BLOCK_SERIAL_SANDWICH: norms on the sublayers' results (SSDK_HT_NORM and SSDK_HT_NORM2 are on their inputs) */
+  SSDK_HT_NORM_POST,     /* [width] */
+  SSDK_HT_NORM2_POST,    /* [width] */
+  SSDK_HT_ATTN_DIFF,     /* [4, D] lq1, lk1, lq2, lk2 of lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (maps = 2) */
+  SSDK_HT_RET_IN,        /* [2 H D + 2 H V, width]: retention q | k | v | g rows */
   SSDK_HT_COUNT
 };
 
@@ -396,7 +404,8 @@ typedef struct ssdk_hyb_layer_cfg {
   /* grouped-query attention (SSDK_MIX_ATTN_DELTA uses heads / dim / vdim / rot_dims / rot_base / attn_scale above) */
   int32_t kv_heads;                  /* key/value heads; query head h reads head h / (heads / kv_heads) */
   int32_t qk_norm;                   /* 1: q and k divided by their RMS over dim after the rotation; 2: RMS norm with a weight over the whole
-                                      * query (key) projection before the rotation */
+                                      * query (key) projection before the rotation; 3: RMS norm with one weight of size dim per head (and map)
+                                      * before the rotation */
   float   sink;                      /* constant added to the softmax denominator (0: plain softmax; 1: a sink of score 0) */
   float   yarn_factor;               /* 0: no frequency scaling; else YaRN with the three values below */
   float   yarn_original, yarn_fast, yarn_slow;
@@ -434,6 +443,14 @@ typedef struct ssdk_hyb_layer_cfg {
   int32_t d_decay_rank;              /* 0: one decay per head; r: one per head and key channel from a rank-r projection */
   int32_t d_gate_rank;               /* 0: output gate straight from h; r: from a rank-r projection */
   int32_t d_gate_act;                /* output gate of the delta rule: 0 silu, 1 sigmoid */
+  /* differential attention and the rest of SSDK_MIX_ATTENTION without a convolution */
+  int32_t maps;                      /* 1; 2: two queries per head and two keys per key/value head over the same values, joined as
+                                      * unit_rms(a1 - lambda a2) (1 - diff); the projections hold the maps of a head side by side */
+  float   diff;
+  int32_t keep_first;                /* keys at positions below keep_first stay visible beside the window (or chunk) */
+  float   wave_factor;               /* 0: none; else rotation frequencies scaled by wavelength with the three values below: kept under
+                                      * original / high, divided by factor over original / low, blended in between */
+  float   wave_low, wave_high, wave_original;
 } ssdk_hyb_layer_cfg;
 
 typedef struct ssdk_hyb_cfg {
@@ -446,7 +463,7 @@ typedef struct ssdk_hyb_cfg {
   int32_t block;             /* SSDK_BLOCK_* */
   float   norm_offset;       /* a norm scales by norm_offset + w: 1 for unit-offset weights, 0 for plain ones */
   float   embed_scale;       /* x = embed[token] * embed_scale */
-  float   residual_mult;     /* m of SSDK_BLOCK_SERIAL_POSTNORM */
+  float   residual_mult;     /* m of SSDK_BLOCK_SERIAL_POSTNORM and SSDK_BLOCK_SERIAL_SANDWICH */
   int32_t canon_taps;        /* SSDK_BLOCK_PARALLEL_ONE_NORM: taps of the sublayers' input convolutions (0: none) */
   int32_t gated_residual;    /* SSDK_BLOCK_PARALLEL_ONE_NORM: 1 = each sublayer's result is multiplied by sigmoid(W_g h + b) */
   int32_t streams;           /* SSDK_BLOCK_SERIAL_PRENORM: residual streams (0: one plain residual) */
@@ -458,8 +475,10 @@ typedef struct ssdk_hyb_engine* ssdk_hyb_handle;
 int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, ssdk_hyb_handle* out);
 int ssdk_hyb_destroy(ssdk_hyb_handle h);
 int ssdk_hyb_bind(ssdk_hyb_handle h, int layer, int tensor, const void* dev_ptr, int64_t rows, int64_t cols);
+/* decays of a retention layer's heads, each in [0, 1] (host pointer; the powers a chunk needs are made in double) */
+int ssdk_hyb_retention_decay(ssdk_hyb_handle h, int layer, const double* decay, int heads);
 /* caller-owned pools: paged cache (per latent-attention layer [num_blocks, block_size, kv_rank + rot_dim] T, per
- * grouped-query attention layer (SSDK_MIX_ATTN_DELTA, SSDK_MIX_ATTENTION) [num_blocks, block_size, G (D + V)] T: keys of all heads, then values; layers back to back), recurrent state (fp32, n_slots slots), workspace */
+ * grouped-query attention layer (SSDK_MIX_ATTN_DELTA, SSDK_MIX_ATTENTION) [num_blocks, block_size, G (D + V)] T (maps = 2: G (2 D + V)): keys of all heads, then values; layers back to back), recurrent state (fp32, n_slots slots), workspace */
 int64_t ssdk_hyb_cache_bytes(ssdk_hyb_handle h, int64_t num_blocks);
 int64_t ssdk_hyb_state_bytes(ssdk_hyb_handle h, int64_t n_slots);
 int64_t ssdk_hyb_workspace_bytes(ssdk_hyb_handle h);

@@ -2,19 +2,24 @@
 // models.  H query heads share G key/value heads (query head h reads head h / (H / G)); key size D and value size V are
 // independent.  A page row holds, for one token, the keys of all G heads (rotated, optionally unit-RMS) and then their
 // values: [G D | G V] of storage type T.  The softmax denominator may carry a constant (`sink`: 1 = a sink of score 0
-// that has no value) or a learned logit per query head; a key mask limits a query to its last `window` positions or to its own
-// chunk of positions.
+// that has no value) or a learned logit per query head; a key mask limits a query to its last `window` positions (beside the first
+// `keep` ones) or to its own chunk of positions.
+// Differential attention (maps = 2): every head has two queries and two keys over ONE value head; each map is an attention of its
+// own and the head is unit_rms(a1 - lambda a2) (1 - diff).  A page row then holds 2 keys per value head, [head, map] in turn; in the
+// kernels G counts keys (2 per value head), H queries, and query (head h, map i) belongs to key 2 (h / (H/G)) + i.
 //
 //   gqa_prep_kernel      per (token, head): rotation of the first rot_dims dimensions in adjacent or half-apart pairs (angle = position *
 //                        frequency in fp32, cos and sin times a constant), optional unit RMS over D; queries go to a
 //                        group-major buffer [G, M, H/G, D] (T), keys and raw values into the token's page row
 //   gqa_conv_prep_kernel the same behind a short convolution over time of q | k | v (bias, taps, history in the state slot) and an
 //                        optional weighted RMS norm over the whole query and key projection, one CTA per row
+//   gqa_head_prep_kernel no convolution: weighted RMS norm per head (and map), rotation, cache write, a warp per head of a row
 //   kv_gather_kernel     one sequence's pages -> contiguous keys [G, ctx_pad, D] and transposed values [G, V, ctx_pad]
 //   portions (>= 2 rows) two batched GEMMs per query block around sink_softmax_kernel (HybRun::gqa_attention)
 //   single-token rows    gqa_decode_partial_kernel (all decoding sequences in one launch, context split flash-decoding
 //                        style, fp32 weights) + gqa_decode_merge_kernel
 //                        (bf16 storage with 16-byte rows: the tensor-core forms of gqa_mma.cuh take both kinds of rows)
+//   diff_heads_kernel    group-major fp32 output of the two maps -> [M, H V] (T): the difference, its unit RMS, the constant
 //   attn_gate_kernel     group-major fp32 output x sigmoid(gate pre-activation) -> [M, H V] (T) for the output projection
 #pragma once
 #include "conv_scan.cuh"  // ConvArgs, conv_at
@@ -203,22 +208,143 @@ __global__ void gqa_conv_prep_kernel(const GqaConvPrepArgs p, const Ragged rg) {
   }
 }
 
-// grid (ctx_pad): position lo + j of sequence s -> keys[g][j][:] and vt[g][:][j]; zero from ctx up to ctx_pad
+// Rows of heads through a warp: dst[d] = (rotated) value of src[d] * inv * w[d] * mult, entries d and d + half of the first 2 half
+// ones turned by the row's angles (cs: half cosines, then half sines).  VEC = 4: D, half and both pointers are whole groups of four.
+template <typename OutT, typename T, int VEC>
+SSDK_DEVINL void head_row(const float* src, OutT* dst, int D, int half, const float* cs, const T* w, float inv, float mult, int lane) {
+  for (int d = lane * VEC; d < D; d += 32 * VEC) {
+    float v[VEC];
+    ld_vec<VEC>(src + d, v);
+    if (w) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] *= inv * ld_f<T>(w + d + e);
+    }
+    if (d < 2 * half) {
+      const bool first = d < half;
+      const int od = first ? d + half : d - half, i = first ? d : d - half;
+      float o[VEC];
+      ld_vec<VEC>(src + od, o);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        if (w) o[e] *= inv * ld_f<T>(w + od + e);
+        v[e] = first ? v[e] * cs[i + e] - o[e] * cs[half + i + e] : v[e] * cs[i + e] + o[e] * cs[half + i + e];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] *= mult;
+    st_row<OutT, VEC>(dst + d, v);
+  }
+}
+
+// the row's angles: cs[0 .. half) cosines, cs[half .. 2 half) sines of pos * f_i, times mult
+SSDK_DEVINL void row_angles(float* cs, int half, int pos, const float* inv_freq, float mult) {
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float sn, c;
+    sincosf((float)pos * inv_freq[i], &sn, &c);
+    cs[i] = c * mult; cs[half + i] = sn * mult;
+  }
+}
+
+struct GqaHeadPrepArgs {
+  GqaPrepArgs g;               // H queries and G keys (maps of them per head / value head); qk_norm, rot_half unused
+  const void* norm_w;          // [2, D] T: query weight, key weight of the RMS norm over a head's entries, or nullptr
+  int maps;
+};
+
+// grid (M, y): the warps of a row's CTAs take its H queries, G keys and G / maps values in turn.  dynamic shared memory: rot_dims floats
+template <typename T, int VEC>
+__global__ void gqa_head_prep_kernel(const GqaHeadPrepArgs p, const Ragged rg) {
+  SSDK_DYN_SMEM(float, hp_cs);
+  const int m = blockIdx.x, s = rg.tok_seq[m], pos = rg.pos0[s] + (m - rg.cu[s]), lane = threadIdx.x & 31;
+  const int H = p.g.H, G = p.g.G, Gv = G / p.maps, D = p.g.D, V = p.g.V, hpg = H / G, half = (p.g.inv_freq ? p.g.rot_dims : 0) >> 1;
+  row_angles(hp_cs, half, pos, p.g.inv_freq, p.g.rot_mult);
+  __syncthreads();
+  const int nw = blockDim.x >> 5;
+  const float* z = p.g.z + (size_t)m * p.g.ldz;
+  T* row = (T*)p.g.cache + page_row(rg, s, pos) * ((size_t)G * D + (size_t)Gv * V);
+  for (int u = blockIdx.y * nw + (threadIdx.x >> 5); u < H + G + Gv; u += gridDim.y * nw) {
+    if (u >= H + G) {
+      const int g = u - H - G;
+      head_row<T, T, VEC>(z + (size_t)(H + G) * D + (size_t)g * V, row + (size_t)G * D + (size_t)g * V, V, 0, hp_cs, (const T*)nullptr, 1.f, 1.f, lane);
+      continue;
+    }
+    const float* src = z + (size_t)u * D;
+    const T* w = p.norm_w ? (const T*)p.norm_w + (u < H ? 0 : D) : nullptr;
+    float inv = 1.f;
+    if (w) {
+      float ss = 0.f;
+      for (int d = lane * VEC; d < D; d += 32 * VEC) {
+        float v[VEC];
+        ld_vec<VEC>(src + d, v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ss = fmaf(v[e], v[e], ss);
+      }
+      inv = 1.0f / sqrtf(warp_sum(ss) / (float)D + p.g.eps);
+    }
+    T* dst;
+    if (u < H) {
+      const int hd = u / p.maps, g = hd / hpg * p.maps + u % p.maps;
+      dst = (T*)p.g.q + (((size_t)g * rg.M + m) * hpg + hd % hpg) * D;
+    } else {
+      dst = row + (size_t)(u - H) * D;
+    }
+    head_row<T, T, VEC>(src, dst, D, half, hp_cs, w, inv, 1.f, lane);
+  }
+}
+
+// grid (ctx_pad): the key of index lo - kept + j of sequence s (KeyMask) -> keys[g][j][:] and vt[g][:][j] (a value head once per map that
+// shares it); zero from ctx up to ctx_pad
 template <typename T>
 __global__ void kv_gather_kernel(const T* __restrict__ cache, T* __restrict__ keys, T* __restrict__ vt, const Ragged rg, int s,
-                                 int lo, int ctx, int ctx_pad, int G, int D, int V) {
+                                 int lo, int kept, int ctx, int ctx_pad, int G, int D, int V, int maps) {
   const int j = blockIdx.x;
-  const T* row = j < ctx ? cache + page_row(rg, s, lo + j) * (size_t)(G * (D + V)) : nullptr;
+  const size_t roww = (size_t)G * D + (size_t)(G / maps) * V;
+  const T* row = j < ctx ? cache + page_row(rg, s, key_position(lo - kept + j, lo, kept)) * roww : nullptr;
   for (int i = threadIdx.x; i < G * D; i += blockDim.x) {
     const int g = i / D, d = i - g * D;
     keys[((size_t)g * ctx_pad + j) * D + d] = row ? row[i] : T(0.f);
   }
-  for (int i = threadIdx.x; i < G * V; i += blockDim.x) vt[(size_t)i * ctx_pad + j] = row ? row[(size_t)G * D + i] : T(0.f);
+  for (int i = threadIdx.x; i < G * V; i += blockDim.x) {
+    const int g = i / V, v = i - g * V;
+    vt[(size_t)i * ctx_pad + j] = row ? row[(size_t)G * D + (size_t)(g / maps) * V + v] : T(0.f);
+  }
+}
+
+// ---- differential attention: what joins the two maps of a head ----
+struct DiffArgs {
+  const void* vec;    // [4, D] T: lq1, lk1, lq2, lk2
+  int D;
+  float diff, eps;
+};
+// lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, by every warp that needs it
+template <typename T>
+SSDK_DEVINL float diff_lambda(const DiffArgs& p) {
+  const T* v = (const T*)p.vec;
+  float a = 0.f, b = 0.f;
+  for (int d = threadIdx.x & 31; d < p.D; d += 32) {
+    a = fmaf(ld_f<T>(v + d), ld_f<T>(v + p.D + d), a);
+    b = fmaf(ld_f<T>(v + 2 * p.D + d), ld_f<T>(v + 3 * p.D + d), b);
+  }
+  return expf(warp_sum(a)) - expf(warp_sum(b)) + p.diff;
+}
+
+// o [G, M, H/G, V] fp32 (G keys = 2 per value head, H queries) -> y [M, (H / 2) V] (T), rows row0 ..; a warp per head.  grid (rows, ceil(H / 2 / warps))
+template <typename T>
+__global__ void diff_heads_kernel(const float* __restrict__ o, const DiffArgs p, T* __restrict__ y, int M, int H, int G, int V, int row0) {
+  const int m = row0 + blockIdx.x, hd = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31, hpg = H / G;
+  if (hd >= H / 2) return;
+  const float lam = diff_lambda<T>(p);
+  const float* a1 = o + (((size_t)(hd / hpg * 2) * M + m) * hpg + hd % hpg) * V;
+  const float* a2 = a1 + (size_t)M * hpg * V;
+  float ss = 0.f;
+  for (int v = lane; v < V; v += 32) { const float x = fmaf(-lam, a2[v], a1[v]); ss = fmaf(x, x, ss); }
+  const float f = (1.0f - p.diff) / sqrtf(warp_sum(ss) / (float)V + p.eps);
+  for (int v = lane; v < V; v += 32) st_f<T>(y + (size_t)m * (H / 2) * V + (size_t)hd * V + v, fmaf(-lam, a2[v], a1[v]) * f);
 }
 
 struct GqaDecodeArgs {
   const void* q;      // [G, M, H/G, D] T
-  const void* cache;  // [rows, G (D + V)] T
+  const void* cache;  // [rows, G D + (G / maps) V] T
   float* part;        // [n_seqs, H, splits, V + 2] fp32: unnormalised P V | running maximum | running sum
   void* y;            // [M, H V] T
   const float* gate;  // pre-activations of a sigmoid gate, gate[m * ld_gate + h V + v], or nullptr
@@ -226,7 +352,9 @@ struct GqaDecodeArgs {
   int H, G, D, V, splits;
   float scale, sink;
   const void* sinks;  // [H] T learned sink logits (they replace the constant), or nullptr
-  KeyMask mask;       // first key the token sees
+  KeyMask mask;       // keys the token sees
+  int maps;           // keys per value head (2: differential attention, joined by gqa_decode_merge_diff_kernel)
+  DiffArgs diff;
 };
 
 constexpr int kGqaDecWarps = 4;
@@ -253,7 +381,8 @@ __global__ void __launch_bounds__(kGqaDecWarps * 32) gqa_decode_partial_kernel(c
   __syncthreads();
   int k_lo, k_hi;
   decode_split(rg.pos0[s] + 1, p.mask, sp, p.splits, &k_lo, &k_hi);
-  const size_t roww = (size_t)G * (D + V);
+  const int first = p.mask.first(rg.pos0[s]), kept = p.mask.kept(first), gv = g / p.maps;
+  const size_t roww = (size_t)G * D + (size_t)(G / p.maps) * V;
   constexpr int kPer = 16 / (int)sizeof(T);
   const bool pool16 = ((uintptr_t)p.cache & 15) == 0;
   const bool vec_k = pool16 && D % kPer == 0 && roww % kPer == 0;
@@ -267,7 +396,7 @@ __global__ void __launch_bounds__(kGqaDecWarps * 32) gqa_decode_partial_kernel(c
   for (int k0 = k_lo + warp * 32; k0 < k_hi; k0 += kGqaDecWarps * 32) {
     const int key = k0 + lane;
     const bool ok = key < k_hi;
-    const size_t prow = ok ? page_row(rg, s, key) : 0;
+    const size_t prow = ok ? page_row(rg, s, key_position(key, first, kept)) : 0;
     float sc = -INFINITY;
     if (ok) {
       const T* kr = (const T*)p.cache + prow * roww + (size_t)g * D;
@@ -306,7 +435,7 @@ __global__ void __launch_bounds__(kGqaDecWarps * 32) gqa_decode_partial_kernel(c
         const int kk = kk0 + u;  // (a lane index below 32 in every case: nk <= 32 and kk0 is a multiple of 8)
         wk[u] = __shfl_sync(0xffffffffu, w, kk);
         const unsigned long long pr = __shfl_sync(0xffffffffu, (unsigned long long)prow, kk);
-        const T* vr = (const T*)p.cache + (size_t)pr * roww + (size_t)G * D + (size_t)g * V + c0;
+        const T* vr = (const T*)p.cache + (size_t)pr * roww + (size_t)G * D + (size_t)gv * V + c0;
         const bool live = kk < nk && c0 < V;
         if (live && vec_v) {
           ld_contig<T, VPL>(vr, f[u]);
@@ -372,6 +501,45 @@ __global__ void gqa_decode_merge_kernel(const GqaDecodeArgs p, const Ragged rg) 
     if (p.gate) a *= sigmoid_f(p.gate[(size_t)row * p.ld_gate + (size_t)hd * V + c]);
     st_f<T>(y + c, a);
   }
+}
+
+// grid (n_seqs, H / 2), differential attention: the two maps' splits are joined as above, then with each other.  dynamic shared memory: V floats
+template <typename T>
+__global__ void gqa_decode_merge_diff_kernel(const GqaDecodeArgs p, const Ragged rg) {
+  SSDK_DYN_SMEM(float, md_o);
+  __shared__ float w[2][kGqaMaxSplits];
+  __shared__ float red[33];
+  const int s = blockIdx.x, hd = blockIdx.y, row = rg.cu[s];
+  if (rg.cu[s + 1] - row != 1) return;
+  const int V = p.V, hpg = p.H / p.G;
+  const size_t stride = (size_t)p.splits * (V + 2);
+  const float* part = p.part + ((size_t)s * p.H + (size_t)(hd / hpg) * 2 * hpg + hd % hpg) * stride;   // (map 2: hpg heads on)
+  if (threadIdx.x < 64) {   // a warp per map, a lane per split: its weight, normalised (the second map's times -lambda)
+    const int j = threadIdx.x & 31, map = threadIdx.x >> 5;
+    const float* pm = part + map * hpg * stride + (size_t)j * (V + 2) + V;
+    const float lam = diff_lambda<T>(p.diff);
+    const float mj = j < p.splits ? pm[0] : -INFINITY, m = warp_max(mj);
+    const float e = mj == -INFINITY ? 0.f : expf(mj - m);
+    const float den = warp_sum(j < p.splits ? e * pm[1] : 0.f);
+    w[map][j] = e / den * (map ? -lam : 1.f);
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < V; c += blockDim.x) {
+    float a = 0.f, b = 0.f;
+#pragma unroll 4
+    for (int j = 0; j < p.splits; ++j) {
+      a = fmaf(w[0][j], part[(size_t)j * (V + 2) + c], a);
+      b = fmaf(w[1][j], part[hpg * stride + (size_t)j * (V + 2) + c], b);
+    }
+    a += b;
+    md_o[c] = a;
+    ss = fmaf(a, a, ss);
+  }
+  ss = block_sum(ss, red);
+  const float f = (1.0f - p.diff.diff) / sqrtf(ss / (float)V + p.diff.eps);
+  T* y = (T*)p.y + (size_t)row * (p.H / 2) * V + (size_t)hd * V;
+  for (int c = threadIdx.x; c < V; c += blockDim.x) st_f<T>(y + c, md_o[c] * f);   // (the thread's own entries)
 }
 
 // o [G, M, H/G, V] fp32 (group-major) and gate pre-activations gz[m * ldg + h * V + v] -> y [M, H V] (T) = o * sigmoid(gz), rows row0 ..

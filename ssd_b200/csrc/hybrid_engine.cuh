@@ -1,7 +1,7 @@
 // hybrid_engine.cuh — host side of the layered (hybrid) model family: the layer program, the pools it addresses
 // (paged latent cache, recurrent-state slots, workspace) and the ragged forward that prefill portions and single decode
 // tokens share.  Included by engine.cu; uses its Launcher / error helpers.  Kernels: layer_ops.cuh, linear.cuh,
-// recurrent.cuh, latent_attention.cuh, moe.cuh; the sampler is sample_kernel of sampling.cuh.
+// recurrent.cuh, retention.cuh, latent_attention.cuh, moe.cuh; the sampler is sample_kernel of sampling.cuh.
 #pragma once
 #include "conv_scan.cuh"
 #include "gqa_attention.cuh"
@@ -11,6 +11,7 @@
 #include "linear.cuh"
 #include "moe.cuh"
 #include "recurrent.cuh"
+#include "retention.cuh"
 
 struct HybTensor {
   const void* p = nullptr;
@@ -26,6 +27,7 @@ struct HybLayer {
   size_t cache_rows_before = 0;  // sum of the row widths of the latent layers before this one
   float* inv_freq = nullptr; // device, [rot_dims / 2]
   float rot_mult = 1.0f;     // factor on cos and sin (frequency scaling)
+  float* decay_pow = nullptr; // retention: device, [heads, kRetChunk + 1] powers of the heads' decays
 };
 
 struct ssdk_hyb_engine {
@@ -56,7 +58,8 @@ struct ssdk_hyb_engine {
   // widths of the shared buffers (elements per row)
   int w_p0 = 0, w_p1 = 0, w_p2 = 0, w_t0 = 0, w_t1 = 0, w_e = 0, w_top = 0, w_ff2 = 0, w_ff = 0, w_sff2 = 0, w_sff = 0;
   size_t delta_floats = 0; float* delta_rec = nullptr;   // chunk records of the delta rule
-  bool any_wkv = false, any_pair = false, any_ffn = false;
+  size_t ret_floats = 0; float* ret_rec = nullptr;       // chunk records of the retention
+  bool any_wkv = false, any_pair = false, any_ffn = false, vec_state = false;   // vec_state: slots are whole 16-byte pieces
   int* h_meta = nullptr;     // pinned staging of the step's integers
   // tcgen05 path of the dense bf16 products: TMA descriptors by (pointer, rows, K, box rows), split-K partials
   bool use_tc = true;
@@ -65,6 +68,7 @@ struct ssdk_hyb_engine {
   bool use_tc_scores = true;    // score GEMM of latent-attention portions on the tcgen05 GEMM (SSDK_HYB_TC_SCORES=0: mma.sync tile)
   bool use_gqa_mma = true;      // grouped-query attention on the tensor cores (SSDK_HYB_GQA_MMA=0: GEMMs around a softmax, CUDA-core decode)
   bool use_tc_glu = true;       // gated feed-forward's activation in the epilogue of the tcgen05 GEMM (SSDK_HYB_TC_GLU=0: a kernel of its own)
+  bool use_retention_mma = true; // retention's chunks on the tensor cores (SSDK_HYB_RETENTION_MMA=0: fp32 FMA)
   bool use_decode_mma = true;   // its tensor-core form for bf16 storage (SSDK_HYB_DECODE_MMA=0: the CUDA-core form)
   std::map<std::tuple<const void*, int64_t, int, int, int>, CUtensorMap> tmaps;
   float* partials = nullptr; size_t partial_floats = 0;
@@ -117,7 +121,10 @@ static int hyb_derive(ssdk_hyb_engine* e) {
     const ssdk_hyb_layer_cfg& c = L.c;
     const int H = c.heads, D = c.dim, V = c.vdim;
     if (H < 1 || D < 1) return fail("hybrid layer: heads / dim must be positive");
-    if (c.window < 0 || c.chunk < 0) return fail("hybrid layer: window %d, chunk %d", c.window, c.chunk);
+    if (c.window < 0 || c.chunk < 0 || c.keep_first < 0) return fail("hybrid layer: window %d, chunk %d, first %d keys kept", c.window, c.chunk, c.keep_first);
+    if (c.keep_first && c.mixer == SSDK_MIX_LATENT_ATTN) return fail("latent attention: kept first keys are built for grouped-query attention");
+    if (c.maps < 1 || c.maps > 2 || (c.maps == 2 && c.mixer != SSDK_MIX_ATTENTION)) return fail("hybrid layer: %d maps (2: the attention mixer)", c.maps);
+    if (c.qk_norm == 3 && c.mixer != SSDK_MIX_ATTENTION) return fail("the weighted norm per head is built for the attention mixer");
     if (g.block == SSDK_BLOCK_SERIAL_PRENORM && (c.mixer == SSDK_MIX_WKV || c.mixer == SSDK_MIX_MLSTM))
       return fail("wkv and mlstm are built for parallel blocks");
     if (g.block == SSDK_BLOCK_PARALLEL_ONE_NORM) {
@@ -193,6 +200,7 @@ static int hyb_derive(ssdk_hyb_engine* e) {
       L.state_off = soff;
       soff += (size_t)Hd * Dd * Vd + (size_t)(c.conv - 1) * Cd;
       L.attn_hist_off = soff;
+      e->vec_state = true;
       if (c.pair_conv > 1) soff += (size_t)(c.pair_conv - 1) * Ca;
       L.cache_row = (size_t)G * (D + V);
       L.cache_rows_before = crow;
@@ -211,33 +219,46 @@ static int hyb_derive(ssdk_hyb_engine* e) {
       if (c.rot_dims < 0 || c.rot_dims > D || (c.rot_dims & 1)) return fail("attention: rot dims %d of %d", c.rot_dims, D);
       if (V > 256 * 4) return fail("attention: value size %d too large", V);
       if (c.conv < 1) return fail("attention: %d taps", c.conv);
-      if (c.qk_norm) return fail("attention: query and key norms are built for the pair");
-      if (ssdk::gqa_conv_prep_smem(H * D + G * (D + V), c.rot_dims) > 200 * 1024) return fail("attention: too many projected channels");
-      const long long Nqkv = (long long)H * D + (long long)G * D + (long long)G * V;
+      if (c.qk_norm && c.qk_norm != 3) return fail("attention: the mixer's query and key norm is the weighted one per head");
+      if ((c.qk_norm == 3 || c.maps == 2) && (c.conv != 1 || !c.rot_half)) return fail("attention: norms per head and two maps are built for half-apart rotation without a convolution");
+      if (c.maps == 2 && (c.learned_sink || c.sink > 0.f)) return fail("attention: two maps have no sink");
+      if (c.qk_norm != 3 && ssdk::gqa_conv_prep_smem(H * D + G * (D + V), c.rot_dims) > 200 * 1024) return fail("attention: too many projected channels");
+      const long long Hq = (long long)H * c.maps, Gk = (long long)G * c.maps;   // queries and keys of a token
+      const long long Nqkv = Hq * D + Gk * D + (long long)G * V;
       soff += (size_t)(c.conv - 1) * Nqkv;
-      L.cache_row = (size_t)G * (D + V);
+      L.cache_row = (size_t)Gk * D + (size_t)G * V;
       L.cache_rows_before = crow;
       crow += L.cache_row;
-      up(e->w_p0, Nqkv); up(e->w_p2, (long long)H * V); up(e->w_t0, (long long)H * V);
-      up(e->w_qcat, (long long)H * D); up(e->w_key, (long long)G * D); up(e->w_kr, (long long)G * V); up(e->w_lh, H);
+      up(e->w_p0, Nqkv); up(e->w_p2, Hq * V); up(e->w_t0, (long long)H * V);
+      up(e->w_qcat, Hq * D); up(e->w_key, Gk * D); up(e->w_kr, Gk * V); up(e->w_lh, Hq);
+    } else if (c.mixer == SSDK_MIX_RETENTION) {
+      if (V < 1 || c.rot_dims < 0 || c.rot_dims > D || (c.rot_dims & 1)) return fail("retention: %d x %d, rot dims %d", D, V, c.rot_dims);
+      if (ssdk::ret_decode_smem(D, V) > 200 * 1024) return fail("retention: head sizes %d x %d too large", D, V);
+      soff = align_up(soff, 4);
+      L.state_off = soff;
+      soff += (size_t)H * D * V;
+      e->vec_state = true;
+      up(e->w_p0, 2LL * H * D + 2LL * H * V); up(e->w_p1, (long long)H * V); up(e->w_p2, 2LL * H * D); up(e->w_t1, (long long)H * V);
+      e->ret_floats = std::max(e->ret_floats, ((size_t)g.max_tokens / ssdk::kRetChunk + g.max_seqs + 1) * H * D * V);
     } else {
       return fail("hybrid layer: unknown mixer %d", c.mixer);
     }
     if (c.mlp == SSDK_MLP_GLU) {
       if (c.ff < 1) return fail("dense feed-forward: ff %d", c.ff);
-      if (e->cfg.block != SSDK_BLOCK_SERIAL_POSTNORM && e->cfg.block != SSDK_BLOCK_SERIAL_PRENORM) return fail("the gated dense feed-forward is built for serial blocks");
+      if (e->cfg.block != SSDK_BLOCK_SERIAL_POSTNORM && e->cfg.block != SSDK_BLOCK_SERIAL_PRENORM && e->cfg.block != SSDK_BLOCK_SERIAL_SANDWICH) return fail("the gated dense feed-forward is built for serial blocks");
       if (c.ff_act != SSDK_ACT_SILU && c.ff_act != SSDK_ACT_GELU_TANH) return fail("dense feed-forward: unknown gate activation %d", c.ff_act);
       up(e->w_p0, 2LL * c.ff); up(e->w_t0, c.ff);
     } else if (c.mlp == SSDK_MLP_FFN) {
       if (c.ff < 1) return fail("dense feed-forward: ff %d", c.ff);
-      if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM || e->cfg.block == SSDK_BLOCK_SERIAL_PRENORM) return fail("the ungated feed-forward is built for parallel blocks");
+      if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM || e->cfg.block == SSDK_BLOCK_SERIAL_PRENORM || e->cfg.block == SSDK_BLOCK_SERIAL_SANDWICH) return fail("the ungated feed-forward is built for parallel blocks");
       if (c.ff_act != SSDK_ACT_RELU2 && c.ff_act != SSDK_ACT_GELU_TANH && c.ff_act != SSDK_ACT_SILU && c.ff_act != SSDK_ACT_POLYNORM)
         return fail("dense feed-forward: unknown activation %d", c.ff_act);
       up(e->w_sff2, c.ff); up(e->w_sff, c.ff);   // it shares the shared expert's buffers: no layer has both
       e->any_ffn = true;
     } else if (c.mlp == SSDK_MLP_MOE) {
       const int Et = c.experts + c.identity;   // router outputs: real experts, then identity experts
-      if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM || e->cfg.block == SSDK_BLOCK_SERIAL_PRENORM) return fail("the mixture of experts is built for parallel blocks");
+      if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM || e->cfg.block == SSDK_BLOCK_SERIAL_PRENORM) return fail("the mixture of experts is built for parallel blocks and for serial ones with norms on both sides");
+      if (c.identity && e->cfg.block == SSDK_BLOCK_SERIAL_SANDWICH) return fail("identity experts are built for parallel blocks");
       if (c.experts < 1 || c.identity < 0 || Et > kRouterMaxE) return fail("moe: 1 <= experts (+ identity) <= %d", kRouterMaxE);
       if (c.groups < 1 || Et % c.groups) return fail("moe: %d router outputs do not form %d equal groups", Et, c.groups);
       if (c.keep < 1 || c.keep > c.groups) return fail("moe: keep %d of %d groups", c.keep, c.groups);
@@ -255,7 +276,7 @@ static int hyb_derive(ssdk_hyb_engine* e) {
       return fail("hybrid layer: unknown feed-forward kind %d", c.mlp);
     }
   }
-  e->slot_floats = e->any_pair ? align_up(soff, 4) : soff;
+  e->slot_floats = e->vec_state ? align_up(soff, 4) : soff;
   e->cache_row_total = crow;
   return 0;
 }
@@ -277,6 +298,7 @@ static int64_t hyb_carve(ssdk_hyb_engine* e, uint8_t* base) {
   e->p1 = (float*)take(cap * e->w_p1 * 4);
   e->p2 = (float*)take(cap * e->w_p2 * 4);
   e->delta_rec = (float*)take(e->delta_floats * 4);
+  e->ret_rec = (float*)take(e->ret_floats * 4);
   e->t0 = take(cap * e->w_t0 * es);
   e->t1 = take(cap * e->w_t1 * es);
   e->mix_out = (float*)take(cap * g.width * 4);
@@ -540,7 +562,10 @@ struct HybRun {
     int n = 0;
     *ctx_max = 0;
     for (int s = 0; s < rg.n_seqs; ++s)
-      if (h_cu[s + 1] - h_cu[s] == 1) { ++n; *ctx_max = std::max(*ctx_max, h_pos0[s] + 1 - mask.first(h_pos0[s])); }
+      if (h_cu[s + 1] - h_cu[s] == 1) {
+        const int first = mask.first(h_pos0[s]);
+        ++n; *ctx_max = std::max(*ctx_max, h_pos0[s] + 1 - first + mask.kept(first));
+      }
     return n;
   }
 
@@ -549,7 +574,7 @@ struct HybRun {
     const int H = c.heads, D = c.dim, V = c.vdim, R = c.rot_dim, KR = c.kv_rank, QR = c.q_rank, W = e->cfg.width;
     const bool own = c.kv_from < 0;   // the layer fills a pool of its own (else it reads an earlier layer's rows of this step and before)
     const int Nq = H * (D + R), Nkv = own ? KR + R : 0;
-    const ssdk::KeyMask mask = {c.window, c.chunk};
+    const ssdk::KeyMask mask = {c.window, c.chunk, 0};
     CKI(check_tensor(Lr, SSDK_HT_LAT_UKT, (int64_t)H * KR, D, "uk^T")); CKI(check_tensor(Lr, SSDK_HT_LAT_UV, (int64_t)H * V, KR, "uv"));
     CKI(check_tensor(Lr, SSDK_HT_MIX_OUT, W, (int64_t)H * V, "mix.o"));
     if (own) CKI(check_tensor(Lr, SSDK_HT_LAT_KVNORM, KR, 1, "dkv.norm"));
@@ -648,7 +673,7 @@ struct HybRun {
         // scores: keys are the 128-row operand, (query, head) rows the tokens
         CKI(lin(qrows, Wd, krows, Wd, e->att_s, cb, rows, cb, Wd, false, 1, 0, 0, 0, tc_attn));
         CKI(L.go(ssdk::sink_softmax_kernel<T>, dim3(rows), dim3(256), 0, (const float*)e->att_s, (T*)e->att_p,
-                 (const T*)sink, H, cb, p0 + q0, c.attn_scale, rows, 0.f, lo + kb, mask));
+                 (const T*)sink, H, cb, p0 + q0, c.attn_scale, rows, 0.f, lo + kb, 0, mask));
         T* o_rows = (T*)e->t0 + (size_t)(r0 + q0) * H * KR;
         if (tc_attn && tc_ok(e->att_p, cb, lat_t, ctx_pad, KR, KR, cb)) {
           // P C: the transposed latents [kv_rank, ctx_pad] are the 128-row operand, read with the row stride of the gather
@@ -861,12 +886,14 @@ struct HybRun {
   // grouped-query attention over the layer's page pool: z holds q | k | v (fp32) -> y [M, H V] (T), times
   // sigmoid(gate pre-activation) if gate is given; og [G, M, H/G, V] fp32 is scratch.  conv (optional): z's
   // columns pass through a bias and a short convolution over time first, norm_w: then through a norm over the whole query
-  // and key projection
+  // and key projection; norm_w without conv: through a norm per head.  Two maps per head (differential attention): z holds maps H
+  // queries and maps G keys, y the H joined heads
   int gqa_attention(HybLayer& Lr, const float* z, int ldz, void* y, float* og, const float* gate, int ld_gate, const void* sinks = nullptr, const ssdk::ConvArgs* conv = nullptr,
                     const void* norm_w = nullptr) {
     const ssdk_hyb_layer_cfg& c = Lr.c;
-    const int H = c.heads, G = c.kv_heads, D = c.dim, V = c.vdim, hpg = H / G;
-    const ssdk::KeyMask mask = {c.window, c.chunk};
+    const int maps = c.maps, H = c.heads * maps, G = c.kv_heads * maps, D = c.dim, V = c.vdim, hpg = H / G;   // queries, keys, queries per key
+    const ssdk::KeyMask mask = {c.window, c.chunk, c.keep_first};
+    const ssdk::DiffArgs diff = {Lr.t[SSDK_HT_ATTN_DIFF].p, D, c.diff, e->cfg.eps};
     const float sink_const = sinks ? 0.f : c.sink;
     if (!e->cache) return fail("hybrid: attention cache not bound");
     uint8_t* pool = e->cache + (size_t)e->num_blocks * e->cfg.block_size * Lr.cache_rows_before * e->esz;
@@ -886,12 +913,21 @@ struct HybRun {
       else if (vec) CKI(L.go(ssdk::gqa_conv_prep_kernel<T, 4, 2>, grid, block, smem, cp, rg));
       else CKI(L.go(ssdk::gqa_conv_prep_kernel<T, 1, 1>, grid, block, smem, cp, rg));
       if (conv->taps > 1) CKI(L.go(ssdk::conv_state_kernel<T>, dim3(rg.n_seqs, (conv->C + 255) / 256), dim3(256), 0, *conv, rg));
+    } else if (norm_w || maps > 1) {
+      ssdk::GqaHeadPrepArgs hp;
+      hp.g = pa; hp.norm_w = norm_w; hp.maps = maps;
+      const bool vec = D % 4 == 0 && V % 4 == 0 && c.rot_dims % 8 == 0 && ldz % 4 == 0 && (((uintptr_t)z | (uintptr_t)pool | (uintptr_t)e->qcat) & 15) == 0;
+      const int units = H + G + G / maps, ys = std::max(1, std::min((units + 7) / 8, 2 * num_sms() / M));   // few rows: a row's heads over several CTAs
+      const size_t smem = (size_t)c.rot_dims * 4;
+      if (vec) CKI(L.go(ssdk::gqa_head_prep_kernel<T, 4>, dim3(M, ys), dim3(256), smem, hp, rg));
+      else CKI(L.go(ssdk::gqa_head_prep_kernel<T, 1>, dim3(M, ys), dim3(256), smem, hp, rg));
     } else {
       CKI(L.go(ssdk::gqa_prep_kernel<T>, dim3(M, H + G), dim3(32), 0, pa, rg));
     }
     // tensor-core forms: bf16, heads of whole 16-byte pieces up to 128 wide, up to 16 query heads per key/value head
     const bool mma = !kF32 && e->use_gqa_mma && D % 8 == 0 && V % 8 == 0 && std::max(D, V) <= 128 && hpg <= 16 && ((uintptr_t)pool & 15) == 0;
-    const int ks = std::max(D, V) <= 32 ? 2 : (std::max(D, V) <= 64 ? 4 : 8), vt = 2 * ks;
+    const int ks = std::max(D, V) <= 32 ? 2 : (std::max(D, V) <= 64 || (maps == 2 && D <= 64) ? 4 : 8);
+    const int vt = V <= 64 && ks < 8 ? 2 * ks : 16;   // (two maps: value heads are often twice as wide as the keys)
     bool fused_decode = false;
     {
       int ctx_max = 0;
@@ -907,17 +943,19 @@ struct HybRun {
         if (splits >= 1) {
           ssdk::GqaDecodeArgs da;
           da.q = e->qcat; da.cache = pool; da.part = e->att_s; da.y = y; da.gate = gate; da.ld_gate = ld_gate; da.H = H; da.G = G; da.D = D; da.V = V; da.splits = splits;
-          da.scale = c.attn_scale; da.sink = sink_const; da.sinks = sinks; da.mask = mask;
+          da.scale = c.attn_scale; da.sink = sink_const; da.sinks = sinks; da.mask = mask; da.maps = maps; da.diff = diff;
           const dim3 grid(rg.n_seqs, H, splits), block(ssdk::kGqaDecWarps * 32), mgrid(rg.n_seqs, G, splits), mblock(128);
           const size_t smem = ssdk::gqa_decode_smem(D, V), msmem = ssdk::gqa_decode_mma_smem(ks, vt, V);
           if (mma && ks == 2) CKI(L.go(ssdk::gqa_decode_mma_kernel<2, 4>, mgrid, mblock, msmem, da, rg));
+          else if (mma && ks == 4 && vt == 16) CKI(L.go(ssdk::gqa_decode_mma_kernel<4, 16>, mgrid, mblock, msmem, da, rg));
           else if (mma && ks == 4) CKI(L.go(ssdk::gqa_decode_mma_kernel<4, 8>, mgrid, mblock, msmem, da, rg));
           else if (mma) CKI(L.go(ssdk::gqa_decode_mma_kernel<8, 16>, mgrid, mblock, msmem, da, rg));
           else if (vpl <= 1) CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 1>, grid, block, smem, da, rg));
           else if (vpl <= 2) CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 2>, grid, block, smem, da, rg));
           else if (vpl <= 4) CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 4>, grid, block, smem, da, rg));
           else CKI(L.go(ssdk::gqa_decode_partial_kernel<T, 8>, grid, block, smem, da, rg));
-          CKI(L.go(ssdk::gqa_decode_merge_kernel<T>, dim3(rg.n_seqs, H), dim3(V <= 64 ? 64 : 128), 0, da, rg));
+          if (maps == 2) CKI(L.go(ssdk::gqa_decode_merge_diff_kernel<T>, dim3(rg.n_seqs, H / 2), dim3(V <= 64 ? 64 : 128), (size_t)V * 4, da, rg));
+          else CKI(L.go(ssdk::gqa_decode_merge_kernel<T>, dim3(rg.n_seqs, H), dim3(V <= 64 ? 64 : 128), 0, da, rg));
           fused_decode = true;
         }
       }
@@ -928,43 +966,70 @@ struct HybRun {
       if (n_max > 1) {
         ssdk::GqaPortionArgs fa;
         fa.q = e->qcat; fa.cache = pool; fa.y = y; fa.gate = gate; fa.ld_gate = ld_gate; fa.H = H; fa.G = G; fa.D = D; fa.V = V;
-        fa.scale = c.attn_scale; fa.sink = sink_const; fa.sinks = sinks; fa.mask = mask;
-        const dim3 grid((n_max * hpg + ssdk::kGpRows - 1) / ssdk::kGpRows, G, rg.n_seqs), block(ssdk::kGpWarps * 32);
-        const size_t smem = 2 * ssdk::gm_tile_bytes(ks, vt);
-        if (ks == 2) CKI(L.go(ssdk::gqa_portion_mma_kernel<2, 4>, grid, block, smem, fa, rg));
-        else if (ks == 4) CKI(L.go(ssdk::gqa_portion_mma_kernel<4, 8>, grid, block, smem, fa, rg));
-        else CKI(L.go(ssdk::gqa_portion_mma_kernel<8, 16>, grid, block, smem, fa, rg));
+        fa.scale = c.attn_scale; fa.sink = sink_const; fa.sinks = sinks; fa.mask = mask; fa.diff = diff;
+        const int tile = ssdk::kGpRows / maps;   // (query, head) rows of a CTA
+        const dim3 grid((n_max * hpg + tile - 1) / tile, G / maps, rg.n_seqs), block(ssdk::kGpWarps * 32);
+        const size_t smem = 2 * ssdk::gm_tile_bytes(ks, vt, maps);
+        if (maps == 2) {
+          if (ks == 2) CKI(L.go(ssdk::gqa_portion_mma_kernel<2, 4, 2>, grid, block, smem, fa, rg));
+          else if (ks == 4 && vt == 8) CKI(L.go(ssdk::gqa_portion_mma_kernel<4, 8, 2>, grid, block, smem, fa, rg));
+          else if (ks == 4) CKI(L.go(ssdk::gqa_portion_mma_kernel<4, 16, 2>, grid, block, smem, fa, rg));
+          else CKI(L.go(ssdk::gqa_portion_mma_kernel<8, 16, 2>, grid, block, smem, fa, rg));
+        } else if (ks == 2) CKI(L.go(ssdk::gqa_portion_mma_kernel<2, 4, 1>, grid, block, smem, fa, rg));
+        else if (ks == 4) CKI(L.go(ssdk::gqa_portion_mma_kernel<4, 8, 1>, grid, block, smem, fa, rg));
+        else CKI(L.go(ssdk::gqa_portion_mma_kernel<8, 16, 1>, grid, block, smem, fa, rg));
       }
     }
     for (int s = 0; s < rg.n_seqs; ++s) {
       const int r0 = h_cu[s], n = h_cu[s + 1] - r0, p0 = h_pos0[s];
       if (n == 1 ? fused_decode : mma) continue;
-      const int lo = mask.first(p0), ctx = p0 + n - lo, ctx_pad = (ctx + 7) / 8 * 8;   // keys lo .. p0 + n - 1
-      CKI(L.go(ssdk::kv_gather_kernel<T>, dim3(ctx_pad), dim3(128), 0, (const T*)pool, (T*)e->keys, (T*)e->lat_t, rg, s, lo, ctx, ctx_pad, G, D, V));
+      int lo = mask.first(p0), kept = mask.kept(lo), ctx = p0 + n - lo + kept, ctx_pad = (ctx + 7) / 8 * 8;   // the kept keys, then lo .. p0 + n - 1
+      const bool per_block = mask.keep > 0;   // kept keys must lie beside a block's own: every query block is gathered by itself
+      auto gather = [&]() {
+        return L.go(ssdk::kv_gather_kernel<T>, dim3(ctx_pad), dim3(128), 0, (const T*)pool, (T*)e->keys, (T*)e->lat_t, rg, s, lo, kept, ctx, ctx_pad, G, D, V, maps);
+      };
+      if (!per_block) CKI(gather());
       const int qb = (int)std::max<size_t>(1, e->att_elems / ((size_t)H * ctx_pad));
       for (int q0 = 0, nq; q0 < n; q0 += nq) {
         nq = mask_block(mask, p0 + q0, n - q0, qb);
+        if (per_block) {
+          lo = mask.first(p0 + q0); kept = mask.kept(lo); ctx = p0 + q0 + nq - lo + kept; ctx_pad = (ctx + 7) / 8 * 8;
+          CKI(gather());
+        }
         const int rows = nq * hpg, kb = (mask.first(p0 + q0) - lo) / 8 * 8;
-        const int cb = (p0 + q0 + nq - lo - kb + 7) / 8 * 8;   // gathered keys kb .. kb + cb - 1 are what this block can see
+        const int cb = (p0 + q0 + nq - lo + kept - kb + 7) / 8 * 8;   // gathered keys kb .. kb + cb - 1 are what this block can see
         const T* qrows = (const T*)e->qcat + (size_t)(r0 + q0) * hpg * D;
         CKI(lin(qrows, D, (const T*)e->keys + (size_t)kb * D, D, e->att_s, cb, rows, cb, D, false, G, (long long)M * hpg * D, (long long)ctx_pad * D,
                 (long long)rows * cb, false));
         CKI(L.go(ssdk::sink_softmax_kernel<T>, dim3(G * rows), dim3(256), 0, (const float*)e->att_s, (T*)e->att_p, (const T*)sinks, hpg, cb,
-                 p0 + q0, c.attn_scale, rows, sink_const, lo + kb, mask));
+                 p0 + q0, c.attn_scale, rows, sink_const, lo + kb, kept, mask));
         CKI(lin(e->att_p, cb, (const T*)e->lat_t + kb, ctx_pad, og + (size_t)(r0 + q0) * hpg * V, V, rows, V, cb, false, G, (long long)rows * cb,
                 (long long)V * ctx_pad, (long long)M * hpg * V, false));
       }
-      CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(n), dim3(256), 0, (const float*)og, gate, ld_gate, (T*)y, M, H, G, V, r0));
+      if (maps == 2) CKI(L.go(ssdk::diff_heads_kernel<T>, dim3(n, (H / 2 + 3) / 4), dim3(128), 0, (const float*)og, diff, (T*)y, M, H, G, V, r0));
+      else CKI(L.go(ssdk::attn_gate_kernel<T>, dim3(n), dim3(256), 0, (const float*)og, gate, ld_gate, (T*)y, M, H, G, V, r0));
     }
     return 0;
   }
 
   // grouped-query attention alone: stacked q | k | v projection, its bias, a short convolution over time on every channel
-  // (history in the state slot), rotation, window, learned sink, output projection
+  // (history in the state slot), rotation, window, learned sink, output projection; or, without bias and convolution, a norm per head
+  // before the rotation and two maps per head
   int attention(HybLayer& Lr) {
     const ssdk_hyb_layer_cfg& c = Lr.c;
-    const int W = e->cfg.width, H = c.heads, G = c.kv_heads, D = c.dim, V = c.vdim, taps = c.conv, Nqkv = H * D + G * D + G * V;
-    CKI(check_tensor(Lr, SSDK_HT_ATTN_IN, Nqkv, W, "attention.in")); CKI(check_tensor(Lr, SSDK_HT_CONV_W, Nqkv, taps, "attention.conv"));
+    const int W = e->cfg.width, H = c.heads, G = c.kv_heads, D = c.dim, V = c.vdim, taps = c.conv, Nqkv = c.maps * (H + G) * D + G * V;
+    CKI(check_tensor(Lr, SSDK_HT_ATTN_IN, Nqkv, W, "attention.in"));
+    if (c.qk_norm == 3 || c.maps == 2) {
+      CKI(check_tensor(Lr, SSDK_HT_MIX_OUT, W, (int64_t)H * V, "mix.o"));
+      if (c.qk_norm == 3) CKI(check_tensor(Lr, SSDK_HT_ATTN_QK_NORM, 2, D, "q.norm|k.norm"));
+      if (c.maps == 2) CKI(check_tensor(Lr, SSDK_HT_ATTN_DIFF, 4, D, "lq1|lk1|lq2|lk2"));
+      if (c.learned_sink) CKI(check_tensor(Lr, SSDK_HT_ATTN_SINK, H, 1, "sink"));
+      CKI(lin(hin, W, Lr.t[SSDK_HT_ATTN_IN].p, W, e->p0, Nqkv, M, Nqkv, W));
+      CKI(gqa_attention(Lr, e->p0, Nqkv, e->t0, e->p2, nullptr, 0, c.learned_sink ? Lr.t[SSDK_HT_ATTN_SINK].p : nullptr, nullptr,
+                        c.qk_norm == 3 ? Lr.t[SSDK_HT_ATTN_QK_NORM].p : nullptr));
+      return lin(e->t0, H * V, Lr.t[SSDK_HT_MIX_OUT].p, H * V, e->mix_out, W, M, W, H * V);
+    }
+    CKI(check_tensor(Lr, SSDK_HT_CONV_W, Nqkv, taps, "attention.conv"));
     CKI(check_tensor(Lr, SSDK_HT_MIX_OUT, W, (int64_t)H * V, "mix.o"));
     if (Lr.t[SSDK_HT_ATTN_IN_B].p) CKI(check_tensor(Lr, SSDK_HT_ATTN_IN_B, Nqkv, 1, "attention.in.b"));
     if (c.learned_sink) CKI(check_tensor(Lr, SSDK_HT_ATTN_SINK, H, 1, "sink"));
@@ -974,6 +1039,59 @@ struct HybRun {
     ca.hist = e->state + Lr.state_off; ca.slot_stride = e->slot_floats; ca.C = Nqkv; ca.taps = taps;
     CKI(gqa_attention(Lr, e->p0, Nqkv, e->t0, e->p2, nullptr, 0, c.learned_sink ? Lr.t[SSDK_HT_ATTN_SINK].p : nullptr, &ca));
     return lin(e->t0, H * V, Lr.t[SSDK_HT_MIX_OUT].p, H * V, e->mix_out, W, M, W, H * V);
+  }
+
+  // linear attention with a fixed decay per head: stacked q | k | v | g projection, rotation, chunks, norm per head, silu gate
+  int retention(HybLayer& Lr) {
+    const ssdk_hyb_layer_cfg& c = Lr.c;
+    const int W = e->cfg.width, H = c.heads, D = c.dim, V = c.vdim, Nin = 2 * H * (D + V);
+    CKI(check_tensor(Lr, SSDK_HT_RET_IN, Nin, W, "retention.in")); CKI(check_tensor(Lr, SSDK_HT_MIX_OUT, W, (int64_t)H * V, "mix.o"));
+    if (!Lr.decay_pow) return fail("retention: the heads' decays were not set");
+    CKI(lin(hin, W, Lr.t[SSDK_HT_RET_IN].p, W, e->p0, Nin, M, Nin, W));
+    ssdk::RetentionArgs a;
+    a.z = e->p0; a.ldz = Nin; a.qk = e->p2; a.pw = Lr.decay_pow; a.chunks = e->ret_rec; a.S = e->state + Lr.state_off; a.slot_stride = e->slot_floats;
+    a.inv_freq = c.rot_dims >= 2 ? Lr.inv_freq : nullptr; a.rot_dims = c.rot_dims; a.y = e->t1; a.H = H; a.D = D; a.V = V;
+    a.k_scale = 1.0f / sqrtf((float)D); a.eps = e->cfg.eps;
+    a.vec = D % 4 == 0 && V % 4 == 0 && c.rot_dims % 8 == 0;   // (buffers, slots and the layer's state start on 16-byte boundaries)
+    int n_dec = 0, n_max = 0;
+    for (int s = 0; s < rg.n_seqs; ++s) { n_dec += h_cu[s + 1] - h_cu[s] == 1; n_max = std::max(n_max, h_cu[s + 1] - h_cu[s]); }
+    const bool mma = !kF32 && e->use_retention_mma && std::max(D, V) <= 128;
+    a.o = !mma && n_max > 1 ? e->p1 : nullptr;   // the FMA form leaves o of all rows for the norm below
+    if (n_dec > 0) {
+      const size_t smem = ssdk::ret_decode_smem(D, V);
+      if (a.vec) CKI(L.go(ssdk::retention_decode_kernel<T, 4>, dim3(rg.n_seqs, H), dim3(ssdk::kRetDecWarps * 32), smem, a, rg));
+      else CKI(L.go(ssdk::retention_decode_kernel<T, 1>, dim3(rg.n_seqs, H), dim3(ssdk::kRetDecWarps * 32), smem, a, rg));
+    }
+    if (n_max > 1) {
+      const int ys = std::max(1, std::min((2 * H + 7) / 8, 2 * num_sms() / M)), nc = (n_max + ssdk::kRetChunk - 1) / ssdk::kRetChunk;
+      const size_t rsm = (size_t)c.rot_dims * 4, hdv = (size_t)H * D * V;
+      if (a.vec) CKI(L.go(ssdk::retention_prep_kernel<4>, dim3(M, ys), dim3(256), rsm, a, rg));
+      else CKI(L.go(ssdk::retention_prep_kernel<1>, dim3(M, ys), dim3(256), rsm, a, rg));
+      const int ks = D <= 32 ? 2 : (D <= 64 ? 4 : 8), vt = V <= 32 ? 4 : (V <= 64 ? 8 : 16);
+      const dim3 cgrid(nc, H, rg.n_seqs), block(256);
+      if (mma) CKI(retention_mma(a, ks, vt, cgrid, false));
+      else CKI(L.go(ssdk::retention_chunk_state_any_kernel, dim3(nc, H * ((D + 63) / 64) * ((V + 63) / 64), rg.n_seqs), block, 0, a, rg));
+      if (a.vec) CKI(L.go(ssdk::retention_state_scan_kernel<4>, dim3(rg.n_seqs, (unsigned)((hdv / 4 + 255) / 256)), block, 0, a, rg));
+      else CKI(L.go(ssdk::retention_state_scan_kernel<1>, dim3(rg.n_seqs, (unsigned)((hdv + 255) / 256)), block, 0, a, rg));
+      if (mma) {
+        CKI(retention_mma(a, ks, vt, cgrid, true));
+      } else {
+        CKI(L.go(ssdk::retention_chunk_out_any_kernel, dim3(nc, H * ((V + 63) / 64), rg.n_seqs), block, 0, a, rg));
+        CKI(L.go(ssdk::head_rmsnorm_gate_kernel<T, 0>, dim3(M, H), dim3(std::min(256, (V + 31) / 32 * 32)), 0, (const float*)e->p1,
+                 (const float*)e->p0 + 2 * H * D + H * V, Nin, (const T*)nullptr, (T*)e->t1, H, V, e->cfg.eps));
+      }
+    }
+    return lin(e->t1, H * V, Lr.t[SSDK_HT_MIX_OUT].p, H * V, e->mix_out, W, M, W, H * V);
+  }
+  template <int KS, int VT>
+  int retention_mma_go(const ssdk::RetentionArgs& a, dim3 grid, bool out) {
+    if (out) return L.go(ssdk::retention_chunk_out_mma_kernel<KS, VT>, grid, dim3(256), ssdk::ret_out_mma_smem(KS, VT), a, rg);
+    return L.go(ssdk::retention_chunk_state_mma_kernel<KS, VT>, grid, dim3(256), ssdk::ret_state_mma_smem(KS, VT), a, rg);
+  }
+  int retention_mma(const ssdk::RetentionArgs& a, int ks, int vt, dim3 grid, bool out) {
+    if (ks == 2) return vt == 4 ? retention_mma_go<2, 4>(a, grid, out) : (vt == 8 ? retention_mma_go<2, 8>(a, grid, out) : retention_mma_go<2, 16>(a, grid, out));
+    if (ks == 4) return vt == 4 ? retention_mma_go<4, 4>(a, grid, out) : (vt == 8 ? retention_mma_go<4, 8>(a, grid, out) : retention_mma_go<4, 16>(a, grid, out));
+    return vt == 4 ? retention_mma_go<8, 4>(a, grid, out) : (vt == 8 ? retention_mma_go<8, 8>(a, grid, out) : retention_mma_go<8, 16>(a, grid, out));
   }
 
   // attention beside a gated delta rule on the same input: ONE stacked input projection; results in mix_out and mix2
@@ -1087,6 +1205,7 @@ struct HybRun {
       case SSDK_MIX_RGLRU: return rglru(Lr);
       case SSDK_MIX_SELECTIVE: return selective(Lr);
       case SSDK_MIX_ATTENTION: return attention(Lr);
+      case SSDK_MIX_RETENTION: return retention(Lr);
       default: return attn_delta(Lr);
     }
   }
@@ -1173,7 +1292,54 @@ struct HybRun {
     return stream_step(Lr, 1, next, 0);
   }
 
+  // ---- serial blocks with a norm before and after each sublayer: x += m * post1(mixer(norm1(x))); x += m * post2(ff(norm2(x))) ----
+  int check_sandwich_layer(const HybLayer& Lr) {
+    const int W = e->cfg.width;
+    CKI(check_tensor(Lr, SSDK_HT_NORM, W, 1, "norm1")); CKI(check_tensor(Lr, SSDK_HT_NORM_POST, W, 1, "norm1b"));
+    if (Lr.c.mlp == SSDK_MLP_NONE) return 0;
+    CKI(check_tensor(Lr, SSDK_HT_NORM2, W, 1, "norm2"));
+    return check_tensor(Lr, SSDK_HT_NORM2_POST, W, 1, "norm2b");
+  }
+  // the result of a sublayer (q 0: mixer, 1: feed-forward) joins the residual; the next sublayer's input follows in the same pass
+  int sandwich_step(HybLayer& Lr, int q, const void* next_w) {
+    const int W = e->cfg.width;
+    ssdk::SandwichArgs a = {};
+    a.x = e->x; a.post_w = Lr.t[q ? SSDK_HT_NORM2_POST : SSDK_HT_NORM_POST].p; a.next_w = next_w; a.h = next_w ? e->h : nullptr;
+    a.width = W; a.eps = e->cfg.eps; a.offset = e->cfg.norm_offset; a.mult = e->cfg.residual_mult;
+    if (q && Lr.c.mlp == SSDK_MLP_MOE) {
+      a.routed = e->eo; a.apos = e->apos; a.wts = e->wts; a.top = Lr.c.top;
+      if (Lr.c.shared_ff > 0) {
+        a.shared = e->so;
+        const int ld = (Lr.c.expert_glu ? 2 : 1) * Lr.c.shared_ff;
+        if (Lr.c.shared_gate) { a.sg = e->sz + ld; a.ld_sg = ld + 1; }
+      }
+    } else {
+      a.y = e->mix_out;
+    }
+    const dim3 grid(M), block(256);
+    if (W % 4 == 0) return L.go(ssdk::sandwich_step_kernel<T, 4>, grid, block, (size_t)W * 4, a);
+    return L.go(ssdk::sandwich_step_kernel<T, 1>, grid, block, (size_t)W * 4, a);
+  }
+  int sandwich_layer(HybLayer& Lr, int li) {
+    const ssdk_hyb_cfg& g = e->cfg;
+    const HybLayer* next = li + 1 < g.n_layers ? &e->layers[li + 1] : nullptr;
+    CKI(check_sandwich_layer(Lr));
+    if (next) CKI(check_sandwich_layer(*next));
+    const void* next_w = next ? next->t[SSDK_HT_NORM].p : nullptr;
+    if (li == 0)
+      CKI(L.go(ssdk::offset_rmsnorm_kernel<T>, dim3(M), dim3(256), 0, (const float*)e->x, (const T*)Lr.t[SSDK_HT_NORM].p, (T*)e->h, (const int*)nullptr,
+               g.width, g.eps, g.norm_offset, (const T*)nullptr, (T*)nullptr));
+    if (Lr.c.mixer == SSDK_MIX_ATTN_DELTA) return fail("the attention pair is built for serial blocks with one norm per sublayer");
+    hin = fin = e->h;
+    CKI(run_mixer(Lr));
+    if (Lr.c.mlp == SSDK_MLP_NONE) return sandwich_step(Lr, 0, next_w);
+    CKI(sandwich_step(Lr, 0, Lr.t[SSDK_HT_NORM2].p));
+    CKI(Lr.c.mlp == SSDK_MLP_MOE ? moe(Lr) : glu(Lr));
+    return sandwich_step(Lr, 1, next_w);
+  }
+
   int layer(HybLayer& Lr, int li) {
+    if (e->cfg.block == SSDK_BLOCK_SERIAL_SANDWICH) return sandwich_layer(Lr, li);
     if (e->cfg.block == SSDK_BLOCK_SERIAL_POSTNORM) return serial_layer(Lr);
     if (e->cfg.block == SSDK_BLOCK_SERIAL_PRENORM) return prenorm_layer(Lr, li);
     const int W = e->cfg.width;
@@ -1220,7 +1386,7 @@ struct HybRun {
       }
     }
     if (Lr.c.mixer == SSDK_MIX_ATTN_DELTA) return fail("the attention pair is built for serial blocks");
-    if (Lr.c.mixer == SSDK_MIX_ATTENTION && !one) return fail("the attention mixer is built for one-norm and serial pre-norm blocks");
+    if (Lr.c.mixer == SSDK_MIX_ATTENTION && !one) return fail("the attention mixer is built for one-norm and serial blocks");
     CKI(run_mixer(Lr));
     ca.x = e->x; ca.mix = e->mix_out; ca.ls1 = scales ? Lr.t[SSDK_HT_LS_MIX].p : nullptr; ca.width = W;
     if (Lr.c.mlp == SSDK_MLP_MOE) {
@@ -1276,10 +1442,31 @@ static int hyb_smem_attrs(ssdk_hyb_engine* e) {
   SSDK_PREP_ATTR(4, 4) SSDK_PREP_ATTR(4, 2) SSDK_PREP_ATTR(1, 1)
 #undef SSDK_PREP_ATTR
 #define SSDK_GQA_ATTR(KS, VT) \
-  CK(cudaFuncSetAttribute(ssdk::gqa_portion_mma_kernel<KS, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_portion_mma_kernel<KS, VT, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
   CK(cudaFuncSetAttribute(ssdk::gqa_decode_mma_kernel<KS, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
-  SSDK_GQA_ATTR(2, 4) SSDK_GQA_ATTR(4, 8) SSDK_GQA_ATTR(8, 16)
+  SSDK_GQA_ATTR(2, 4) SSDK_GQA_ATTR(4, 8) SSDK_GQA_ATTR(4, 16) SSDK_GQA_ATTR(8, 16)
 #undef SSDK_GQA_ATTR
+  CK(cudaFuncSetAttribute(ssdk::gqa_portion_mma_kernel<2, 4, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::gqa_portion_mma_kernel<4, 8, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::gqa_portion_mma_kernel<8, 16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+#define SSDK_RET_ATTR(KS, VT) \
+  CK(cudaFuncSetAttribute(ssdk::retention_chunk_state_mma_kernel<KS, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::retention_chunk_out_mma_kernel<KS, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  SSDK_RET_ATTR(2, 4) SSDK_RET_ATTR(2, 8) SSDK_RET_ATTR(2, 16) SSDK_RET_ATTR(4, 4) SSDK_RET_ATTR(4, 8) SSDK_RET_ATTR(4, 16)
+  SSDK_RET_ATTR(8, 4) SSDK_RET_ATTR(8, 8) SSDK_RET_ATTR(8, 16)
+#undef SSDK_RET_ATTR
+#define SSDK_ROW_ATTR(T) \
+  CK(cudaFuncSetAttribute(ssdk::retention_decode_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::retention_decode_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::sandwich_step_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::sandwich_step_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_head_prep_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_head_prep_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_decode_merge_diff_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  SSDK_ROW_ATTR(bf16) SSDK_ROW_ATTR(float)
+#undef SSDK_ROW_ATTR
+  CK(cudaFuncSetAttribute(ssdk::retention_prep_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
+  CK(cudaFuncSetAttribute(ssdk::retention_prep_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
 #define SSDK_STREAM_ATTR(SM, VEC) \
   CK(cudaFuncSetAttribute(ssdk::stream_step_kernel<bf16, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
   CK(cudaFuncSetAttribute(ssdk::stream_step_kernel<float, SM, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
@@ -1372,7 +1559,7 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
   if (cfg->width < 1 || cfg->vocab < 1 || cfg->n_layers < 1) return fail("ssdk_hyb_create: bad sizes");
   if (cfg->dtype != SSDK_DT_F32 && cfg->dtype != SSDK_DT_BF16) return fail("ssdk_hyb_create: unknown dtype %d", cfg->dtype);
   if (cfg->block != SSDK_BLOCK_PARALLEL_PRENORM && cfg->block != SSDK_BLOCK_SERIAL_POSTNORM && cfg->block != SSDK_BLOCK_PARALLEL_TWO_NORMS &&
-      cfg->block != SSDK_BLOCK_PARALLEL_ONE_NORM && cfg->block != SSDK_BLOCK_SERIAL_PRENORM) return fail("ssdk_hyb_create: unknown block kind %d", cfg->block);
+      cfg->block != SSDK_BLOCK_PARALLEL_ONE_NORM && cfg->block != SSDK_BLOCK_SERIAL_PRENORM && cfg->block != SSDK_BLOCK_SERIAL_SANDWICH) return fail("ssdk_hyb_create: unknown block kind %d", cfg->block);
   if (cfg->streams < 0 || cfg->streams > ssdk::kMaxStreams || (cfg->streams && cfg->block != SSDK_BLOCK_SERIAL_PRENORM))
     return fail("ssdk_hyb_create: %d residual streams (serial pre-norm blocks take up to %d)", cfg->streams, ssdk::kMaxStreams);
   if ((size_t)cfg->width * 4 > kScanSmemMax) return fail("ssdk_hyb_create: width %d too large", cfg->width);
@@ -1388,6 +1575,7 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
   e->use_tc = env_int("SSDK_HYB_TCGEN05", 1) != 0;
   e->use_decode_attn = env_int("SSDK_HYB_DECODE_ATTN", 1) != 0;
   e->use_decode_mma = env_int("SSDK_HYB_DECODE_MMA", 1) != 0;
+  e->use_retention_mma = env_int("SSDK_HYB_RETENTION_MMA", 1) != 0;
   e->use_gqa_mma = env_int("SSDK_HYB_GQA_MMA", 1) != 0;
   e->use_tc_glu = env_int("SSDK_HYB_TC_GLU", 1) != 0;
   e->use_tc_scores = env_int("SSDK_HYB_TC_SCORES", 1) != 0;
@@ -1396,7 +1584,7 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
   for (int i = 0; i < cfg->n_layers; ++i) e->layers[i].c = layers[i];
   if (hyb_derive(e) != 0) { delete e; return -1; }
   for (auto& L : e->layers) {
-    if ((L.c.mixer != SSDK_MIX_LATENT_ATTN && L.c.mixer != SSDK_MIX_ATTN_DELTA && L.c.mixer != SSDK_MIX_ATTENTION) || L.c.rot_dims < 2) continue;
+    if ((L.c.mixer != SSDK_MIX_LATENT_ATTN && L.c.mixer != SSDK_MIX_ATTN_DELTA && L.c.mixer != SSDK_MIX_ATTENTION && L.c.mixer != SSDK_MIX_RETENTION) || L.c.rot_dims < 2) continue;
     const int half = L.c.rot_dims / 2;
     std::vector<float> f(half);
     const double dims = (double)L.c.rot_dims, base = (double)L.c.rot_base;
@@ -1414,6 +1602,18 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
       }
       L.rot_mult = (float)(0.1 * log(factor) + 1.0);
     }
+    if (L.c.wave_factor > 0.f) {
+      // by wavelength: shorter than original / high kept, longer than original / low slowed by `factor`, a blend of both in between
+      const double kPi = 3.14159265358979323846, factor = (double)L.c.wave_factor, orig = (double)L.c.wave_original;
+      const double low = (double)L.c.wave_low, high = (double)L.c.wave_high;
+      for (int i = 0; i < half; ++i) {
+        const double fi = pow(base, -2.0 * i / dims), turns = orig * fi / (2.0 * kPi);   // = original / wavelength
+        double g = fi;
+        if (turns < low) g = fi / factor;
+        else if (turns < high) { const double s = (turns - low) / (high - low); g = (1.0 - s) * fi / factor + s * fi; }
+        f[i] = (float)g;
+      }
+    }
     if (cudaMalloc(&L.inv_freq, half * 4) != cudaSuccess ||
         cudaMemcpy(L.inv_freq, f.data(), half * 4, cudaMemcpyHostToDevice) != cudaSuccess) {
       delete e;
@@ -1429,7 +1629,10 @@ int ssdk_hyb_create(const ssdk_hyb_cfg* cfg, const ssdk_hyb_layer_cfg* layers, s
 int ssdk_hyb_destroy(ssdk_hyb_handle e) {
   if (!e) return 0;
   for (auto& L : e->layers)
+  {
     if (L.inv_freq) cudaFree(L.inv_freq);
+    if (L.decay_pow) cudaFree(L.decay_pow);
+  }
   if (e->h_meta) cudaFreeHost(e->h_meta);
   delete e;
   return 0;
@@ -1448,6 +1651,22 @@ int ssdk_hyb_bind(ssdk_hyb_handle e, int layer, int tensor, const void* dev_ptr,
   }
   if (layer < 0 || layer >= e->cfg.n_layers) return fail("ssdk_hyb_bind: layer %d out of range", layer);
   e->layers[layer].t[tensor] = t;
+  return 0;
+}
+
+int ssdk_hyb_retention_decay(ssdk_hyb_handle e, int layer, const double* decay, int heads) {
+  if (!e || !decay) return fail("ssdk_hyb_retention_decay: null argument");
+  if (layer < 0 || layer >= e->cfg.n_layers) return fail("ssdk_hyb_retention_decay: layer %d out of range", layer);
+  HybLayer& L = e->layers[layer];
+  if (L.c.mixer != SSDK_MIX_RETENTION || heads != L.c.heads) return fail("ssdk_hyb_retention_decay: layer %d has no %d retention heads", layer, heads);
+  const int n = ssdk::kRetChunk + 1;
+  std::vector<float> pw((size_t)heads * n);
+  for (int h = 0; h < heads; ++h) {
+    if (!(decay[h] >= 0.0 && decay[h] <= 1.0)) return fail("ssdk_hyb_retention_decay: decay %g of head %d", decay[h], h);
+    for (int i = 0; i < n; ++i) pw[(size_t)h * n + i] = (float)pow(decay[h], (double)i);
+  }
+  if (!L.decay_pow && cudaMalloc(&L.decay_pow, pw.size() * 4) != cudaSuccess) return fail("ssdk_hyb_retention_decay: no device memory");
+  if (cudaMemcpy(L.decay_pow, pw.data(), pw.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) return fail("ssdk_hyb_retention_decay: copy failed");
   return 0;
 }
 

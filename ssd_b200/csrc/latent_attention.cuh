@@ -111,37 +111,45 @@ __global__ void latent_gather_kernel(const T* __restrict__ cache, T* __restrict_
   }
 }
 
-// Which keys a causal query sees: those at first(pos) .. pos.  A sliding window keeps the last `window` positions, chunks are
-// counted from the sequence's start and end at the query's own chunk; 0 = no window, no chunks.
+// Which keys a causal query sees: those at first(pos) .. pos, and those before position `keep`.  A sliding window keeps the last
+// `window` positions, chunks are counted from the sequence's start and end at the query's own chunk; 0 = no window, no chunks,
+// no kept first keys.
+// Kernels walk a query's keys as one run of indices: index i >= first stands for position i, and the kept keys before `first` sit
+// right in front of it, at first - kept .. first - 1 (without kept keys an index IS a position).
 struct KeyMask {
-  int window, chunk;
+  int window, chunk, keep;
   __host__ __device__ __forceinline__ int first(int pos) const {
     int f = window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0;
     if (chunk > 0) { const int c = pos / chunk * chunk; f = c > f ? c : f; }
     return f;
   }
-  __host__ __device__ __forceinline__ bool any() const { return window > 0 || chunk > 0; }
+  // kept keys in front of `first`
+  __host__ __device__ __forceinline__ int kept(int first) const { return keep < first ? keep : first; }
 };
+// index -> position (see KeyMask)
+SSDK_DEVINL int key_position(int i, int first, int kept) { return i >= first ? i : i - (first - kept); }
 
 // Softmax with a sink over the score rows of one query block.  The rows come in `batches` of rows_per_batch (one batch
 // per key/value head of grouped-query attention; a single batch for latent attention); inside a batch row r is
-// (query q0 + r / H, head r % H) with H the heads that share the batch's keys.  Column j of a row is the key at position
-// key_first + j; the query at position pos sees the keys at mask.first(pos) .. pos.
+// (query q0 + r / H, head r % H) with H the heads that share the batch's keys.  Column j of a row is the key of index
+// key_first - kept + j (KeyMask); the query at position pos sees the keys at mask.first(pos) .. pos and those before mask.keep.
 // sc [rows, ld] fp32 raw dot products -> pr [rows, ld] (T) weights, zero outside the visible range and in the padding.
 // The sink is a learned per-head logit (`sink`, indexed batch * H + head) or, without one, the constant sink_const added
 // to the denominator (0: plain softmax); it joins the maximum, is not scaled and contributes nothing to the output.
 template <typename T>
 __global__ void sink_softmax_kernel(const float* __restrict__ sc, T* __restrict__ pr, const T* __restrict__ sink, int H, int ld,
-                                    int pos_first, float scale, int rows_per_batch, float sink_const, int key_first, KeyMask mask) {
+                                    int pos_first, float scale, int rows_per_batch, float sink_const, int key_first, int kept, KeyMask mask) {
   __shared__ float red[33];
   const int r = blockIdx.x, batch = r / rows_per_batch, rb = r - batch * rows_per_batch;
   const int h = rb % H, pos = pos_first + rb / H;
-  const int n = pos - key_first + 1;                                             // columns [j0, n) are the keys this row sees
-  const int j0 = max(0, mask.first(pos) - key_first);
+  const int n = pos - key_first + kept + 1;                                      // columns [j0, n) are the keys this row sees,
+  const int j0 = max(0, mask.first(pos) - key_first + kept);
+  const int jk = min(min(mask.keep, j0), n);                                     // and [0, jk), the kept first ones
   const float* srow = sc + (size_t)r * ld;
   const float sk = sink ? ld_f<T>(sink + batch * H + h) : (sink_const > 0.f ? logf(sink_const) : -INFINITY);
   float mx = sk;
   for (int j = j0 + threadIdx.x; j < n; j += blockDim.x) mx = fmaxf(mx, srow[j] * scale);
+  for (int j = threadIdx.x; j < jk; j += blockDim.x) mx = fmaxf(mx, srow[j] * scale);
   __syncthreads();
   mx = warp_max(mx);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = mx;
@@ -150,10 +158,11 @@ __global__ void sink_softmax_kernel(const float* __restrict__ sc, T* __restrict_
   for (int w = 1; w < (int)(blockDim.x >> 5); ++w) mx = fmaxf(mx, red[w]);
   float sum = 0.f;
   for (int j = j0 + threadIdx.x; j < n; j += blockDim.x) sum += expf(srow[j] * scale - mx);
+  for (int j = threadIdx.x; j < jk; j += blockDim.x) sum += expf(srow[j] * scale - mx);
   sum = block_sum(sum, red) + expf(sk - mx);
   const float inv = 1.0f / sum;
   for (int j = threadIdx.x; j < ld; j += blockDim.x)
-    st_f<T>(pr + (size_t)r * ld + j, (j >= j0 && j < n) ? expf(srow[j] * scale - mx) * inv : 0.f);
+    st_f<T>(pr + (size_t)r * ld + j, ((j >= j0 && j < n) || j < jk) ? expf(srow[j] * scale - mx) * inv : 0.f);
 }
 
 // ---- single-token (decode) rows: one launch over all such sequences, the context split flash-decoding style ----
@@ -169,10 +178,10 @@ struct LatentDecodeArgs {
   KeyMask mask;       // first key the token sees
 };
 
-// keys [k_lo, k_hi) of split j (of `splits`) for a single token at position ctx - 1
+// key indices [k_lo, k_hi) of split j (of `splits`) for a single token at position ctx - 1
 SSDK_DEVINL void decode_split(int ctx, const KeyMask& mask, int j, int splits, int* k_lo, int* k_hi) {
-  const int first = mask.first(ctx - 1), per = (ctx - first + splits - 1) / splits;
-  *k_lo = first + j * per;
+  const int first = mask.first(ctx - 1), begin = first - mask.kept(first), per = (ctx - begin + splits - 1) / splits;
+  *k_lo = begin + j * per;
   *k_hi = min(ctx, *k_lo + per);
 }
 

@@ -17,6 +17,8 @@
 //                             an RMS norm and a factor each) is written back, x_t = sum_s mix[s, t] x_s + out[t] y, and the next
 //                             sublayer's input norm(sum_t in[t] x_t) is made from the new streams while they are in registers
 //   stream_sum_kernel         the sum of the streams
+//   sandwich_step_kernel      serial block with a norm before AND after a sublayer: x += mult * norm(y), h = norm(x), y the mixer's
+//                             result or a mixture of experts' (sum_k w_k expert_k + shared, made here)
 //   block_combine_kernel      parallel block: x += ls1 * g1 * mixer + ls2 * g2 * (sum_k w_k expert_k + sigmoid(sg) * shared + b);
 //                             ls1, ls2, sg, b are optional (1, 1, no gate, 0), and so are the per-token, per-channel residual
 //                             gates g = sigmoid(pre-activation + bias); an identity expert's output is the feed-forward's
@@ -228,10 +230,10 @@ __global__ void head_rmsnorm_gate_kernel(const float* __restrict__ o, const floa
   for (int j = threadIdx.x; j < V; j += blockDim.x) ss = fmaf(orow[j], orow[j], ss);
   ss = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(ss / (float)V + eps);
-  for (int j = threadIdx.x; j < V; j += blockDim.x) {
+  for (int j = threadIdx.x; j < V; j += blockDim.x) {   // (w may be nullptr: no channel weight)
     const float gz = g[(size_t)m * ldg + hd * V + j];
     const float ga = GATE == 0 ? gz * sigmoid_f(gz) : sigmoid_f(gz);
-    st_f<T>(y + (size_t)m * H * V + hd * V + j, orow[j] * inv * ld_f<T>(w + hd * V + j) * ga);
+    st_f<T>(y + (size_t)m * H * V + hd * V + j, orow[j] * inv * (w ? ld_f<T>(w + hd * V + j) : 1.f) * ga);
   }
 }
 
@@ -375,6 +377,18 @@ template <int VEC> SSDK_DEVINL void st_vec(float* p, const float* f) {
   else *p = f[0];
 }
 
+// VEC floats -> storage type (VEC = 4: p is aligned to 4 elements)
+template <typename T, int VEC> SSDK_DEVINL void st_row(T* p, const float* f) {
+  if constexpr (VEC == 4 && sizeof(T) == 2) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(f[0], f[1]), hi = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+  } else if constexpr (VEC == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    st_f<T>(p, f[0]);
+  }
+}
+
 // grid (M).  SM >= S: streams held in registers; VEC = 4 needs a width that is a multiple of 4.  dynamic shared memory: width floats
 template <typename T, int SM, int VEC>
 __global__ void stream_step_kernel(const StreamStepArgs p) {
@@ -459,6 +473,88 @@ __global__ void stream_step_kernel(const StreamStepArgs p) {
 #pragma unroll
       for (int e = 0; e < VEC; ++e) st_f<T>(h + e, ss_u[c + e]);
     }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------- norms on both sides
+// x[m] += mult * norm(y[m]; post_w), then h[m] = norm(x[m]; next_w): the step between two sublayers in one pass.  y is either a
+// tensor or the output of a mixture of experts: sum_k wts[k] routed[apos[k]] (+ sigmoid(sg)) * shared.
+struct SandwichArgs {
+  float* x;              // [M, width] residual, updated in place
+  const float* y;        // [M, width] the sublayer's result, or nullptr (mixture of experts)
+  const float* routed;   // [M * top, width] expert outputs in assignment order
+  const int* apos;       // [M * top] row of (token, k) in `routed`
+  const float* wts;      // [M * top] routing weights
+  int top;
+  const float* shared;   // [M, width] shared expert's output, or nullptr
+  const float* sg;       // pre-activation of the shared expert's gate: sg[m * ld_sg], or nullptr (no gate)
+  int ld_sg;
+  const void* post_w;    // [width] T weight of the norm on y
+  const void* next_w;    // [width] T weight of the norm of the next sublayer's input
+  void* h;               // [M, width] T that input, or nullptr: no sublayer follows
+  int width;
+  float eps, offset, mult;
+};
+
+// grid (M).  VEC = 4 needs a width that is a multiple of 4.  dynamic shared memory: width floats
+template <typename T, int VEC>
+__global__ void sandwich_step_kernel(const SandwichArgs p) {
+  SSDK_DYN_SMEM(float, sw_u);
+  __shared__ float red[33];
+  const int m = blockIdx.x, W = p.width;
+  const size_t row = (size_t)m * W;
+  const float sgate = (p.shared && p.sg) ? sigmoid_f(p.sg[(size_t)m * p.ld_sg]) : 1.f;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float y[VEC];
+    if (p.y) {
+      ld_vec<VEC>(p.y + row + c, y);
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y[e] = 0.f;
+      for (int k = 0; k < p.top; ++k) {
+        const size_t a = (size_t)m * p.top + k;
+        float v[VEC];
+        ld_vec<VEC>(p.routed + (size_t)p.apos[a] * W + c, v);
+        const float w = p.wts[a];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = fmaf(w, v[e], y[e]);
+      }
+      if (p.shared) {
+        float v[VEC];
+        ld_vec<VEC>(p.shared + row + c, v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = fmaf(sgate, v[e], y[e]);
+      }
+    }
+    st_vec<VEC>(sw_u + c, y);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(y[e], y[e], ss);
+  }
+  ss = block_sum(ss, red);
+  float inv = 1.0f / sqrtf(ss / (float)W + p.eps);
+  ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {   // the thread's own entries of the shared row
+    float y[VEC], x[VEC];
+    ld_vec<VEC>(sw_u + c, y);
+    ld_vec<VEC>(p.x + row + c, x);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      x[e] = fmaf(p.mult, y[e] * inv * (p.offset + ld_f<T>((const T*)p.post_w + c + e)), x[e]);
+      ss = fmaf(x[e], x[e], ss);
+    }
+    st_vec<VEC>(p.x + row + c, x);
+    st_vec<VEC>(sw_u + c, x);
+  }
+  if (!p.h) return;
+  ss = block_sum(ss, red);
+  inv = 1.0f / sqrtf(ss / (float)W + p.eps);
+  for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
+    float x[VEC];
+    ld_vec<VEC>(sw_u + c, x);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) x[e] *= inv * (p.offset + ld_f<T>((const T*)p.next_w + c + e));
+    st_row<T, VEC>((T*)p.h + row + c, x);
   }
 }
 

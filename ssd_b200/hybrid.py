@@ -1,4 +1,4 @@
-"""Layered ("hybrid") models: a program of layers, each one token mixer + an optional feed-forward.  Five designs are
+"""Layered ("hybrid") models: a program of layers, each one token mixer + an optional feed-forward.  Six designs are
 served through this module, told apart by config.json's `"architecture"`:
 
     Pikavik   parallel pre-norm blocks (mixer and mixture-of-experts feed-forward read the same normed input, unit-offset
@@ -26,6 +26,13 @@ served through this module, told apart by config.json's `"architecture"`:
               rule with a decay per key channel (low-rank decay and output-gate projections), both results RMS-normed
               and averaged; dense silu-GLU feed-forward; scaled logits
 
+    Vegilix   serial blocks with a norm before and after each sublayer (x += m * norm(sublayer(norm x)), unit-offset norm
+              weights); some layers run several times in a row with the same weights, each pass with a cache or state of its
+              own; mixers `attention` (differential: two softmax maps per head over the same values, a weighted RMS norm per
+              head and map, rotate-half rotation with frequencies scaled by wavelength, a sliding window beside kept first
+              keys) and `retention` (linear attention with a fixed decay per head); silu-GLU experts whose weights are the
+              softmax over the chosen logits, plus an ungated shared expert
+
     HybridSpec     what config.json (and, for sizes it does not list, the checkpoint's tensor shapes) says
     load_hybrid_weights   safetensors -> device tensors in the packed layout libssdk's ssdk_hyb_bind expects
     HybridRunner   owner of the device state behind one ssdk_hyb handle (weights, paged latent cache, recurrent-state
@@ -47,7 +54,7 @@ import torch
 from . import lib as L
 
 MIXERS = {"wkv": L.MIX_WKV, "mlstm": L.MIX_MLSTM, "latent_attention": L.MIX_LATENT_ATTN, "rglru": L.MIX_RGLRU,
-          "mamba1": L.MIX_SELECTIVE, "parallel": L.MIX_ATTN_DELTA, "attention": L.MIX_ATTENTION}
+          "mamba1": L.MIX_SELECTIVE, "parallel": L.MIX_ATTN_DELTA, "attention": L.MIX_ATTENTION, "retention": L.MIX_RETENTION}
 # which mixers and feed-forwards a design may list, and how its blocks join the residual stream
 DESIGNS = {
     "Pikavik": {"mixers": ("wkv", "mlstm", "latent_attention"), "mlp": ("moe",), "block": L.BLOCK_PARALLEL_PRENORM,
@@ -70,6 +77,9 @@ DESIGNS = {
     "Vatolorn": {"mixers": ("parallel",), "mlp": ("dense",), "block": L.BLOCK_SERIAL_PRENORM, "norm_offset": 0.0,
                  "pair": {"qk_norm": 2, "pair_norm": 1, "d_gate_act": 1, "left_scale": 0.5, "right_scale": 0.5},
                  "pair_low_rank": True, "ffn": {"ff_act": L.ACT_SILU}},
+    "Vegilix": {"mixers": ("attention", "retention"), "mlp": ("moe",), "block": L.BLOCK_SERIAL_SANDWICH, "norm_offset": 1.0,
+                "attention": {"rot_half": 1, "learned_sink": 0, "maps": 2, "qk_norm": 3},
+                "moe": {"route_top_softmax": 1, "group_best": 1, "expert_act": L.ACT_SILU, "expert_glu": 1, "shared_gate": 0}},
 }
 RGLRU_DECAY_MULT = 8.0  # log a = -8 r softplus(lam)
 
@@ -158,6 +168,17 @@ class LayerSpec:
     d_decay_rank: int = 0
     d_gate_rank: int = 0
     d_gate_act: int = 0
+    # attention without a convolution: maps per head (2: differential attention, `diff` its constant), first keys that stay visible
+    # beside the window, rotation frequencies scaled by wavelength
+    maps: int = 1
+    diff: float = 0.0
+    keep_first: int = 0
+    wave_factor: float = 0.0
+    wave_low: float = 0.0
+    wave_high: float = 0.0
+    wave_original: float = 0.0
+    # retention: decay per head
+    decay: tuple = ()
 
     def cfg(self) -> L.HybLayerCfg:
         mlp = {"moe": L.MLP_MOE, "dense": L.MLP_GLU, "ffn": L.MLP_FFN, None: L.MLP_NONE}[self.mlp]
@@ -172,7 +193,8 @@ class LayerSpec:
                              self.route_softmax, self.route_bias, self.group_best, self.route_renorm, self.expert_act,
                              self.shared_gate, self.ff_act, self.window, self.rot_half, self.expert_glu,
                              self.route_top_softmax, self.chunk, self.pair_gate, self.pair_conv, self.pair_norm,
-                             whole8(self.d_decay_rank), whole8(self.d_gate_rank), self.d_gate_act)
+                             whole8(self.d_decay_rank), whole8(self.d_gate_rank), self.d_gate_act,
+                             self.maps, self.diff, self.keep_first, self.wave_factor, self.wave_low, self.wave_high, self.wave_original)
 
 
 @dataclass
@@ -187,6 +209,16 @@ class HybridSpec:
     canon_taps: int = 0       # one-norm blocks: taps of the sublayers' input convolutions (0: none)
     streams: int = 0          # serial pre-norm blocks: residual streams (0: one plain residual)
     logit_scale: float = 1.0
+    loop: tuple | None = None  # (start, stop, times): layers start .. stop - 1 run `times` times in a row
+
+    @property
+    def runs(self) -> list[int]:
+        """The layers in the order they run; a looped layer appears once per pass (same weights, its own cache or state)."""
+        n = len(self.layers)
+        if not self.loop:
+            return list(range(n))
+        start, stop, times = self.loop
+        return list(range(start)) + list(range(start, stop)) * times + list(range(stop, n))
 
     @property
     def gated_residual(self) -> bool:
@@ -261,8 +293,22 @@ class HybridSpec:
                                vdim=int(m.get("vdim", m["dim"])), attn_scale=float(m["scale"]), conv=int(m.get("conv") or 1),
                                rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)),
                                window=int((m.get("mask") or {}).get("size", 0)))
+                ls.keep_first = int((m.get("mask") or {}).get("keep_first", 0))
+                sc = rot.get("scaling")
+                if sc:
+                    ls.wave_factor, ls.wave_original = float(sc["factor"]), float(sc["original"])
+                    ls.wave_low, ls.wave_high = float(sc["low"]), float(sc["high"])
                 for key, val in (design.get("attention") or {}).items():
                     setattr(ls, key, val)
+                if ls.maps == 2:
+                    ls.diff = float(m["diff"])
+            elif kind == "retention":
+                rot = m.get("rot") or {}
+                ls = LayerSpec(mixer=kind, heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim", m["dim"])),
+                               rot_dims=int(rot.get("dims", 0)), rot_base=float(rot.get("base", 10000.0)),
+                               decay=tuple(float(d) for d in m["decay"]))
+                if len(ls.decay) != ls.heads:
+                    raise ValueError(f"layer {i}: {len(ls.decay)} decays for {ls.heads} heads")
             else:
                 ls = LayerSpec(mixer=kind, heads=int(m["heads"]), dim=int(m["dim"]))
             if kind == "wkv":
@@ -306,12 +352,19 @@ class HybridSpec:
                     for key, val in (design.get("moe") or {}).items():
                         setattr(ls, key, val)
             layers.append(ls)
+        loop = cfg.get("loop")
+        if loop:
+            loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+            if not (0 <= loop[0] < loop[1] <= len(layers) and loop[2] >= 1):
+                raise ValueError(f"loop {loop} does not fit {len(layers)} layers")
+            if any(l.kv_from >= 0 for l in layers):
+                raise ValueError("a loop beside layers that read another layer's cache is not built")
         return cls(width=int(cfg["width"]), vocab=int(cfg["vocab"]), eps=float(cfg["norm"]["eps"]), layers=layers,
                    architecture=arch, embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
                    residual_mult=float(cfg.get("residual_mult", 1.0)),
                    canon_taps=int((cfg.get("canon") or {}).get("taps", 0)) if design["block"] == L.BLOCK_PARALLEL_ONE_NORM else 0,
                    streams=int(cfg.get("streams") or 0) if design["block"] == L.BLOCK_SERIAL_PRENORM else 0,
-                   logit_scale=float(cfg.get("logit_scale", 1.0)))
+                   logit_scale=float(cfg.get("logit_scale", 1.0)), loop=loop or None)
 
     @classmethod
     def from_dir(cls, path: str) -> "HybridSpec":
@@ -363,7 +416,8 @@ def pack_hybrid_weights(spec: HybridSpec, raw: dict[str, torch.Tensor], dtype: t
     two_norms = spec.block == L.BLOCK_PARALLEL_TWO_NORMS
     one_norm = spec.block == L.BLOCK_PARALLEL_ONE_NORM
     serial_pre = spec.block == L.BLOCK_SERIAL_PRENORM
-    scales = not two_norms and not one_norm and not serial_pre
+    sandwich = spec.block == L.BLOCK_SERIAL_SANDWICH
+    scales = not two_norms and not one_norm and not serial_pre and not sandwich
     for i, ls in enumerate(spec.layers):
         p, mx = f"l{i}.", f"l{i}.mix."
         lw = {"NORM": dev(t(p + "norm1"))}
@@ -382,7 +436,11 @@ def pack_hybrid_weights(spec: HybridSpec, raw: dict[str, torch.Tensor], dtype: t
             lw["MIX_OUT"] = dev(t(mx + "o"))
             if scales:
                 lw["LS_MIX"] = dev(t(p + "ls1"))
-        if two_norms and ls.mlp:
+        if sandwich:   # norms on the sublayers' results
+            lw["NORM_POST"] = dev(t(p + "norm1b"))
+            if ls.mlp:
+                lw["NORM2_POST"] = dev(t(p + "norm2b"))
+        if (two_norms or sandwich) and ls.mlp:
             lw["NORM2"] = dev(t(p + "norm2"))
         if ls.mixer == "rglru":
             lw["RGLRU_IN"] = dev(torch.cat([t(mx + "y"), t(mx + "x")]))
@@ -425,13 +483,21 @@ def pack_hybrid_weights(spec: HybridSpec, raw: dict[str, torch.Tensor], dtype: t
             lw["ATTN_IN"] = dev(torch.cat([t(mx + "q"), t(mx + "k"), t(mx + "v")]))
             if mx + "q.b" in raw:
                 lw["ATTN_IN_B"] = dev(torch.cat([t(mx + "q.b"), t(mx + "k.b"), t(mx + "v.b")]))
-            if mx + "q.conv" in raw:
+            if ls.qk_norm == 3:   # one weight per query, one per key entry, the same for every head and map
+                lw["ATTN_QK_NORM"] = dev(torch.stack([t(mx + "q.norm"), t(mx + "k.norm")]))
+            if ls.maps == 2:
+                lw["ATTN_DIFF"] = dev(torch.stack([t(mx + s) for s in ("lq1", "lk1", "lq2", "lk2")]))
+            if ls.qk_norm == 3 or ls.maps == 2:
+                pass   # straight from the projection
+            elif mx + "q.conv" in raw:
                 lw["CONV_W"] = dev(torch.cat([t(mx + "q.conv"), t(mx + "k.conv"), t(mx + "v.conv")]))
             else:   # no convolution: one tap of weight 1
                 lw["CONV_W"] = dev(torch.ones(lw["ATTN_IN"].shape[0], 1))
             if ls.learned_sink:
                 lw["ATTN_SINK"] = dev(t(mx + "sink"))
             lw["MIX_OUT"] = dev(t(mx + "o"))
+        elif ls.mixer == "retention":
+            lw["RET_IN"], lw["MIX_OUT"] = dev(torch.cat([t(mx + s) for s in "qkvg"])), dev(t(mx + "o"))
         elif ls.mixer == "wkv":
             lw["WKV_MU"] = dev(torch.stack([t(mx + "mu." + s) for s in "rkvgw"]))
             for s in "rkvg":
@@ -517,6 +583,24 @@ def random_hybrid_weights(spec: HybridSpec, dtype: torch.dtype, device, seed: in
             w["HEAD"] = w["EMBED"]
     for ls in spec.layers:
         H, D, V = ls.heads, ls.dim, ls.vdim
+        if spec.block == L.BLOCK_SERIAL_SANDWICH:
+            lw = {"NORM": vec(W), "NORM_POST": vec(W), "MIX_OUT": lin(W, H * V)}
+            if ls.mixer == "retention":
+                lw["RET_IN"] = lin(2 * H * (D + V), W)
+            elif ls.mixer == "attention" and ls.qk_norm == 3:
+                lw["ATTN_IN"], lw["ATTN_QK_NORM"] = lin(ls.maps * (H + ls.kv_heads) * D + ls.kv_heads * V, W), vec(2 * D, 1.0).view(2, D)
+                if ls.maps == 2:
+                    lw["ATTN_DIFF"] = vec(4 * D).view(4, D)
+            else:
+                raise ValueError("random weights of blocks with norms on both sides are made for retention and attention with norms per head")
+            if ls.mlp == "moe":
+                lw["NORM2"], lw["NORM2_POST"], lw["ROUTER"] = vec(W), vec(W), lin(ls.experts, W)
+                mats = 2 if ls.expert_glu else 1
+                lw["EXPERT_IN"], lw["EXPERT_OUT"] = lin(ls.experts, mats * ls.ff, W), lin(ls.experts, W, ls.ff)
+                if ls.shared_ff:
+                    lw["SHARED_IN"], lw["SHARED_OUT"] = lin(mats * ls.shared_ff + (1 if ls.shared_gate else 0), W), lin(W, ls.shared_ff)
+            w["layers"].append(lw)
+            continue
         if spec.block == L.BLOCK_PARALLEL_ONE_NORM:
             subs = 2 if ls.mlp else 1
             lw = {"NORM": vec(W, 1.0), "MIX_OUT": lin(W, H * V)}
@@ -668,10 +752,11 @@ class HybridRunner:
         self.dtype = {"bfloat16": torch.bfloat16, "float32": torch.float32}[dtype]
         # logits of one call live on the device as fp32 + bf16: all rows of a call unless that exceeds ~6 GB
         self.max_logit_rows = max_logit_rows or max(1, min(max_tokens, (1 << 30) // spec.vocab))
-        cfg = L.HybCfg(spec.width, spec.vocab, len(spec.layers), L.DT_BF16 if self.dtype == torch.bfloat16 else L.DT_F32,
+        self.runs = spec.runs   # the engine's layers: one per run
+        cfg = L.HybCfg(spec.width, spec.vocab, len(self.runs), L.DT_BF16 if self.dtype == torch.bfloat16 else L.DT_F32,
                        spec.eps, max_tokens, max_seqs, self.max_logit_rows, block_size, self.max_blocks, spec.block, spec.norm_offset,
                        spec.embed_scale, spec.residual_mult, spec.canon_taps, int(spec.gated_residual), spec.streams, spec.logit_scale)
-        layer_cfgs = (L.HybLayerCfg * len(spec.layers))(*[l.cfg() for l in spec.layers])
+        layer_cfgs = (L.HybLayerCfg * len(self.runs))(*[spec.layers[i].cfg() for i in self.runs])
         h = C.c_void_p()
         L.check(self.lib.ssdk_hyb_create(C.byref(cfg), layer_cfgs, C.byref(h)), "ssdk_hyb_create")
         self.h = h
@@ -697,16 +782,19 @@ class HybridRunner:
 
         for name in ("EMBED", "HEAD", "FINAL_NORM"):
             bind(-1, name, w[name])
-        for i, lw in enumerate(w["layers"]):
-            for name, t in lw.items():
-                bind(i, name, t)
+        for r, i in enumerate(self.runs):
+            for name, t in w["layers"][i].items():
+                bind(r, name, t)
+            if self.spec.layers[i].decay:
+                d = self.spec.layers[i].decay
+                L.check(self.lib.ssdk_hyb_retention_decay(self.h, r, (C.c_double * len(d))(*d), len(d)), f"decays of layer {i}")
 
     # ------------------------------------------------------------------ the step function
     def forward(self, entries, *, want_logits: bool = True, temps=None, seed: int = 0, residual: bool = False):
         """entries: list of (tokens, pos0, slot, block_table, want) — `tokens` continue a sequence at position pos0 whose
         state lives in `slot` and whose latent rows live in the pages `block_table`; `want` lists the places among
         `tokens` whose logits (and, with `temps`, sampled tokens) are asked for.  Returns (logits [n_want, vocab] float32
-        or None, tokens list or None[, residual [layers, rows, width]]), rows in the order of the entries."""
+        or None, tokens list or None[, residual [layer runs, rows, width]]), rows in the order of the entries."""
         total = sum(len(e[0]) for e in entries)
         if total > self.max_tokens or len(entries) > self.max_seqs or sum(len(e[4]) for e in entries) > self.max_logit_rows:
             return self._forward_split(entries, want_logits, temps, seed, residual)
@@ -727,7 +815,7 @@ class HybridRunner:
         temps_a = np.ascontiguousarray(temps, dtype=np.float32) if temps is not None else None
         if temps_a is not None and len(temps_a) != n_want:
             raise ValueError("one temperature per wanted row")
-        res = np.empty((len(self.spec.layers), total, self.spec.width), dtype=np.float32) if residual else None
+        res = np.empty((len(self.runs), total, self.spec.width), dtype=np.float32) if residual else None
         ids_a, cu_a, pos_a, slot_a, want_a = _i32(ids), _i32(cu), _i32(pos0), _i32(slots), _i32(want_rows or [0])
         L.check(self.lib.ssdk_hyb_forward(
             self.h, len(entries), total, ids_a.ctypes.data_as(L.c_i32p), cu_a.ctypes.data_as(L.c_i32p),

@@ -60,6 +60,8 @@ class HybLayerCfg(C.Structure):
         ("window", C.c_int32), ("rot_half", C.c_int32), ("expert_glu", C.c_int32), ("route_top_softmax", C.c_int32),
         ("chunk", C.c_int32), ("pair_gate", C.c_int32), ("pair_conv", C.c_int32), ("pair_norm", C.c_int32),
         ("d_decay_rank", C.c_int32), ("d_gate_rank", C.c_int32), ("d_gate_act", C.c_int32),
+        ("maps", C.c_int32), ("diff", C.c_float), ("keep_first", C.c_int32), ("wave_factor", C.c_float), ("wave_low", C.c_float),
+        ("wave_high", C.c_float), ("wave_original", C.c_float),
     ]
 
 
@@ -77,16 +79,18 @@ class HybCfg(C.Structure):
 
 # hybrid-model enums (include/ssdk.h)
 DT_F32, DT_BF16 = 0, 1
-MIX_WKV, MIX_MLSTM, MIX_LATENT_ATTN, MIX_RGLRU, MIX_SELECTIVE, MIX_ATTN_DELTA, MIX_ATTENTION = 0, 1, 2, 3, 4, 5, 6
+MIX_WKV, MIX_MLSTM, MIX_LATENT_ATTN, MIX_RGLRU, MIX_SELECTIVE, MIX_ATTN_DELTA, MIX_ATTENTION, MIX_RETENTION = 0, 1, 2, 3, 4, 5, 6, 7
 MLP_NONE, MLP_MOE, MLP_GLU, MLP_FFN = 0, 1, 2, 3
 ACT_CLAMPED, ACT_SILU, ACT_GELU_TANH, ACT_RELU2, ACT_POLYNORM = 0, 1, 2, 3, 4
 BLOCK_PARALLEL_PRENORM, BLOCK_SERIAL_POSTNORM, BLOCK_PARALLEL_TWO_NORMS, BLOCK_PARALLEL_ONE_NORM, BLOCK_SERIAL_PRENORM = 0, 1, 2, 3, 4
+BLOCK_SERIAL_SANDWICH = 5
 HT_NAMES = ("EMBED HEAD FINAL_NORM NORM LS_MIX LS_MLP WKV_MU WKV_R WKV_K WKV_V WKV_G WKV_W1 WKV_W2 WKV_W0 WKV_U MLSTM_IN "
             "MLSTM_IB MLSTM_FB LAT_DOWN LAT_QNORM LAT_KVNORM LAT_UQ LAT_UKT LAT_UV LAT_SINK MIX_NORM MIX_OUT ROUTER "
             "EXPERT_IN EXPERT_OUT SHARED_IN SHARED_OUT NORM2 GLU_IN GLU_OUT CONV_W CONV_B RGLRU_IN RGLRU_IN_B RGLRU_GATE "
             "RGLRU_GATE_B RGLRU_LAM SEL_IN SEL_X SEL_DT SEL_DT_B SEL_ALOG SEL_D PAIR_IN ATTN_OUT DELTA_ALOG DELTA_DT_B "
             "LAT_IN FFN_IN FFN_IN_B FFN_OUT FFN_OUT_B ROUTER_BIAS ATTN_IN ATTN_IN_B ATTN_SINK FFN_ACT CANON_W RES_GATE "
-            "RES_GATE_B ATTN_CONV_W ATTN_QK_NORM DELTA_A2 DELTA_G2 PAIR_NORM HC_IN HC_OUT HC_MIX").split()
+            "RES_GATE_B ATTN_CONV_W ATTN_QK_NORM DELTA_A2 DELTA_G2 PAIR_NORM HC_IN HC_OUT HC_MIX "
+            "NORM_POST NORM2_POST ATTN_DIFF RET_IN").split()
 HT = {n: i for i, n in enumerate(HT_NAMES)}
 
 # weight kinds (enum in include/ssdk.h)
@@ -137,6 +141,7 @@ SIGNATURES: dict[str, tuple] = {
     "ssdk_hyb_create": (C.c_int, [C.POINTER(HybCfg), C.POINTER(HybLayerCfg), C.POINTER(VP)]),
     "ssdk_hyb_destroy": (C.c_int, [VP]),
     "ssdk_hyb_bind": (C.c_int, [VP, C.c_int, C.c_int, VP, C.c_int64, C.c_int64]),
+    "ssdk_hyb_retention_decay": (C.c_int, [VP, C.c_int, C.POINTER(C.c_double), C.c_int]),
     "ssdk_hyb_cache_bytes": (C.c_int64, [VP, C.c_int64]),
     "ssdk_hyb_state_bytes": (C.c_int64, [VP, C.c_int64]),
     "ssdk_hyb_workspace_bytes": (C.c_int64, [VP]),
