@@ -1,4 +1,4 @@
-"""Throughput of the hybrid families (bench.py --arch pikavik | kefurax | lisenex | kokatar | vatolorn).
+"""Throughput of the hybrid families (bench.py --arch pikavik | kefurax | lisenex | kokatar | vatolorn | vegilix).
 
 --arch pikavik: a Pikavik stack beside the closest dense model of the framework (below).
 --arch kefurax: a Kefurax stack (attention + delta-rule pair with a dense feed-forward, selective scan, rglru, ...) beside
@@ -14,6 +14,10 @@ same width, depth, vocabulary and feed-forward / expert sizes.
 beside a delta rule with a decay per key channel; dense silu-GLU feed-forward) beside the closest existing model of the
 framework, a Kefurax stack whose every layer is the attention + delta-rule pair, of the same width, depth, vocabulary, head
 counts and sizes and feed-forward size.
+--arch vegilix: a Vegilix stack (norms before and after each sublayer; windowed differential attention with kept first keys,
+every fourth layer a retention; silu experts with a shared one) beside the closest existing model of the framework, a Kokatar
+stack whose every layer is grouped-query attention with a mixture of experts, of the same width, depth, vocabulary, window,
+projection sizes of the attention and expert sizes.
 
 For every size: a Pikavik stack (mLSTM, wkv, wkv, latent attention, ... each with a grouped mixture of experts and a
 shared expert) with random weights, and a Llama stack of the same width, depth and ACTIVE feed-forward size
@@ -118,7 +122,34 @@ def lisenex_spec(z):
     return HybridSpec(z["width"], z["vocab"], 1e-6, layers, architecture="Lisenex", embed_scale=float(z["width"]) ** 0.5)
 
 
-def kokatar_spec(z, window=1024):
+def vegilix_spec(z, window=1024):
+    """Layers that resemble a real model's: differential attention with two maps of 64 over values of 128 per head, four heads per
+    key/value head, half of a map rotated with scaled frequencies, a window beside four kept keys; in every fourth layer a retention
+    with 128 x 128 heads, fully rotated, decays 1 - 2^-5 .. 1 - 2^-12; `experts` silu experts with a shared one in every layer."""
+    from .hybrid import DESIGNS, HybridSpec, LayerSpec
+    d = DESIGNS["Vegilix"]
+    W = z["width"]
+    heads = W // 128
+    layers = []
+    for i in range(z["layers"]):
+        if i % 4 == 2:
+            ls = LayerSpec("retention", heads, 128, 128, rot_dims=128, rot_base=10000.0, decay=tuple(1.0 - 2.0 ** -(5 + 7 * h / max(1, heads - 1)) for h in range(heads)))
+        else:
+            ls = LayerSpec("attention", heads, 64, 128, rot_dims=32, rot_base=10000.0, attn_scale=64 ** -0.5, kv_heads=max(1, heads // 4), window=window,
+                           keep_first=4, conv=1, diff=0.5, wave_factor=4.0, wave_low=1.0, wave_high=4.0, wave_original=4096.0, **d["attention"])
+        ls.mlp, ls.experts, ls.top, ls.ff, ls.shared_ff = "moe", z["experts"], z["top"], z["ff"], z["sff"]
+        for k, v in d["moe"].items():
+            setattr(ls, k, v)
+        layers.append(ls)
+    return HybridSpec(W, z["vocab"], 1e-6, layers, architecture="Vegilix", residual_mult=0.5)
+
+
+def kokatar_attention_spec(z, window=1024):
+    """A Kokatar stack of grouped-query attention with a mixture of experts only."""
+    return kokatar_spec(z, window, attention_only=True)
+
+
+def kokatar_spec(z, window=1024, attention_only=False):
     """Layers that resemble a real model's: attention with 128-wide heads, four query heads per key/value head, half of a
     head rotated, 4 taps on q | k | v; latent attention with 16 heads of 64 / 128 over a latent of 256 / 512; every layer
     looks back `window` tokens; 4 taps on the sublayers' inputs; feed-forwards alternate between a dense one as wide as a
@@ -129,13 +160,13 @@ def kokatar_spec(z, window=1024):
     heads = W // 128
     layers = []
     for i in range(z["layers"]):
-        if i % 3 == 0:
+        if attention_only or i % 3 == 0:
             ls = LayerSpec("attention", heads, 128, 128, rot_dims=64, rot_base=10000.0, attn_scale=128 ** -0.5,
                            kv_heads=max(1, heads // 4), conv=4, window=window, **d["attention"])
         else:
             ls = LayerSpec("latent_attention", z["lh"], z["ld"], z["ld"], kv_rank=z["kvr"], attn_scale=z["ld"] ** -0.5, window=window,
                            **d["latent"])
-        if i % 2 == 0:
+        if not attention_only and i % 2 == 0:
             ls.mlp, ls.ff, ls.ff_act = "ffn", z["top"] * z["ff"] + z["sff"], d["ffn"]["ff_act"]
         else:
             ls.mlp, ls.experts, ls.top, ls.ff, ls.shared_ff = "moe", z["experts"], z["top"], z["ff"], z["sff"]
@@ -309,7 +340,28 @@ def run_vatolorn(args):
     return out
 
 
+def run_vegilix(args):
+    out = {"metric": "prefill and decode tokens/s, Vegilix beside Kokatar attention at equal width / depth / attention projections / experts",
+           "dtype": "bf16", "data": "synthetic (random weights, random token ids)", "n_gpus": 1, "steps": args.steps,
+           "warmup": args.warmup, "timing": "CUDA events around the public forward call, median; every pass streams the stack's "
+           "weights (> 126 MB L2 for size m; size s partly L2-resident, stated here)", "sizes": {}}
+    names = [args.hybrid_size] if args.hybrid_size != "all" else list(SIZES)
+    for name in names:
+        z = SIZES[name]
+        row = {"config": {k: z[k] for k in ("width", "layers", "experts", "top", "ff", "sff", "vocab")}, "prompt": args.prompt_len_hybrid,
+               "decode_batch": args.hybrid_batch, "window": 1024}
+        row["vegilix"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, spec_fn=vegilix_spec)
+        if not args.no_dense_arm:
+            row["kokatar_attention"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, spec_fn=kokatar_attention_spec)
+        if args.hybrid_fp32:
+            row["vegilix_fp32"] = run_pikavik(z, args.prompt_len_hybrid, args.hybrid_batch, args.warmup, args.steps, "float32", vegilix_spec)
+        out["sizes"][name] = row
+    return out
+
+
 def run(args):
+    if getattr(args, "arch", "pikavik") == "vegilix":
+        return run_vegilix(args)
     if getattr(args, "arch", "pikavik") == "vatolorn":
         return run_vatolorn(args)
     if getattr(args, "arch", "pikavik") == "kokatar":
