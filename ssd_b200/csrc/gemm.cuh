@@ -20,7 +20,7 @@
 //     in a fixed order, so results are deterministic.
 //   * epilogues: bf16 store, fp32 split-K partial, or fused SiLU(gate)*up where a tile is
 //     64 gate rows + 64 up rows of the packed gate|up matrix (layers/activation.py:11-14); EPI_GLU is its form for the layered
-//     models: any number of row chunks, silu or gelu_tanh, gate and up kept in fp32 up to the product.
+//     models: any number of row chunks (or a routed batch's tiles), silu or gelu_tanh, gate and up kept in fp32 up to the product.
 //   * PDL: weight tiles of the first kStages are requested BEFORE griddepcontrol.wait, so
 //     the HBM stream of this GEMM starts under the tail of the previous kernel.
 #pragma once
@@ -66,7 +66,7 @@ struct GemmParams {
   unsigned* sk_counters;  // [tiles] arrival tickets, zero on entry and on exit
   int sk_width;           // row width of the partial buffer (N, or 2 * ffn for gate|up)
   PublishParams pub;      // EPI_PUBLISH only
-  // grouped mode (EPI_PARTIAL, g_tile_expert != nullptr): blockIdx.z indexes a device-side list of row tiles, each of one
+  // grouped mode (EPI_PARTIAL and EPI_GLU, g_tile_expert != nullptr): blockIdx.z indexes a device-side list of row tiles, each of one
   // expert: tile t multiplies the rows g_tile_row0[t] .. + g_tile_rows[t] (<= UMMA_N) of the X map, whose rows are sorted by
   // expert, with the weight rows of expert g_tile_expert[t] (g_expert_rows rows of the stacked W map per expert).  CTAs
   // beyond *g_n_tiles leave at once.  Rows of the X box that belong to the next expert are multiplied and dropped.
@@ -158,7 +158,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
   int m_base = (int)blockIdx.z * UMMA_N;
   int m_valid = min(UMMA_N, p.M - m_base);
   int w_row0 = 0;   // first weight row of this CTA's expert in the stacked W map (grouped mode)
-  if (EPI == EPI_PARTIAL && p.g_tile_expert != nullptr) {
+  if ((EPI == EPI_PARTIAL || EPI == EPI_GLU) && p.g_tile_expert != nullptr) {
     if ((int)blockIdx.z >= *p.g_n_tiles) return;   // the whole CTA, before any barrier or TMEM allocation
     m_base = p.g_tile_row0[blockIdx.z];
     m_valid = min(UMMA_N, p.g_tile_rows[blockIdx.z]);

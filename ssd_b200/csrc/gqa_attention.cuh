@@ -208,11 +208,11 @@ __global__ void gqa_conv_prep_kernel(const GqaConvPrepArgs p, const Ragged rg) {
   }
 }
 
-// Rows of heads through a warp: dst[d] = (rotated) value of src[d] * inv * w[d] * mult, entries d and d + half of the first 2 half
+// Rows of heads through LANES neighbouring lanes: dst[d] = (rotated) value of src[d] * inv * w[d] * mult, entries d and d + half of the first 2 half
 // ones turned by the row's angles (cs: half cosines, then half sines).  VEC = 4: D, half and both pointers are whole groups of four.
-template <typename OutT, typename T, int VEC>
+template <typename OutT, typename T, int VEC, int LANES = 32>
 SSDK_DEVINL void head_row(const float* src, OutT* dst, int D, int half, const float* cs, const T* w, float inv, float mult, int lane) {
-  for (int d = lane * VEC; d < D; d += 32 * VEC) {
+  for (int d = lane * VEC; d < D; d += LANES * VEC) {
     float v[VEC];
     ld_vec<VEC>(src + d, v);
     if (w) {
@@ -251,36 +251,41 @@ struct GqaHeadPrepArgs {
   int maps;
 };
 
-// grid (M, y): the warps of a row's CTAs take its H queries, G keys and G / maps values in turn.  dynamic shared memory: rot_dims floats
-template <typename T, int VEC>
+// grid (M, y): groups of LANES lanes of a row's CTAs take its H queries, G keys and G / maps values in turn.  dynamic shared memory:
+// rot_dims floats
+template <typename T, int VEC, int LANES>
 __global__ void gqa_head_prep_kernel(const GqaHeadPrepArgs p, const Ragged rg) {
   SSDK_DYN_SMEM(float, hp_cs);
-  const int m = blockIdx.x, s = rg.tok_seq[m], pos = rg.pos0[s] + (m - rg.cu[s]), lane = threadIdx.x & 31;
+  const int m = blockIdx.x, s = rg.tok_seq[m], pos = rg.pos0[s] + (m - rg.cu[s]), lane = threadIdx.x & (LANES - 1);
   const int H = p.g.H, G = p.g.G, Gv = G / p.maps, D = p.g.D, V = p.g.V, hpg = H / G, half = (p.g.inv_freq ? p.g.rot_dims : 0) >> 1;
   row_angles(hp_cs, half, pos, p.g.inv_freq, p.g.rot_mult);
   __syncthreads();
-  const int nw = blockDim.x >> 5;
+  const int nw = blockDim.x / LANES;
   const float* z = p.g.z + (size_t)m * p.g.ldz;
   T* row = (T*)p.g.cache + page_row(rg, s, pos) * ((size_t)G * D + (size_t)Gv * V);
-  for (int u = blockIdx.y * nw + (threadIdx.x >> 5); u < H + G + Gv; u += gridDim.y * nw) {
+  // (every lane of a warp makes the same number of rounds: the sums below are exchanged by all of them)
+  for (int u0 = blockIdx.y * nw; u0 < H + G + Gv; u0 += gridDim.y * nw) {
+    const int u = u0 + threadIdx.x / LANES;
+    float ss = 0.f;
+    if (p.norm_w && u < H + G) {
+      for (int d = lane * VEC; d < D; d += LANES * VEC) {
+        float v[VEC];
+        ld_vec<VEC>(z + (size_t)u * D + d, v);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ss = fmaf(v[e], v[e], ss);
+      }
+    }
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (u >= H + G + Gv) continue;
     if (u >= H + G) {
       const int g = u - H - G;
-      head_row<T, T, VEC>(z + (size_t)(H + G) * D + (size_t)g * V, row + (size_t)G * D + (size_t)g * V, V, 0, hp_cs, (const T*)nullptr, 1.f, 1.f, lane);
+      head_row<T, T, VEC, LANES>(z + (size_t)(H + G) * D + (size_t)g * V, row + (size_t)G * D + (size_t)g * V, V, 0, hp_cs, (const T*)nullptr, 1.f, 1.f, lane);
       continue;
     }
     const float* src = z + (size_t)u * D;
     const T* w = p.norm_w ? (const T*)p.norm_w + (u < H ? 0 : D) : nullptr;
-    float inv = 1.f;
-    if (w) {
-      float ss = 0.f;
-      for (int d = lane * VEC; d < D; d += 32 * VEC) {
-        float v[VEC];
-        ld_vec<VEC>(src + d, v);
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) ss = fmaf(v[e], v[e], ss);
-      }
-      inv = 1.0f / sqrtf(warp_sum(ss) / (float)D + p.g.eps);
-    }
+    const float inv = w ? 1.0f / sqrtf(ss / (float)D + p.g.eps) : 1.f;
     T* dst;
     if (u < H) {
       const int hd = u / p.maps, g = hd / hpg * p.maps + u % p.maps;
@@ -288,7 +293,7 @@ __global__ void gqa_head_prep_kernel(const GqaHeadPrepArgs p, const Ragged rg) {
     } else {
       dst = row + (size_t)(u - H) * D;
     }
-    head_row<T, T, VEC>(src, dst, D, half, hp_cs, w, inv, 1.f, lane);
+    head_row<T, T, VEC, LANES>(src, dst, D, half, hp_cs, w, inv, 1.f, lane);
   }
 }
 

@@ -394,6 +394,10 @@ struct HybRun {
     }
     return 0;
   }
+  // bf16 with whole k-blocks and enough 64-column tiles to stream the weights
+  bool tc_glu_ok(const void* A, const void* W, int ff, int K) const {
+    return e->use_tc_glu && (ff + 63) / 64 * ((M + kMaxTokens - 1) / kMaxTokens) >= 24 && tc_ok(A, K, W, K, 2 * ff, 2 * ff, K);
+  }
   // y [m, ff] (bf16) = act(x Wg^T) * (x Wu^T) in the GEMM's epilogue; W holds the gate rows, then the up rows
   int lin_tc_glu(const void* A, const void* W, void* y, int m_total, int ff, int K, bool gelu) {
     const CUtensorMap* tm;
@@ -408,8 +412,9 @@ struct HybRun {
     return launch_gemm(L, un, EPI_GLU, tmW, tmX, p, (ff + 63) / 64, 1, chunks);
   }
   // grouped form: rows of X sorted by expert, tile list on the device (expert_plan_kernel with tiles of `un` rows);
-  // C[r, :] = X[r, :] Wm[expert(r)]^T with Wm the experts' [N, K] matrices stacked by rows
-  int lin_tc_grouped(const void* X, const void* Wm, float* C, int rows, int N, int K, int n_experts, int un, int max_tiles) {
+  // C[r, :] = X[r, :] Wm[expert(r)]^T with Wm the experts' [N, K] matrices stacked by rows; glu: N holds gate rows, then as many up rows,
+  // and C [rows, N / 2] (bf16) is silu(gate) * up
+  int lin_tc_grouped(const void* X, const void* Wm, void* C, int rows, int N, int K, int n_experts, int un, int max_tiles, bool glu = false) {
     const CUtensorMap* tm;
     CKI(e->tmap(Wm, (int64_t)n_experts * N, K, 64, &tm));
     const CUtensorMap tmW = *tm;
@@ -420,6 +425,10 @@ struct HybRun {
     p.sk_partials = nullptr; p.sk_counters = nullptr; p.sk_width = 0; p.out = C;
     p.g_tile_expert = e->tile_expert; p.g_tile_row0 = e->tile_row0; p.g_tile_rows = e->tile_rows; p.g_n_tiles = e->n_tiles;
     p.g_expert_rows = N;
+    if (glu) {
+      p.N = p.ldo = p.hi_row_offset = N / 2; p.tile_rows = 64;
+      return launch_gemm(L, un, EPI_GLU, tmW, tmX, p, (N / 2 + 63) / 64, 1, max_tiles);
+    }
     return launch_gemm(L, un, EPI_PARTIAL, tmW, tmX, p, (N + kTileRows - 1) / kTileRows, 1, max_tiles);
   }
   // C[M, N] (fp32 unless out_t) = A[M, K] W[N, K]^T
@@ -697,11 +706,18 @@ struct HybRun {
 
   const void* fin = nullptr;   // the feed-forward's input in the storage type (the mixer's input, or the second norm's rows)
 
+  // y [rows, ff] = act(gate columns) * up columns of z, few rows spread over the machine
+  template <int ACT>
+  int glu_act(const float* z, int ldz, T* y, int ff, int rows, const int* n_rows) {
+    if (ff % 4 == 0 && ldz % 4 == 0 && (((uintptr_t)z | (uintptr_t)y) & 15) == 0) return L.go(ssdk::glu_act_kernel<T, ACT, 4>, act_grid(rows, ff / 4), dim3(256), 0, z, ldz, y, ff, n_rows);
+    return L.go(ssdk::glu_act_kernel<T, ACT, 1>, act_grid(rows, ff), dim3(256), 0, z, ldz, y, ff, n_rows);
+  }
+
   // an expert's activation over `rows` rows of z [rows, ldz] -> y [rows, ff]: gated (z = gate | up columns) or not (z = up columns)
   int expert_act(const ssdk_hyb_layer_cfg& c, const float* z, int ldz, T* y, int ff, float limit, int rows, const int* n_rows) {
     const dim3 grid(rows), block(128);
     if (c.expert_glu) {
-      if (c.expert_act == SSDK_ACT_SILU) return L.go(ssdk::glu_act_kernel<T, SSDK_ACT_SILU>, grid, block, 0, z, ldz, y, ff, n_rows);
+      if (c.expert_act == SSDK_ACT_SILU) return glu_act<SSDK_ACT_SILU>(z, ldz, y, ff, rows, n_rows);
       return L.go(ssdk::clamped_glu_kernel<T>, grid, block, 0, z, ldz, y, ff, limit, n_rows);
     }
     if (c.expert_act == SSDK_ACT_SILU) return L.go(ssdk::act_cols_kernel<T, SSDK_ACT_SILU>, grid, block, 0, z, ldz, y, ff, n_rows);
@@ -726,6 +742,7 @@ struct HybRun {
     // else the mma.sync / FMA tile, which gathers by index itself (tiles of kLinBM rows)
     const bool tc_moe = !kF32 && e->use_tc && e->use_tc_experts && A >= 256 && W % kBlockK == 0 && ff % kBlockK == 0 &&
                         (((uintptr_t)Lr.t[SSDK_HT_EXPERT_IN].p | (uintptr_t)Lr.t[SSDK_HT_EXPERT_OUT].p) & 15) == 0;
+    const bool silu_glu = c.expert_glu && c.expert_act == SSDK_ACT_SILU, glu = tc_moe && silu_glu && e->use_tc_glu;   // activation in the GEMM's epilogue
     const int tile = tc_moe ? 128 : ssdk::kLinBM;
     ssdk::PlanArgs pa;
     pa.sel = e->sel; pa.apos = e->apos; pa.arow = e->arow; pa.tile_expert = e->tile_expert; pa.tile_row0 = e->tile_row0;
@@ -736,14 +753,14 @@ struct HybRun {
     ssdk::LinearArgs a = {};
     if (tc_moe) {
       CKI(L.go(ssdk::gather_rows_kernel<T>, dim3(A), dim3(128), 0, (const T*)fin, (const int*)e->arow, (const int*)e->n_rows, (T*)e->xs, W));
-      CKI(lin_tc_grouped(e->xs, Lr.t[SSDK_HT_EXPERT_IN].p, e->eg, A, Nin, W, E, tile, A / tile + E + 1));
+      CKI(lin_tc_grouped(e->xs, Lr.t[SSDK_HT_EXPERT_IN].p, glu ? e->ey : (void*)e->eg, A, Nin, W, E, tile, A / tile + E + 1, glu));
     } else {
       a.A = fin; a.W = Lr.t[SSDK_HT_EXPERT_IN].p; a.C = e->eg; a.M = A; a.N = Nin; a.K = W; a.lda = W; a.ldw = W; a.ldc = Nin;
       a.a_rows = e->arow; a.tile_expert = e->tile_expert; a.tile_row0 = e->tile_row0; a.tile_rows = e->tile_rows; a.n_tiles = e->n_tiles;
       a.sW_expert = (long long)Nin * W;
       CKI(lin_args<float>(a, A, 1));
     }
-    CKI(expert_act(c, (const float*)e->eg, Nin, (T*)e->ey, ff, c.limit, A, n_real_rows));
+    if (!glu) CKI(expert_act(c, (const float*)e->eg, Nin, (T*)e->ey, ff, c.limit, A, n_real_rows));
     if (tc_moe) {
       CKI(lin_tc_grouped(e->ey, Lr.t[SSDK_HT_EXPERT_OUT].p, e->eo, A, W, ff, E, tile, A / tile + E + 1));
     } else {
@@ -755,8 +772,12 @@ struct HybRun {
     if (c.shared_ff > 0) {
       const int sff = c.shared_ff, Ns = (c.expert_glu ? 2 : 1) * sff + (c.shared_gate ? 1 : 0);
       CKI(check_tensor(Lr, SSDK_HT_SHARED_IN, Ns, W, "shared.in")); CKI(check_tensor(Lr, SSDK_HT_SHARED_OUT, W, sff, "shared.out"));
-      CKI(lin(fin, W, Lr.t[SSDK_HT_SHARED_IN].p, W, e->sz, Ns, M, Ns, W));
-      CKI(expert_act(c, (const float*)e->sz, Ns, (T*)e->sy, sff, c.shared_limit, M, (const int*)nullptr));
+      if (silu_glu && !c.shared_gate && tc_glu_ok(fin, Lr.t[SSDK_HT_SHARED_IN].p, sff, W)) {
+        CKI(lin_tc_glu(fin, Lr.t[SSDK_HT_SHARED_IN].p, e->sy, M, sff, W, false));
+      } else {
+        CKI(lin(fin, W, Lr.t[SSDK_HT_SHARED_IN].p, W, e->sz, Ns, M, Ns, W));
+        CKI(expert_act(c, (const float*)e->sz, Ns, (T*)e->sy, sff, c.shared_limit, M, (const int*)nullptr));
+      }
       CKI(lin(e->sy, sff, Lr.t[SSDK_HT_SHARED_OUT].p, sff, e->so, W, M, W, sff));
     }
     return 0;
@@ -792,16 +813,16 @@ struct HybRun {
   int glu(HybLayer& Lr) {
     const int W = e->cfg.width, ff = Lr.c.ff;
     CKI(check_tensor(Lr, SSDK_HT_GLU_IN, 2 * ff, W, "mlp.gate|up")); CKI(check_tensor(Lr, SSDK_HT_GLU_OUT, W, ff, "mlp.down"));
-    // bf16 with whole k-blocks and enough 64-column tiles to stream the weights: activation and product in the GEMM's epilogue
-    if (e->use_tc_glu && (ff + 63) / 64 * ((M + kMaxTokens - 1) / kMaxTokens) >= 24 && tc_ok(hin, W, Lr.t[SSDK_HT_GLU_IN].p, W, 2 * ff, 2 * ff, W)) {
+    // activation and product in the GEMM's epilogue
+    if (tc_glu_ok(hin, Lr.t[SSDK_HT_GLU_IN].p, ff, W)) {
       CKI(lin_tc_glu(hin, Lr.t[SSDK_HT_GLU_IN].p, e->t0, M, ff, W, Lr.c.ff_act == SSDK_ACT_GELU_TANH));
       return lin(e->t0, ff, Lr.t[SSDK_HT_GLU_OUT].p, ff, e->mix_out, W, M, W, ff);
     }
     CKI(lin(hin, W, Lr.t[SSDK_HT_GLU_IN].p, W, e->p0, 2 * ff, M, 2 * ff, W));
     if (Lr.c.ff_act == SSDK_ACT_SILU)
-      CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_SILU>, act_grid(M, ff), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
+      CKI(glu_act<SSDK_ACT_SILU>((const float*)e->p0, 2 * ff, (T*)e->t0, ff, M, nullptr));
     else
-      CKI(L.go(ssdk::glu_act_kernel<T, SSDK_ACT_GELU_TANH>, act_grid(M, ff), dim3(256), 0, (const float*)e->p0, 2 * ff, (T*)e->t0, ff, (const int*)nullptr));
+      CKI(glu_act<SSDK_ACT_GELU_TANH>((const float*)e->p0, 2 * ff, (T*)e->t0, ff, M, nullptr));
     return lin(e->t0, ff, Lr.t[SSDK_HT_GLU_OUT].p, ff, e->mix_out, W, M, W, ff);
   }
 
@@ -917,10 +938,12 @@ struct HybRun {
       ssdk::GqaHeadPrepArgs hp;
       hp.g = pa; hp.norm_w = norm_w; hp.maps = maps;
       const bool vec = D % 4 == 0 && V % 4 == 0 && c.rot_dims % 8 == 0 && ldz % 4 == 0 && (((uintptr_t)z | (uintptr_t)pool | (uintptr_t)e->qcat) & 15) == 0;
-      const int units = H + G + G / maps, ys = std::max(1, std::min((units + 7) / 8, 2 * num_sms() / M));   // few rows: a row's heads over several CTAs
+      const bool pairs = vec && D <= 64;   // half a warp per head
+      const int units = H + G + G / maps, per = pairs ? 16 : 8, ys = std::max(1, std::min((units + per - 1) / per, 2 * num_sms() / M));   // few rows: a row's heads over several CTAs
       const size_t smem = (size_t)c.rot_dims * 4;
-      if (vec) CKI(L.go(ssdk::gqa_head_prep_kernel<T, 4>, dim3(M, ys), dim3(256), smem, hp, rg));
-      else CKI(L.go(ssdk::gqa_head_prep_kernel<T, 1>, dim3(M, ys), dim3(256), smem, hp, rg));
+      if (pairs) CKI(L.go(ssdk::gqa_head_prep_kernel<T, 4, 16>, dim3(M, ys), dim3(256), smem, hp, rg));
+      else if (vec) CKI(L.go(ssdk::gqa_head_prep_kernel<T, 4, 32>, dim3(M, ys), dim3(256), smem, hp, rg));
+      else CKI(L.go(ssdk::gqa_head_prep_kernel<T, 1, 32>, dim3(M, ys), dim3(256), smem, hp, rg));
     } else {
       CKI(L.go(ssdk::gqa_prep_kernel<T>, dim3(M, H + G), dim3(32), 0, pa, rg));
     }
@@ -1064,15 +1087,15 @@ struct HybRun {
     }
     if (n_max > 1) {
       const int ys = std::max(1, std::min((2 * H + 7) / 8, 2 * num_sms() / M)), nc = (n_max + ssdk::kRetChunk - 1) / ssdk::kRetChunk;
-      const size_t rsm = (size_t)c.rot_dims * 4, hdv = (size_t)H * D * V;
+      const size_t rsm = (size_t)c.rot_dims * 4, hdv = (size_t)H * D * V, sb = ssdk::kRetScanThreads;
       if (a.vec) CKI(L.go(ssdk::retention_prep_kernel<4>, dim3(M, ys), dim3(256), rsm, a, rg));
       else CKI(L.go(ssdk::retention_prep_kernel<1>, dim3(M, ys), dim3(256), rsm, a, rg));
       const int ks = D <= 32 ? 2 : (D <= 64 ? 4 : 8), vt = V <= 32 ? 4 : (V <= 64 ? 8 : 16);
       const dim3 cgrid(nc, H, rg.n_seqs), block(256);
       if (mma) CKI(retention_mma(a, ks, vt, cgrid, false));
       else CKI(L.go(ssdk::retention_chunk_state_any_kernel, dim3(nc, H * ((D + 63) / 64) * ((V + 63) / 64), rg.n_seqs), block, 0, a, rg));
-      if (a.vec) CKI(L.go(ssdk::retention_state_scan_kernel<4>, dim3(rg.n_seqs, (unsigned)((hdv / 4 + 255) / 256)), block, 0, a, rg));
-      else CKI(L.go(ssdk::retention_state_scan_kernel<1>, dim3(rg.n_seqs, (unsigned)((hdv + 255) / 256)), block, 0, a, rg));
+      if (a.vec) CKI(L.go(ssdk::retention_state_scan_kernel<4>, dim3(rg.n_seqs, (unsigned)((hdv / 4 + sb - 1) / sb)), dim3(sb), 0, a, rg));
+      else CKI(L.go(ssdk::retention_state_scan_kernel<1>, dim3(rg.n_seqs, (unsigned)((hdv + sb - 1) / sb)), dim3(sb), 0, a, rg));
       if (mma) {
         CKI(retention_mma(a, ks, vt, cgrid, true));
       } else {
@@ -1460,8 +1483,9 @@ static int hyb_smem_attrs(ssdk_hyb_engine* e) {
   CK(cudaFuncSetAttribute(ssdk::retention_decode_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
   CK(cudaFuncSetAttribute(ssdk::sandwich_step_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
   CK(cudaFuncSetAttribute(ssdk::sandwich_step_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
-  CK(cudaFuncSetAttribute(ssdk::gqa_head_prep_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
-  CK(cudaFuncSetAttribute(ssdk::gqa_head_prep_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_head_prep_kernel<T, 4, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_head_prep_kernel<T, 4, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
+  CK(cudaFuncSetAttribute(ssdk::gqa_head_prep_kernel<T, 1, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)); \
   CK(cudaFuncSetAttribute(ssdk::gqa_decode_merge_diff_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, big));
   SSDK_ROW_ATTR(bf16) SSDK_ROW_ATTR(float)
 #undef SSDK_ROW_ATTR

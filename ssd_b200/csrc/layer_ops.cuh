@@ -88,6 +88,28 @@ SSDK_DEVINL void st_contig(T* p, const float* f) {
   for (int i = 0; i < kBytes / 16; ++i) reinterpret_cast<uint4*>(p)[i] = make_uint4(w[4 * i], w[4 * i + 1], w[4 * i + 2], w[4 * i + 3]);
 }
 
+// VEC channels per thread and step
+template <int VEC> SSDK_DEVINL void ld_vec(const float* p, float* f) {
+  if constexpr (VEC == 4) { const float4 v = *reinterpret_cast<const float4*>(p); f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
+  else f[0] = *p;
+}
+template <int VEC> SSDK_DEVINL void st_vec(float* p, const float* f) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
+
+// VEC floats -> storage type (VEC = 4: p is aligned to 4 elements)
+template <typename T, int VEC> SSDK_DEVINL void st_row(T* p, const float* f) {
+  if constexpr (VEC == 4 && sizeof(T) == 2) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(f[0], f[1]), hi = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+  } else if constexpr (VEC == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    st_f<T>(p, f[0]);
+  }
+}
+
 template <typename T>
 __global__ void embed_rows_kernel(const int* __restrict__ ids, const T* __restrict__ embed, float* __restrict__ x, int width,
                                   int vocab, float scale, T* __restrict__ xt, int copies) {
@@ -156,13 +178,19 @@ SSDK_DEVINL float act_f(float g) {
 }
 
 // z [rows, ldz] fp32 with gate columns [0, ff) and up columns [ff, 2 ff) -> y [rows, ff] (T) = act(gate) * up; rows at
-// and beyond *n_rows (optional, on the device) are skipped
-template <typename T, int ACT>
+// and beyond *n_rows (optional, on the device) are skipped.  VEC = 4: ff, ldz and the pointers are whole groups of four
+template <typename T, int ACT, int VEC>
 __global__ void glu_act_kernel(const float* __restrict__ z, int ldz, T* __restrict__ y, int ff, const int* __restrict__ n_rows) {
   const int r = blockIdx.x;
   if (n_rows && r >= *n_rows) return;
-  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ff; c += gridDim.y * blockDim.x)   // (columns may be spread over gridDim.y)
-    st_f<T>(y + (size_t)r * ff + c, act_f<ACT>(z[(size_t)r * ldz + c]) * z[(size_t)r * ldz + ff + c]);
+  for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; c < ff; c += gridDim.y * blockDim.x * VEC) {   // (columns may be spread over gridDim.y)
+    float g[VEC], u[VEC];
+    ld_vec<VEC>(z + (size_t)r * ldz + c, g);
+    ld_vec<VEC>(z + (size_t)r * ldz + ff + c, u);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) g[e] = act_f<ACT>(g[e]) * u[e];
+    st_row<T, VEC>(y + (size_t)r * ff + c, g);
+  }
 }
 
 // z [rows, ff] fp32, b [ff] (T, optional) -> y [rows, ff] (T) = act(z + b)
@@ -366,28 +394,6 @@ struct StreamStepArgs {
   int S, width;
   float eps, offset;
 };
-
-// VEC channels per thread and step
-template <int VEC> SSDK_DEVINL void ld_vec(const float* p, float* f) {
-  if constexpr (VEC == 4) { const float4 v = *reinterpret_cast<const float4*>(p); f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
-  else f[0] = *p;
-}
-template <int VEC> SSDK_DEVINL void st_vec(float* p, const float* f) {
-  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  else *p = f[0];
-}
-
-// VEC floats -> storage type (VEC = 4: p is aligned to 4 elements)
-template <typename T, int VEC> SSDK_DEVINL void st_row(T* p, const float* f) {
-  if constexpr (VEC == 4 && sizeof(T) == 2) {
-    const __nv_bfloat162 lo = __floats2bfloat162_rn(f[0], f[1]), hi = __floats2bfloat162_rn(f[2], f[3]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
-  } else if constexpr (VEC == 4) {
-    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  } else {
-    st_f<T>(p, f[0]);
-  }
-}
 
 // grid (M).  SM >= S: streams held in registers; VEC = 4 needs a width that is a multiple of 4.  dynamic shared memory: width floats
 template <typename T, int SM, int VEC>

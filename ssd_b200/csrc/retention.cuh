@@ -168,11 +168,12 @@ __global__ void __launch_bounds__(256) retention_chunk_out_any_kernel(const Rete
 }
 
 // ------------------------------------------------------------------------------------------------ walk over the chunks
-// grid (n_seqs, ceil(H D V / (256 VEC))), 256 threads: VEC entries of the state per thread, eight chunks requested ahead
+constexpr int kRetScanThreads = 128;
+// grid (n_seqs, ceil(H D V / (kRetScanThreads VEC))): VEC entries of the state per thread, eight chunks requested at a time
 template <int VEC>
-__global__ void __launch_bounds__(256) retention_state_scan_kernel(const RetentionArgs p, const Ragged rg) {
+__global__ void __launch_bounds__(kRetScanThreads) retention_state_scan_kernel(const RetentionArgs p, const Ragged rg) {
   const int s = blockIdx.x, rows = rg.cu[s + 1] - rg.cu[s];
-  const size_t HDV = (size_t)p.H * p.D * p.V, e0 = ((size_t)blockIdx.y * 256 + threadIdx.x) * VEC;
+  const size_t HDV = (size_t)p.H * p.D * p.V, e0 = ((size_t)blockIdx.y * kRetScanThreads + threadIdx.x) * VEC;
   if (rows < 2 || e0 >= HDV) return;
   const float* pw = p.pw + e0 / ((size_t)p.D * p.V) * (kRetChunk + 1);   // (VEC divides V: one head)
   const int nc = (rows + kRetChunk - 1) / kRetChunk;
@@ -202,39 +203,50 @@ __global__ void __launch_bounds__(256) retention_state_scan_kernel(const Retenti
 }
 
 // ------------------------------------------------------------------------------------------------ tensor-core form
-// fp32 rows -> two bf16 tiles (x = hi + lo) of ROWS x COLS (row stride COLS + 8); zero beyond n rows and `cols` columns; w (optional):
-// a factor per row
+// A ROWS x COLS tile of fp32 rows on its way to two bf16 tiles (x = hi + lo, row stride COLS + 8): `fetch` requests it all (zero beyond
+// n rows and `cols` columns), `put` splits it into shared memory, so that a tile's loads run under the products before it
 template <int ROWS, int COLS>
-SSDK_DEVINL void ret_split(const float* src, size_t ld, int n, int cols, const float* w, int w_step, bool vec, __nv_bfloat16* hi, __nv_bfloat16* lo) {
-  constexpr int LD = COLS + 8, Q = COLS / 4;
-#pragma unroll 4
-  for (int e = threadIdx.x; e < ROWS * Q; e += 256) {
-    const int r = e / Q, c = e % Q * 4;
-    float f[4] = {0.f, 0.f, 0.f, 0.f};
-    if (r < n) {
-      if (vec) {
-        if (c < cols) ld_vec<4>(src + (size_t)r * ld + c, f);
-      } else {
+struct RetFetch {
+  static constexpr int Q = COLS / 4, N = ROWS * Q / 256, LD = COLS + 8;
+  static_assert(ROWS * Q % 256 == 0, "whole rounds of 256 threads");
+  float f[N][4];
+  SSDK_DEVINL void fetch(const float* src, size_t ld, int n, int cols, bool vec) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
-          if (c + i < cols) f[i] = src[(size_t)r * ld + c + i];
-      }
-      if (w) {
-        const float wr = w[r * w_step];
+    for (int i = 0; i < N; ++i) {
+      const int e = threadIdx.x + i * 256, r = e / Q, c = e % Q * 4;
+      f[i][0] = f[i][1] = f[i][2] = f[i][3] = 0.f;
+      if (r < n) {
+        if (vec) {
+          if (c < cols) ld_vec<4>(src + (size_t)r * ld + c, f[i]);
+        } else {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) f[i] *= wr;
+          for (int j = 0; j < 4; ++j)
+            if (c + j < cols) f[i][j] = src[(size_t)r * ld + c + j];
+        }
       }
     }
-    uint32_t h[2], l[2];
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      h[i] = pack_bf16x2(f[2 * i], f[2 * i + 1]);
-      l[i] = pack_bf16x2(f[2 * i] - __uint_as_float(h[i] << 16), f[2 * i + 1] - __uint_as_float(h[i] & 0xffff0000u));
-    }
-    *reinterpret_cast<uint2*>(hi + r * LD + c) = make_uint2(h[0], h[1]);
-    *reinterpret_cast<uint2*>(lo + r * LD + c) = make_uint2(l[0], l[1]);
   }
-}
+  // w (optional): a factor per row, w[r * step]; rows from n on are zero already
+  SSDK_DEVINL void put(__nv_bfloat16* hi, __nv_bfloat16* lo, const float* w = nullptr, int step = 0, int n = ROWS) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const int e = threadIdx.x + i * 256, r = e / Q, c = e % Q * 4;
+      if (w) {
+        const float wr = r < n ? w[r * step] : 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) f[i][j] *= wr;
+      }
+      uint32_t h[2], l[2];
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        h[j] = pack_bf16x2(f[i][2 * j], f[i][2 * j + 1]);
+        l[j] = pack_bf16x2(f[i][2 * j] - __uint_as_float(h[j] << 16), f[i][2 * j + 1] - __uint_as_float(h[j] & 0xffff0000u));
+      }
+      *reinterpret_cast<uint2*>(hi + r * LD + c) = make_uint2(h[0], h[1]);
+      *reinterpret_cast<uint2*>(lo + r * LD + c) = make_uint2(l[0], l[1]);
+    }
+  }
+};
 // c += (ah + al) (bh + bl) without the product of the two low terms
 SSDK_DEVINL void ret_mma(float* c, const uint32_t* ah, const uint32_t* al, const uint32_t* bh, const uint32_t* bl) {
   mma_bf16_16816(c, al, bh[0], bh[1]);
@@ -254,9 +266,14 @@ __global__ void __launch_bounds__(256, 2) retention_chunk_state_mma_kernel(const
   if (rg.cu[s + 1] - rg.cu[s] < 2 || left <= 0) return;
   const int n = min(left, kRetChunk), H = p.H, D = p.D, V = p.V, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   T *kh = (T*)rs_sm, *kl = kh + kRetChunk * LDK, *vh = kl + kRetChunk * LDK, *vl = vh + kRetChunk * LDV;
-  ret_split<kRetChunk, KS * 16>(p.qk + (size_t)r0 * 2 * H * D + (size_t)(H + hd) * D, (size_t)2 * H * D, n, D,
-                                p.pw + (size_t)hd * (kRetChunk + 1) + n - 1, -1, p.vec, kh, kl);
-  ret_split<kRetChunk, VT * 8>(p.z + (size_t)r0 * p.ldz + 2 * (size_t)H * D + (size_t)hd * V, p.ldz, n, V, nullptr, 0, p.vec, vh, vl);
+  {
+    RetFetch<kRetChunk, KS * 16> fk;
+    RetFetch<kRetChunk, VT * 8> fv;
+    fk.fetch(p.qk + (size_t)r0 * 2 * H * D + (size_t)(H + hd) * D, (size_t)2 * H * D, n, D, p.vec);
+    fv.fetch(p.z + (size_t)r0 * p.ldz + 2 * (size_t)H * D + (size_t)hd * V, p.ldz, n, V, p.vec);
+    fk.put(kh, kl, p.pw + (size_t)hd * (kRetChunk + 1) + n - 1, -1, n);
+    fv.put(vh, vl);
+  }
   __syncthreads();
   float* out = p.chunks + ((size_t)(ret_record(rg, s) + c) * H + hd) * D * V;
   // operand addresses of this lane: k is read transposed (rows of the result are its columns)
@@ -312,8 +329,21 @@ __global__ void __launch_bounds__(256, 2) retention_chunk_out_mma_kernel(const R
   const size_t ldq = (size_t)2 * H * D;
   const float* q = p.qk + (size_t)r0 * ldq + (size_t)hd * D;
   if (tid <= kRetChunk) s_pw[tid] = p.pw[(size_t)hd * (kRetChunk + 1) + tid];
-  ret_split<kRetChunk, KS * 16>(q, ldq, n, D, nullptr, 0, p.vec, qh, ql);
-  ret_split<kRetChunk, KS * 16>(q + (size_t)H * D, ldq, n, D, nullptr, 0, p.vec, kh, kl);
+  {
+    RetFetch<kRetChunk, KS * 16> fq, fk;
+    fq.fetch(q, ldq, n, D, p.vec);
+    fk.fetch(q + (size_t)H * D, ldq, n, D, p.vec);
+    fq.put(qh, ql);
+    fk.put(kh, kl);
+  }
+  // the first slab of the state is on its way under the scores, the next one (at last v) under the products with the one before
+  const bool carried = c > 0 || rg.pos0[s] > 0;
+  const float* S = p.chunks + ((size_t)(ret_record(rg, s) + c) * H + hd) * D * V;
+  const float* v = p.z + (size_t)r0 * p.ldz + 2 * (size_t)H * D + (size_t)hd * V;
+  RetFetch<kSlab, VT * 8> fs;
+  RetFetch<kRetChunk, VT * 8> fv;
+  if (carried) fs.fetch(S, V, D, V, p.vec);
+  else fv.fetch(v, p.ldz, n, V, p.vec);
   __syncthreads();
   const int qa = (rt * 16 + (lane & 15)) * LDK + (lane >> 4) * 8;          // this lane's rows of q
   // scores of the warp's 16 rows against its 32 keys
@@ -350,10 +380,13 @@ __global__ void __launch_bounds__(256, 2) retention_chunk_out_mma_kernel(const R
 #pragma unroll
   for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
   const int va = (((lane >> 3) & 1) * 8 + (lane & 7)) * LDV + (lane >> 4) * 8 + half * NT * 8;   // this lane's rows of a value tile
-  if (c > 0 || rg.pos0[s] > 0) {   // q . S, a slab of the state's rows at a time
-    const float* S = p.chunks + ((size_t)(ret_record(rg, s) + c) * H + hd) * D * V;
-    for (int d0 = 0; d0 < D; d0 += kSlab) {
-      ret_split<kSlab, VT * 8>(S + (size_t)d0 * V, V, D - d0, V, nullptr, 0, p.vec, vh, vl);
+  if (carried) {   // q . S, a slab of the state's rows at a time
+#pragma unroll
+    for (int d0 = 0; d0 < KS * 16; d0 += kSlab) {
+      if (d0 >= D) break;
+      fs.put(vh, vl);
+      if (d0 + kSlab < D) fs.fetch(S + (size_t)(d0 + kSlab) * V, V, D - d0 - kSlab, V, p.vec);
+      else fv.fetch(v, p.ldz, n, V, p.vec);
       __syncthreads();
 #pragma unroll
       for (int k = 0; k < kSlab / 16; ++k) {
@@ -375,7 +408,7 @@ __global__ void __launch_bounds__(256, 2) retention_chunk_out_mma_kernel(const R
 #pragma unroll
     for (int j = 0; j < NT; ++j) { acc[j][0] *= f0; acc[j][1] *= f0; acc[j][2] *= f1; acc[j][3] *= f1; }
   }
-  ret_split<kRetChunk, VT * 8>(p.z + (size_t)r0 * p.ldz + 2 * (size_t)H * D + (size_t)hd * V, p.ldz, n, V, nullptr, 0, p.vec, vh, vl);
+  fv.put(vh, vl);
   __syncthreads();
   for (int k = 0; k <= rt; ++k) {   // keys at and before the warp's rows
     uint32_t ah[4], al[4];
@@ -441,14 +474,27 @@ __global__ void __launch_bounds__(kRetDecWarps * 32) retention_decode_kernel(con
   float* cs = k + D;                            // [2 half]
   float* o = cs + D;                            // [V]
   const float* z = p.z + (size_t)row * p.ldz;
+  const float* v = z + 2 * (size_t)H * D + (size_t)hd * V;
+  float* S = p.S + (size_t)rg.slot[s] * p.slot_stride + (size_t)hd * D * V;
+  const bool carried = pos > 0;
+  // a warp's next kRows rows of the state, columns c .., requested before they are needed: the first under the rotation
+  constexpr int kRows = 8;
+  float st[kRows][VEC];
+  auto fetch = [&](int d0, int c) {
+#pragma unroll
+    for (int i = 0; i < kRows; ++i) {
+      const int d = d0 + i * kRetDecWarps;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st[i][e] = 0.f;
+      if (carried && d < D && c < V) ld_vec<VEC>(S + (size_t)d * V + c, st[i]);
+    }
+  };
+  fetch(warp, lane * VEC);
   row_angles(cs, half, pos, p.inv_freq, 1.f);
   __syncthreads();
   if (warp < 2) head_row<float, float, 1>(z + (size_t)(warp * H + hd) * D, warp ? k : q, D, half, cs, (const float*)nullptr, 1.f, warp ? p.k_scale : 1.f, lane);
   __syncthreads();
   const float a = p.pw[(size_t)hd * (kRetChunk + 1) + 1];
-  const float* v = z + 2 * (size_t)H * D + (size_t)hd * V;
-  float* S = p.S + (size_t)rg.slot[s] * p.slot_stride + (size_t)hd * D * V;
-  const bool carried = pos > 0;
   float ss = 0.f;
   for (int v0 = 0; v0 < V; v0 += 32 * VEC) {
     const int c = v0 + lane * VEC;
@@ -457,16 +503,18 @@ __global__ void __launch_bounds__(kRetDecWarps * 32) retention_decode_kernel(con
     for (int e = 0; e < VEC; ++e) { acc[e] = 0.f; vv[e] = 0.f; }
     if (c < V) {
       ld_vec<VEC>(v + c, vv);
-#pragma unroll 8
-      for (int d = warp; d < D; d += kRetDecWarps) {
-        float st[VEC];
+      if (v0 > 0) fetch(warp, c);
+      for (int d0 = warp; d0 < D; d0 += kRows * kRetDecWarps) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) st[e] = 0.f;
-        if (carried) ld_vec<VEC>(S + (size_t)d * V + c, st);
-        const float kd = k[d], qd = q[d];
+        for (int i = 0; i < kRows; ++i) {
+          const int d = d0 + i * kRetDecWarps;
+          if (d >= D) break;
+          const float kd = k[d], qd = q[d];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) { st[e] = fmaf(a, st[e], kd * vv[e]); acc[e] = fmaf(qd, st[e], acc[e]); }
-        st_vec<VEC>(S + (size_t)d * V + c, st);
+          for (int e = 0; e < VEC; ++e) { st[i][e] = fmaf(a, st[i][e], kd * vv[e]); acc[e] = fmaf(qd, st[i][e], acc[e]); }
+          st_vec<VEC>(S + (size_t)d * V + c, st[i]);
+        }
+        if (d0 + kRows * kRetDecWarps < D) fetch(d0 + kRows * kRetDecWarps, c);
       }
     }
 #pragma unroll
